@@ -35,6 +35,7 @@ class NormSpec:
     kind: str = "rmsnorm"
     param_name: str = "weight"     # checkpoint name of the weight relative to the norm's prefix ("" : the prefix itself)
     offset: float = 0.0            # the norm multiplies by offset + stored weight (1.0: a weight stored around zero)
+    scalar: bool = False           # the stored weight is a single number (shape []) for all coordinates
 
 
 @dataclass(frozen=True)
@@ -146,7 +147,9 @@ class RoutedMLPSpec:
     its "output" or its "input".  `correction`: whether the checkpoint holds a correction of the choice.  `score` "softmax_chosen": the
     router's outputs themselves are ranked and the chosen experts' weights are the softmax over the chosen outputs alone; with it
     go `expert` "silu" weighted at the "output".  `router_bias`: the router's outputs get a stored bias.  `shared_size` > 0: one
-    more expert of that size (of the routed experts' form) runs for every token with weight 1."""
+    more expert of that size (of the routed experts' form) runs for every token with weight 1, or with `shared_gate` times
+    sigmoid of a projection of the input, one number per token.  `group_score`: a group's score is its "best" choice score or
+    the sum of its best "pair".  `normalize`: the chosen experts' scores are divided by their sum."""
     hidden_size: int
     expert_size: int
     num_experts: int
@@ -163,6 +166,9 @@ class RoutedMLPSpec:
     correction: bool = True
     router_bias: bool = False
     shared_size: int = 0
+    shared_gate: bool = False
+    group_score: str = "best"
+    normalize: bool = False
     kind: str = "routed_mlp"
 
 
@@ -289,6 +295,51 @@ class MixerPairSpec:
 
 
 @dataclass(frozen=True)
+class GatedAttentionSpec:
+    """Grouped-query attention with an output gate per element: q, k, v (with biases if `proj_bias`); `qk_norm` "row" (whole q
+    and k rows, a weight per column), "head_unit" (every head, no weight) or "none"; `position`: rotation in halves; scores times
+    `softmax_scale`, position i sees j with 0 <= i - j < window (None: every j <= i); `sink_zero`: one is added to the softmax's
+    denominator (a sink of score 0); the heads' outputs times sigmoid of a projection of the input, element by element."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    softmax_scale: float
+    norm_eps: float
+    window: int | None = None
+    position: RopeSpec | None = None
+    proj_bias: bool = False
+    qk_norm: str = "none"
+    sink_zero: bool = False
+    kind: str = "gated_attention"
+
+
+@dataclass(frozen=True)
+class MambaSpec:
+    """Selective scan with a decay per (channel, state): [x | z] = W_in h; x through a causal convolution with bias and silu;
+    [low | B | C] = W_x x; dt = softplus(W_dt low + b); S <- exp(-dt exp(A_log)) S + dt x B, y = S C + D x; W_o (y silu(z))."""
+    hidden_size: int
+    inner_size: int
+    state_size: int
+    dt_rank: int
+    conv_kernel: int
+    kind: str = "mamba"
+
+
+@dataclass(frozen=True)
+class HGRN2Spec:
+    """Linear attention whose forget gate also decides what is written: q = silu(.), f = l + (1 - l) sigmoid(.) per key channel
+    with a stored lower bound l, S <- diag(f) S + (1 - f) v^T, o = S^T q, RMS-normed per head (one weight for all heads)."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    norm_eps: float
+    kind: str = "hgrn2"
+
+
+@dataclass(frozen=True)
 class MinGRUSpec:
     """A gated recurrence per channel whose gates read the current token only: S <- (1 - z) S + z c with z = sigmoid(.),
     c = u + 1/2 (u >= 0) or sigmoid(u) (u < 0); output product over S * silu(gate)."""
@@ -389,7 +440,8 @@ class OutNormBlockSpec:
 @dataclass(frozen=True)
 class StreamBlockSpec:
     """Pre-norm block on a 32-bit stream: x <- x + s1 * mixer(norm(x)); with a feed-forward x <- x + s2 * ff(norm(x))
-    (s1, s2: a stored scale per channel, when `layer_scale`); then, with `side`, the token's side input."""
+    (s1, s2: a stored scale per channel, when `layer_scale`); then, with `side`, the token's side input.  `input_conv` > 0: the
+    mixer reads h + conv(h) instead of the normed rows h, conv a causal convolution per channel of so many taps."""
     prefix: str
     mixer: MixerSlot
     mixer_norm: NormSpec
@@ -402,6 +454,8 @@ class StreamBlockSpec:
     layer_scale_names: tuple[str, str] = ("ls1", "ls2")
     side: TokenSideSpec | None = None
     side_name: str = "side."
+    input_conv: int = 0
+    input_conv_name: str = "canon1"
     kind: str = "prenorm_stream"
 
 
@@ -424,6 +478,14 @@ class StreamInputSpec:
     is stored at the model's root under `name`."""
     hidden_size: int
     name: str
+    kind: str = "product"
+
+
+@dataclass(frozen=True)
+class StreamAddSpec:
+    """x <- x + x0 on a 32-bit stream, x0 the embedding's output as the stream began with it.  It has no tensors."""
+    hidden_size: int
+    kind: str = "add"
 
 
 @dataclass(frozen=True)

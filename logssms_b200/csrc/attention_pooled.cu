@@ -14,7 +14,8 @@
 //   Two options turn the same kernels into other attentions.  `pool` = 0: there are no blocks (with a window beyond
 //   every position: plain causal attention).  `slopes` (a number per query head): m_h * (i - j) is taken off the scaled
 //   score of token j.  `sinks` (a number per query head): exp(sink_h) joins the softmax's denominator, with no key and no
-//   value.  Without rotation tables (`v_rot` = 0) values are summed as they are cached.
+//   value.  Without rotation tables (`v_rot` = 0) values are summed as they are cached.  `gate` (a row of logits per token,
+//   one per output column): every output column is multiplied by sigmoid of its logit before it is rounded and stored.
 //
 //   pooled_prepare : per (token, head): rotate the query; rotate key and value and store them at the token's slot
 //   normed_prepare : per (token, head): RMS-norm the query and the key over the head's columns with a weight each
@@ -209,11 +210,19 @@ __device__ __forceinline__ int blocks_behind(int i, int window, int pool) {
     return pool > 0 ? max(0, (i - window + 1) / pool) : 0;
 }
 
-// what two options add to a softmax: a slope per head on the distance to a token, a sink per head in the denominator
+// what the options add to an attention: a slope per head on the distance to a token, a sink per head in the denominator, a
+// gate per output column
 struct ScoreExtras {
     const float* slopes;      // [Hq] or null
     const float* sinks;       // [Hq] or null
+    const void* gate;         // [tokens, Hq * vdim] view of logits in the activation dtype, or null
+    long gate_stride;
 };
+
+template <typename T>
+__device__ __forceinline__ float gate_factor(const ScoreExtras& e, size_t token, size_t column) {
+    return 1.f / (1.f + expf(-to_f32(((const T*)e.gate)[token * e.gate_stride + column])));
+}
 
 // (maximum, sum, weighted values scaled by `f`) of a softmax once the sink has joined it
 __device__ __forceinline__ void join_sink(float sink, float& m, float& l, float& f) {
@@ -310,6 +319,7 @@ __global__ void __launch_bounds__(kWarps * 32) pooled_attention_kernel(
                 const float co = cs[c >> 1], si = cs[half + (c >> 1)];
                 val = (c & 1) ? own * co - partner * si : own * co + partner * si;
             }
+            if (extras.gate != nullptr) val *= gate_factor<T>(extras, t, (size_t)head * vdim + c);
             out[((size_t)t * Hq + head) * vdim + c] = from_f32<T>(val);
         }
     }
@@ -320,7 +330,7 @@ extern "C" int lb_pooled_attention(const void* q, const void* k_cache, const voi
                                    int pooled_width, const int* token_req, const int* positions, const int* token_list,
                                    int num_tokens, const float* v_table, int v_rot, int table_rows, void* out, int Hq, int Hkv,
                                    int dim, int vdim, int page_size, float scale, int window, int pool, const float* slopes,
-                                   const float* sinks, int dtype, void* stream) {
+                                   const float* sinks, const void* gate, long gate_stride, int dtype, void* stream) {
     if (num_tokens <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || dim <= 0 || vdim <= 0 || page_size <= 0 || window <= 0 || pool < 0 || (v_rot & 1)
         || v_rot > vdim || table_rows <= 0)
@@ -330,7 +340,7 @@ extern "C" int lb_pooled_attention(const void* q, const void* k_cache, const voi
     LB_DISPATCH_DTYPE(dtype, pooled_attention_kernel<T><<<grid, kWarps * 32, (size_t)kWarps * dim * sizeof(float), (cudaStream_t)stream>>>(
         (const T*)q, (const T*)k_cache, (const T*)v_cache, (const T*)kp_cache, (const T*)vp_cache, block_table, table_width,
         pooled_table, pooled_width, token_req, positions, token_list, v_table, v_rot, table_rows, (T*)out, Hq, Hkv, dim, vdim,
-        page_size, scale, window, pool, ScoreExtras{slopes, sinks}));
+        page_size, scale, window, pool, ScoreExtras{slopes, sinks, gate, gate_stride}));
     return launch_status();
 }
 
@@ -492,7 +502,8 @@ template <typename T>
 __global__ void __launch_bounds__(32) pooled_merge_kernel(const float* __restrict__ partial, const int* __restrict__ positions,
                                                           const int* __restrict__ token_list, const float* __restrict__ v_table, int v_rot,
                                                           int table_rows, T* __restrict__ out, int Hq, int vdim, int splits,
-                                                          const float* __restrict__ sinks) {
+                                                          ScoreExtras extras) {
+    const float* sinks = extras.sinks;
     const int lane = threadIdx.x, slot = blockIdx.x, head = blockIdx.y;
     const int t = token_list != nullptr ? token_list[slot] : slot;
     if (t < 0) return;
@@ -525,6 +536,7 @@ __global__ void __launch_bounds__(32) pooled_merge_kernel(const float* __restric
                 const float co = cs[c >> 1], si = cs[half + (c >> 1)];
                 val = (c & 1) ? own * co - partner * si : own * co + partner * si;
             }
+            if (extras.gate != nullptr) val *= gate_factor<T>(extras, t, (size_t)head * vdim + c);
             out[((size_t)t * Hq + head) * vdim + c] = from_f32<T>(val);
         }
     }
@@ -553,7 +565,8 @@ extern "C" int lb_pooled_attention_split(const void* q, const void* k_cache, con
                                          int pooled_width, const int* token_req, const int* positions, const int* token_list,
                                          int num_tokens, const float* v_table, int v_rot, int table_rows, float* partial, void* out,
                                          int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
-                                         int splits, const float* slopes, const float* sinks, int dtype, void* stream) {
+                                         int splits, const float* slopes, const float* sinks, const void* gate, long gate_stride,
+                                         int dtype, void* stream) {
     if (num_tokens <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || dim <= 0 || dim % 4 || vdim <= 0 || page_size <= 0 || window <= 0 || pool < 0 || (v_rot & 1)
         || v_rot > vdim || table_rows <= 0 || splits <= 0 || splits > 65535 || Hq > 65535)
@@ -563,13 +576,14 @@ extern "C" int lb_pooled_attention_split(const void* q, const void* k_cache, con
     int code;
 #define LB_SPLIT(PER) LB_DISPATCH_DTYPE(dtype, code = (launch_split<T, PER>(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, \
         pooled_table, pooled_width, token_req, positions, token_list, num_tokens, partial, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits, \
-        ScoreExtras{slopes, nullptr}, stream)))
+        ScoreExtras{slopes, nullptr, nullptr, 0}, stream)))
     if (per == 1) { LB_SPLIT(1); } else if (per == 2) { LB_SPLIT(2); } else { LB_SPLIT(4); }
 #undef LB_SPLIT
     if (code != 0) return code;
     dim3 grid(num_tokens, Hq);
     LB_DISPATCH_DTYPE(dtype, pooled_merge_kernel<T><<<grid, 32, 0, (cudaStream_t)stream>>>(partial, positions, token_list, v_table, v_rot,
-                                                                                           table_rows, (T*)out, Hq, vdim, splits, sinks));
+                                                                                           table_rows, (T*)out, Hq, vdim, splits,
+                                                                                           ScoreExtras{nullptr, sinks, gate, gate_stride}));
     return launch_status();
 }
 
@@ -803,11 +817,13 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         if (r_lo < n_q) {
             float u = o[n][0] * inv_lo, v = o[n][1] * inv_lo;
             if (c < v_rot) { const float co = cs_lo[c >> 1], si = cs_lo[half + (c >> 1)]; const float u2 = u * co + v * si; v = v * co - u * si; u = u2; }
+            if (extras.gate != nullptr) { u *= gate_factor<__nv_bfloat16>(extras, row0 + r_lo, (size_t)head * vdim + c); v *= gate_factor<__nv_bfloat16>(extras, row0 + r_lo, (size_t)head * vdim + c + 1); }
             *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r_lo) * Hq + head) * vdim + c) = pack_bf16(u, v);
         }
         if (r_hi < n_q) {
             float u = o[n][2] * inv_hi, v = o[n][3] * inv_hi;
             if (c < v_rot) { const float co = cs_hi[c >> 1], si = cs_hi[half + (c >> 1)]; const float u2 = u * co + v * si; v = v * co - u * si; u = u2; }
+            if (extras.gate != nullptr) { u *= gate_factor<__nv_bfloat16>(extras, row0 + r_hi, (size_t)head * vdim + c); v *= gate_factor<__nv_bfloat16>(extras, row0 + r_hi, (size_t)head * vdim + c + 1); }
             *reinterpret_cast<uint32_t*>(out + ((size_t)(row0 + r_hi) * Hq + head) * vdim + c) = pack_bf16(u, v);
         }
     }
@@ -865,15 +881,17 @@ extern "C" int lb_pooled_attention_tile(const void* q, const void* k_cache, cons
                                         int pooled_width, const int* cu, const int* start_pos, const int* tiles, int num_tiles,
                                         const int* positions, int tokens, const float* v_table, int v_rot, int table_rows, void* out,
                                         int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
-                                        float* partial, int splits, const float* slopes, const float* sinks, void* stream) {
+                                        float* partial, int splits, const float* slopes, const float* sinks, const void* gate,
+                                        long gate_stride, void* stream) {
     // (with several CTAs per run the sink joins in the merge, once)
     const int code = tile_dispatch(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, pooled_table, pooled_width, cu,
                                    start_pos, tiles, num_tiles, v_table, v_rot, table_rows, out, Hq, Hkv, dim, vdim, page_size, scale,
-                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks}, stream);
+                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks, gate, gate_stride}, stream);
     if (code != 0 || splits <= 1 || num_tiles <= 0 || tokens <= 0) return code;
     dim3 grid(tokens, Hq);
     pooled_merge_kernel<__nv_bfloat16><<<grid, 32, 0, (cudaStream_t)stream>>>(partial, positions, nullptr, v_table, v_rot, table_rows,
-                                                                            (__nv_bfloat16*)out, Hq, vdim, splits, sinks);
+                                                                            (__nv_bfloat16*)out, Hq, vdim, splits,
+                                                                            ScoreExtras{nullptr, sinks, gate, gate_stride});
     return launch_status();
 }
 
@@ -989,6 +1007,127 @@ extern "C" int lb_rownorm_prepare(const void* qk, long row_stride, const int* po
     LB_DISPATCH_DTYPE(dtype, rownorm_prepare_kernel<T><<<tokens, 256, 0, (cudaStream_t)stream>>>(
         (const T*)qk, row_stride, positions, slot_mapping, table, rot, table_rows, wq, wk, eps, (T*)q_out, (T*)k_cache, (T*)v_cache,
         Hq, Hkv, dim, write_kv));
+    return launch_status();
+}
+
+// ------------------------------------------------------------------------------------------------------------------
+//   qk_prepare : per token, from qkv = [q (Hq * dim) | k (Hkv * dim) | v (Hkv * vdim)]: q and k normed (`norm` 0: not at all;
+//                1: by the root mean square of the whole q or k row, all heads at once, times a weight per column of the
+//                row; 2: by the root mean square of every head's columns; weights may be null), then rotated in halves: of every
+//                head's first `rot` columns, column i and column i + rot / 2 turn by the angle of the token's table row (cos |
+//                sin of rot / 2 pairs).  (A rotation keeps a head's root mean square: norm 2 before or after it is the same.)
+//                q to q_out, k and v to the caches at the token's slot.  Norms and rotation are 32-bit.
+// V columns move at a time (V = 2: even dim, vdim and rot / 2).
+template <typename T, int V>
+__global__ void __launch_bounds__(256) qk_prepare_kernel(const T* __restrict__ qkv, long row_stride, const int* __restrict__ positions,
+                                                         const int* __restrict__ slot_mapping, const float* __restrict__ table, int rot,
+                                                         int table_rows, const float* __restrict__ wq, const float* __restrict__ wk, int norm,
+                                                         float eps, T* __restrict__ q_out, T* __restrict__ k_cache, T* __restrict__ v_cache,
+                                                         int Hq, int Hkv, int dim, int vdim, int write_kv) {
+    extern __shared__ float head_inv[];                      // [Hq + Hkv]
+    __shared__ float red[32];
+    const size_t t = blockIdx.x;
+    const T* row = qkv + t * row_stride;
+    const int nq = Hq * dim, nk = Hkv * dim, nv = Hkv * vdim;
+    auto load = [&](const T* p, float (&f)[V]) {
+        if (V == 2 && sizeof(T) == 2) {
+            const float2 v2 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+            f[0] = v2.x; f[V - 1] = v2.y;
+        } else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) f[e] = to_f32(p[e]);
+        }
+    };
+    auto store = [&](T* p, const float (&f)[V]) {
+        if (V == 2 && sizeof(T) == 2) *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(f[0], f[V - 1]);
+        else {
+#pragma unroll
+            for (int e = 0; e < V; ++e) p[e] = from_f32<T>(f[e]);
+        }
+    };
+    float inv_q = 1.f, inv_k = 1.f;
+    if (norm == 1) {
+        float sq = 0.f, sk = 0.f, f[V];
+        for (int c = threadIdx.x * V; c < nq; c += blockDim.x * V) { load(row + c, f);
+#pragma unroll
+            for (int e = 0; e < V; ++e) sq += f[e] * f[e]; }
+        for (int c = threadIdx.x * V; c < nk; c += blockDim.x * V) { load(row + nq + c, f);
+#pragma unroll
+            for (int e = 0; e < V; ++e) sk += f[e] * f[e]; }
+        inv_q = 1.f / sqrtf(block_sum(sq, red) / (float)nq + eps);
+        inv_k = 1.f / sqrtf(block_sum(sk, red) / (float)nk + eps);
+    } else if (norm == 2) {
+        const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
+        for (int h = warp; h < Hq + Hkv; h += nwarps) {
+            float ss = 0.f, f[V];
+            for (int c = lane * V; c < dim; c += 32 * V) { load(row + (size_t)h * dim + c, f);
+#pragma unroll
+                for (int e = 0; e < V; ++e) ss += f[e] * f[e]; }
+            ss = warp_sum(ss);
+            if (lane == 0) head_inv[h] = 1.f / sqrtf(ss / (float)dim + eps);
+        }
+        __syncthreads();
+    }
+    const float* cs = table + (size_t)min(max(positions[t], 0), table_rows - 1) * rot;
+    const int half = rot >> 1;
+    const long slot = write_kv ? (long)slot_mapping[t] : -1;
+    for (int c = threadIdx.x * V; c < nq + nk; c += blockDim.x * V) {
+        const bool is_q = c < nq;
+        if (!is_q && slot < 0) continue;
+        const int cc = is_q ? c : c - nq;                    // column of the whole q (or k) row
+        const int d = cc % dim;                              // column of its head
+        const float* w = is_q ? wq : wk;
+        const int wrap = norm == 2 ? dim : 1 << 30;          // norm 2: one weight per column of a head
+        const float inv = norm == 2 ? head_inv[c / dim] : (is_q ? inv_q : inv_k);
+        float val[V];
+        load(row + c, val);
+#pragma unroll
+        for (int e = 0; e < V; ++e) val[e] *= inv * (w != nullptr ? w[(cc + e) % wrap] : 1.f);
+        if (d < rot) {
+            const bool second = d >= half;
+            const int pd = second ? -half : half;
+            float partner[V];
+            load(row + c + pd, partner);
+#pragma unroll
+            for (int e = 0; e < V; ++e) {
+                const float pv = partner[e] * inv * (w != nullptr ? w[(cc + pd + e) % wrap] : 1.f);
+                const int i = (second ? d - half : d) + e;
+                const float co = cs[i], si = cs[half + i];
+                val[e] = second ? val[e] * co + pv * si : val[e] * co - pv * si;
+            }
+        }
+        if (is_q) store(q_out + t * nq + cc, val);
+        else store(k_cache + (size_t)slot * nk + cc, val);
+    }
+    if (slot < 0) return;
+    for (int c = threadIdx.x * V; c < nv; c += blockDim.x * V) {
+        float f[V];
+        load(row + nq + nk + c, f);
+        store(v_cache + (size_t)slot * nv + c, f);
+    }
+}
+
+// qkv: [tokens, >= (Hq + Hkv) * dim + Hkv * vdim] (column view allowed); table: float32 [table_rows, rot] (rot 0: no rotation);
+// wq, wk: float32 [Hq * dim], [Hkv * dim] (norm 1) or [dim] each (norm 2), or null
+extern "C" int lb_qk_prepare(const void* qkv, long row_stride, const int* positions, const int* slot_mapping, const float* table, int rot,
+                             int table_rows, const float* wq, const float* wk, int norm, float eps, void* q_out, void* k_cache,
+                             void* v_cache, int tokens, int Hq, int Hkv, int dim, int vdim, int write_kv, int dtype, void* stream) {
+    if (tokens <= 0) return kOk;
+    if (Hq <= 0 || Hkv <= 0 || Hq + Hkv > 8192 || dim <= 0 || vdim <= 0 || rot < 0 || rot > dim || (rot & 1) || table_rows <= 0 || norm < 0 || norm > 2)
+        return kBadSize;
+    const size_t smem = (size_t)(Hq + Hkv) * sizeof(float);
+    const bool pairs = dtype == kBF16 && dim % 2 == 0 && vdim % 2 == 0 && rot % 4 == 0 && row_stride % 2 == 0 && ((uintptr_t)qkv & 3) == 0
+                       && ((uintptr_t)q_out & 3) == 0 && ((uintptr_t)k_cache & 3) == 0 && ((uintptr_t)v_cache & 3) == 0;
+    if (pairs) {
+        typedef __nv_bfloat16 bf;
+        qk_prepare_kernel<bf, 2><<<tokens, 256, smem, (cudaStream_t)stream>>>(
+            (const bf*)qkv, row_stride, positions, slot_mapping, table, rot, table_rows, wq, wk, norm, eps, (bf*)q_out, (bf*)k_cache, (bf*)v_cache,
+            Hq, Hkv, dim, vdim, write_kv);
+        return launch_status();
+    }
+    LB_DISPATCH_DTYPE(dtype, qk_prepare_kernel<T, 1><<<tokens, 256, smem, (cudaStream_t)stream>>>(
+        (const T*)qkv, row_stride, positions, slot_mapping, table, rot, table_rows, wq, wk, norm, eps, (T*)q_out, (T*)k_cache, (T*)v_cache,
+        Hq, Hkv, dim, vdim, write_kv));
     return launch_status();
 }
 

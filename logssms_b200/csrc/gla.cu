@@ -5,13 +5,20 @@
 //   S_t     = diag(a_t) S_{t-1} + k_t v_t^T            (S: [key channels, value channels] per head, 32-bit)
 //   o_t     = S_t^T (q_t * q_scale)
 //
+//  With `lower` (a bound per key channel; `z_bias` is added to z) the decay is a forget gate that also decides what is
+//  written, and q passes silu first:
+//   a_t = lower + (1 - lower) sigmoid(z_t),   k_t = 1 - a_t = (1 - lower) sigmoid(-z_t),   q_t <- silu(q_t)
+//  The gate and the key made from it stay 32-bit: there is no key operand in memory.  In the chunked form, whose products
+//  take bfloat16 operands, the scaled queries and keys and the state's copy then enter as TWO bfloat16 terms each (hi =
+//  bf16(x), lo = bf16(x - hi)), so that they are applied to 16 bits and more instead of 8 (values are bfloat16 as projected).
+//
 //  gla_scan      : the recurrence over every request's tokens of a step, state read from and written back to the
 //                  request's slot (a request that starts at position 0 starts from zeros whatever the slot holds).
 //                  A CTA owns (request, head, a tile of value channels); a thread owns R state rows of one value
 //                  column, DS threads of a warp share a column.  q, k, the decays and v of 8 tokens at a time are
 //                  staged in shared memory, so the inner loop touches registers and shared memory only.
 //  gla_norm_gate : y = o / sqrt(mean_head(o^2) + eps) * w[c] * act(g), o in 32-bit, w shared by the heads; act is
-//                  silu or the sigmoid.  With one "head" of the full width it is the gated norm over all heads together.
+//                  silu or the sigmoid (without g: no gate).  With one "head" of the full width it is the gated norm over all heads together.
 #include "lb200/common.cuh"
 using namespace lb200;
 
@@ -21,12 +28,25 @@ __device__ __forceinline__ float log_sigmoid(float z) {
     return z < 0.f ? z - log1pf(expf(z)) : -log1pf(expf(-z));
 }
 
+// A forget gate with a lower bound: the decay a = l + (1 - l) sigmoid(z), its logarithm, and the key k = 1 - a.  The
+// logarithm is taken from k where a is near one and stays finite where a underflows.
+struct BoundedGate {
+    const float* lower;       // [H * dim], or null: the decays are of another kind
+    const float* bias;        // [H * dim] added to z, or null
+};
+__device__ __forceinline__ float gate_key(float z, float l) { return (1.f - l) / (1.f + expf(z)); }
+__device__ __forceinline__ float gate_decay(float z, float l) { return l + (1.f - l) / (1.f + expf(-z)); }
+__device__ __forceinline__ float gate_log_decay(float z, float l, float key) {
+    if (key < 0.5f) return log1pf(-key);
+    return l > 0.f ? logf(gate_decay(z, l)) : log_sigmoid(z);
+}
+
 template <typename T, int R, int DS>
 __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long row_stride,
                                 const float* __restrict__ z, float* __restrict__ o, float* state,
                                 const int* __restrict__ cu, const int* __restrict__ start_pos, const int* __restrict__ slots,
                                 const int* __restrict__ request_list, int H, int dim, int vdim, float inv_tau, float q_scale,
-                                const float* __restrict__ head_decay) {
+                                const float* __restrict__ head_decay, BoundedGate gate) {
     constexpr int DP = R * DS;                       // key channels, padded
     extern __shared__ float sm[];
     const int cols = blockDim.x / DS;
@@ -57,8 +77,16 @@ __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k
             if (d < dim) {
                 const size_t row = (size_t)(t0 + tt);
                 qv = to_f32(q[row * row_stride + h * dim + d]) * q_scale;
-                kv = to_f32(k[row * row_stride + h * dim + d]);
-                av = head_decay != nullptr ? head_decay[h] : expf(log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau);
+                if (gate.lower != nullptr) {
+                    const float l = gate.lower[h * dim + d];
+                    const float zz = z[(row * H + h) * dim + d] + (gate.bias != nullptr ? gate.bias[h * dim + d] : 0.f);
+                    qv = silu_f(qv);
+                    kv = gate_key(zz, l);
+                    av = gate_decay(zz, l);
+                } else {
+                    kv = to_f32(k[row * row_stride + h * dim + d]);
+                    av = head_decay != nullptr ? head_decay[h] : expf(log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau);
+                }
             }
             qs[i] = qv; ks[i] = kv; as[i] = av;
         }
@@ -93,7 +121,8 @@ __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k
 template <typename T, int R, int DS>
 static int launch_gla_scan(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                            const int* cu, const int* start_pos, const int* slots, const int* request_list, int num_requests,
-                           int H, int dim, int vdim, float inv_tau, float q_scale, const float* head_decay, cudaStream_t stream) {
+                           int H, int dim, int vdim, float inv_tau, float q_scale, const float* head_decay, BoundedGate gate,
+                           cudaStream_t stream) {
     // few requests: narrow tiles, so that more CTAs share the work
     const int want = (num_requests * H * ((vdim * DS + 127) / 128) < 148) ? 32 : 128;
     const int threads = min(want, (vdim * DS + 31) / 32 * 32);
@@ -103,21 +132,24 @@ static int launch_gla_scan(const void* q, const void* k, const void* v, long row
     static size_t have = 0;
     ensure_dynamic_smem(gla_scan_kernel<T, R, DS>, smem, have);
     gla_scan_kernel<T, R, DS><<<grid, threads, smem, stream>>>((const T*)q, (const T*)k, (const T*)v, row_stride, z, o, state, cu,
-                                                               start_pos, slots, request_list, H, dim, vdim, inv_tau, q_scale, head_decay);
+                                                               start_pos, slots, request_list, H, dim, vdim, inv_tau, q_scale, head_decay, gate);
     return launch_status();
 }
 
 // q, k: [tokens, H*dim] and v: [tokens, H*vdim], column views of one projection buffer (common row stride, in
-// elements); z: float32 [tokens, H*dim]; o: float32 [tokens, H*vdim]; state: float32 [slots, H, dim, vdim].
+// elements); z: float32 [tokens, H*dim]; o: float32 [tokens, H*vdim]; state: float32 [slots, H, dim, vdim].  With `lower`
+// (float32 [H*dim]; `z_bias` float32 [H*dim] or null) k is not read and q_scale must be 1.
 extern "C" int lb_gla_scan(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                            const int* cu, const int* start_pos, const int* slots, const int* request_list, int num_requests,
-                           int H, int dim, int vdim, float tau, float q_scale, const float* head_decay, int dtype, void* stream) {
+                           int H, int dim, int vdim, float tau, float q_scale, const float* head_decay, const float* lower,
+                           const float* z_bias, int dtype, void* stream) {
     if (num_requests <= 0) return kOk;
     if (H <= 0 || dim <= 0 || vdim <= 0 || !(tau > 0.f)) return kBadSize;
+    if (lower != nullptr && (z == nullptr || head_decay != nullptr || q_scale != 1.f)) return kBadSize;
     if (dim > 512) return kTooLarge;
     cudaStream_t st = (cudaStream_t)stream;
 #define LB_GLA(R_, DS_) LB_DISPATCH_DTYPE(dtype, return (launch_gla_scan<T, R_, DS_>(q, k, v, row_stride, z, o, state, cu, start_pos, \
-        slots, request_list, num_requests, H, dim, vdim, 1.f / tau, q_scale, head_decay, st)))
+        slots, request_list, num_requests, H, dim, vdim, 1.f / tau, q_scale, head_decay, BoundedGate{lower, z_bias}, st)))
     if (dim <= 16) { LB_GLA(16, 1); }
     else if (dim <= 32) { LB_GLA(32, 1); }
     else if (dim <= 64) { LB_GLA(64, 1); }
@@ -142,8 +174,12 @@ __global__ void gla_norm_gate_kernel(const float* __restrict__ o, const T* __res
     ss = block_sum(ss, red);
     const float inv = 1.f / sqrtf(ss / (float)vdim + eps);
     for (int c = threadIdx.x; c < vdim; c += blockDim.x) {
-        const float g = to_f32(gate[row * gate_stride + h * vdim + c]);
-        out[(row * H + h) * vdim + c] = from_f32<T>(orow[c] * inv * weight[c] * (sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g)));
+        float f = 1.f;
+        if (gate != nullptr) {
+            const float g = to_f32(gate[row * gate_stride + h * vdim + c]);
+            f = sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g);
+        }
+        out[(row * H + h) * vdim + c] = from_f32<T>(orow[c] * inv * weight[c] * f);
     }
 }
 
@@ -180,7 +216,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
         const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k, long row_stride, const float* __restrict__ z,
         const int* __restrict__ cu, const int* __restrict__ chunks, __nv_bfloat16* __restrict__ q_in,
         __nv_bfloat16* __restrict__ k_end, float* __restrict__ A, float* __restrict__ D, int H, int dim, float inv_tau,
-        float q_scale, const float* __restrict__ head_decay) {
+        float q_scale, const float* __restrict__ head_decay, BoundedGate gate, size_t plane) {
     extern __shared__ float sm[];
     float* b = sm;                         // [16][dim] log-decays, then their running sums
     float* qs = b + kChunk * dim;
@@ -195,9 +231,17 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
         float ld = 0.f, qv = 0.f, kv = 0.f;
         if (j < n) {
             const size_t row = (size_t)(t0 + j);
-            ld = head_decay != nullptr ? logf(head_decay[h]) : log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau;
             qv = to_f32(q[row * row_stride + h * dim + d]) * q_scale;
-            kv = to_f32(k[row * row_stride + h * dim + d]);
+            if (gate.lower != nullptr) {
+                const float l = gate.lower[h * dim + d];
+                const float zz = z[(row * H + h) * dim + d] + (gate.bias != nullptr ? gate.bias[h * dim + d] : 0.f);
+                qv = silu_f(qv);
+                kv = gate_key(zz, l);
+                ld = gate_log_decay(zz, l, kv);
+            } else {
+                ld = head_decay != nullptr ? logf(head_decay[h]) : log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau;
+                kv = to_f32(k[row * row_stride + h * dim + d]);
+            }
         }
         b[i] = ld; qs[i] = qv; ks[i] = kv;
     }
@@ -211,8 +255,14 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
     for (int i = threadIdx.x; i < n * dim; i += blockDim.x) {
         const int j = i / dim, d = i % dim;
         const size_t at = ((size_t)(t0 + j) * H + h) * dim + d;
-        q_in[at] = __float2bfloat16_rn(qs[i] * expf(b[i]));
-        k_end[at] = __float2bfloat16_rn(ks[i] * expf(b[(kChunk - 1) * dim + d] - b[i]));
+        const float qe = qs[i] * expf(b[i]), ke = ks[i] * expf(b[(kChunk - 1) * dim + d] - b[i]);
+        const __nv_bfloat16 qh = __float2bfloat16_rn(qe), kh = __float2bfloat16_rn(ke);
+        q_in[at] = qh;
+        k_end[at] = kh;
+        if (plane != 0) {                  // the second term of each operand, one plane further
+            q_in[plane + at] = __float2bfloat16_rn(qe - __bfloat162float(qh));
+            k_end[plane + at] = __float2bfloat16_rn(ke - __bfloat162float(kh));
+        }
     }
     // A: a warp per pair (i, j), its lanes over the key channels
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nwarps = blockDim.x >> 5;
@@ -243,12 +293,13 @@ __device__ __forceinline__ uint32_t pack2(__nv_bfloat16 lo, __nv_bfloat16 hi) {
 // MODE 1: a segment from a zero state, no output: leaves its end state in seg_state[item] and the product of its
 //         chunks' decays in seg_decay[item]; `gla_segment_pass` then turns the end states into start states;
 // MODE 2: a segment from seg_state[item], writing o.
-template <int MT, int MODE>
+// SPLIT: q_in and k_end hold two planes, the two bfloat16 terms of each operand, and the state's copy is made of two terms.
+template <int MT, int MODE, bool SPLIT>
 __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
         const __nv_bfloat16* __restrict__ q_in, const __nv_bfloat16* __restrict__ k_end, const __nv_bfloat16* __restrict__ v,
         long v_stride, const float* __restrict__ A, const float* __restrict__ D, float* __restrict__ o, float* state,
         const int* __restrict__ cu, const int* __restrict__ start_pos, const int* __restrict__ slots,
-        const int* __restrict__ per_request, int H, int dim, int vdim, float* seg_state, float* seg_decay) {
+        const int* __restrict__ per_request, int H, int dim, int vdim, float* seg_state, float* seg_decay, size_t plane) {
     constexpr int NT = kScanCols / 8;
     extern __shared__ __align__(16) unsigned char raw[];
     const int DP = dim + 8, VP = kScanCols + 8;
@@ -258,6 +309,10 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
     __nv_bfloat16* Vs = Sb + dim * VP;                                   // [16][VP]
     float* As = reinterpret_cast<float*>(Vs + kChunk * VP);              // [16][16]
     float* Ds = As + kChunk * kChunk;                                    // [dim]
+    // SPLIT: the second terms
+    __nv_bfloat16* Ql = reinterpret_cast<__nv_bfloat16*>(Ds + dim);      // [16][DP]
+    __nv_bfloat16* Kl = Ql + kChunk * DP;                                // [16][DP]
+    __nv_bfloat16* Sl = Kl + kChunk * DP;                                // [dim][VP]
     constexpr int W = MODE == 0 ? 3 : 4;
     const int req = per_request[W * blockIdx.z];
     if (req < 0) return;
@@ -285,7 +340,7 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
     // The next chunk's operands travel from global memory to registers while this chunk is computed (16-byte pieces of
     // q e^{b} and k e^{..}, which are contiguous; v, A and the chunk's decay by plain loads).
     constexpr int kQK = 4;                                 // 16-byte pieces of a [16][dim] tile per thread: dim <= 256
-    uint4 rq[kQK], rk[kQK];
+    uint4 rq[kQK], rk[kQK], rql[SPLIT ? kQK : 1], rkl[SPLIT ? kQK : 1];
     __nv_bfloat16 rv[4];
     float ra[2], rd[2];
     const int pieces = dim / 8;                            // per row
@@ -296,12 +351,17 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
         for (int u = 0; u < kQK; ++u) {
             const int i = threadIdx.x + u * 128;
             rq[u] = rk[u] = make_uint4(0, 0, 0, 0);
+            if (SPLIT) rql[u] = rkl[u] = make_uint4(0, 0, 0, 0);
             if (i < kChunk * pieces) {
                 const int j = i / pieces, pc = i % pieces;
                 if (j < n) {
                     const size_t at = ((size_t)(t0 + j) * H + h) * dim + pc * 8;
                     rq[u] = *reinterpret_cast<const uint4*>(q_in + at);
                     rk[u] = *reinterpret_cast<const uint4*>(k_end + at);
+                    if (SPLIT) {
+                        rql[u] = *reinterpret_cast<const uint4*>(q_in + plane + at);
+                        rkl[u] = *reinterpret_cast<const uint4*>(k_end + plane + at);
+                    }
                 }
             }
         }
@@ -330,6 +390,10 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
                 const int j = i / pieces, pc = i % pieces;
                 *reinterpret_cast<uint4*>(Qs + j * DP + pc * 8) = rq[u];
                 *reinterpret_cast<uint4*>(Ks + j * DP + pc * 8) = rk[u];
+                if (SPLIT) {
+                    *reinterpret_cast<uint4*>(Ql + j * DP + pc * 8) = rql[u];
+                    *reinterpret_cast<uint4*>(Kl + j * DP + pc * 8) = rkl[u];
+                }
             }
         }
 #pragma unroll
@@ -351,8 +415,14 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
                     const int c = nt * 8 + 2 * t;
-                    *reinterpret_cast<__nv_bfloat162*>(Sb + r0 * VP + c) = __floats2bfloat162_rn(S[m][nt][0], S[m][nt][1]);
-                    *reinterpret_cast<__nv_bfloat162*>(Sb + (r0 + 8) * VP + c) = __floats2bfloat162_rn(S[m][nt][2], S[m][nt][3]);
+                    const __nv_bfloat162 s0 = __floats2bfloat162_rn(S[m][nt][0], S[m][nt][1]), s1 = __floats2bfloat162_rn(S[m][nt][2], S[m][nt][3]);
+                    *reinterpret_cast<__nv_bfloat162*>(Sb + r0 * VP + c) = s0;
+                    *reinterpret_cast<__nv_bfloat162*>(Sb + (r0 + 8) * VP + c) = s1;
+                    if (SPLIT) {
+                        const float2 h0 = __bfloat1622float2(s0), h1 = __bfloat1622float2(s1);
+                        *reinterpret_cast<__nv_bfloat162*>(Sl + r0 * VP + c) = __floats2bfloat162_rn(S[m][nt][0] - h0.x, S[m][nt][1] - h0.y);
+                        *reinterpret_cast<__nv_bfloat162*>(Sl + (r0 + 8) * VP + c) = __floats2bfloat162_rn(S[m][nt][2] - h1.x, S[m][nt][3] - h1.y);
+                    }
                 }
             }
         }
@@ -370,6 +440,16 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
                 const uint32_t b0 = pack2(Sb[(kk + 2 * t) * VP + cw + g], Sb[(kk + 2 * t + 1) * VP + cw + g]);
                 const uint32_t b1 = pack2(Sb[(kk + 2 * t + 8) * VP + cw + g], Sb[(kk + 2 * t + 9) * VP + cw + g]);
                 mma_bf16_16816(acc, a, b0, b1);
+                if (SPLIT) {               // + hi lo + lo hi (lo lo is below 2^-16 of the product)
+                    const uint32_t c0 = pack2(Sl[(kk + 2 * t) * VP + cw + g], Sl[(kk + 2 * t + 1) * VP + cw + g]);
+                    const uint32_t c1 = pack2(Sl[(kk + 2 * t + 8) * VP + cw + g], Sl[(kk + 2 * t + 9) * VP + cw + g]);
+                    mma_bf16_16816(acc, a, c0, c1);
+                    a[0] = *reinterpret_cast<const uint32_t*>(Ql + g * DP + kk + 2 * t);
+                    a[1] = *reinterpret_cast<const uint32_t*>(Ql + (g + 8) * DP + kk + 2 * t);
+                    a[2] = *reinterpret_cast<const uint32_t*>(Ql + g * DP + kk + 2 * t + 8);
+                    a[3] = *reinterpret_cast<const uint32_t*>(Ql + (g + 8) * DP + kk + 2 * t + 8);
+                    mma_bf16_16816(acc, a, b0, b1);
+                }
             }
 #pragma unroll
             for (int e = 0; e < 4; ++e) {
@@ -390,12 +470,20 @@ __global__ void __launch_bounds__(128) gla_chunk_scan_kernel(
                 a[1] = pack2(Ks[(2 * t) * DP + r0 + 8], Ks[(2 * t + 1) * DP + r0 + 8]);
                 a[2] = pack2(Ks[(2 * t + 8) * DP + r0], Ks[(2 * t + 9) * DP + r0]);
                 a[3] = pack2(Ks[(2 * t + 8) * DP + r0 + 8], Ks[(2 * t + 9) * DP + r0 + 8]);
+                uint32_t al[4];
+                if (SPLIT) {
+                    al[0] = pack2(Kl[(2 * t) * DP + r0], Kl[(2 * t + 1) * DP + r0]);
+                    al[1] = pack2(Kl[(2 * t) * DP + r0 + 8], Kl[(2 * t + 1) * DP + r0 + 8]);
+                    al[2] = pack2(Kl[(2 * t + 8) * DP + r0], Kl[(2 * t + 9) * DP + r0]);
+                    al[3] = pack2(Kl[(2 * t + 8) * DP + r0 + 8], Kl[(2 * t + 9) * DP + r0 + 8]);
+                }
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
                     S[m][nt][0] *= d0; S[m][nt][1] *= d0; S[m][nt][2] *= d1; S[m][nt][3] *= d1;
                     const uint32_t b0 = pack2(Vs[(2 * t) * VP + nt * 8 + g], Vs[(2 * t + 1) * VP + nt * 8 + g]);
                     const uint32_t b1 = pack2(Vs[(2 * t + 8) * VP + nt * 8 + g], Vs[(2 * t + 9) * VP + nt * 8 + g]);
                     mma_bf16_16816(S[m][nt], a, b0, b1);
+                    if (SPLIT) mma_bf16_16816(S[m][nt], al, b0, b1);
                 }
             }
         }
@@ -444,32 +532,40 @@ __global__ void gla_segment_pass_kernel(float* seg_state, const float* __restric
 // the scan; chunks: int32 [num_chunks, 2] (request, first token within its portion; request -1: nothing);
 // per_request: int32 [num_long, 3] (request, its first chunk, its number of chunks).  Scratch: q_in, k_end
 // [tokens, H, dim] bfloat16, A float32 [tokens, H, 16], D float32 [num_chunks, H, dim].  dim: a multiple of 16, <= 256.
+// With `lower` (see `lb_gla_scan`) q_in and k_end have two planes of `tokens` rows each.
 extern "C" int lb_gla_chunked(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                               const int* cu, const int* start_pos, const int* slots, const int* chunks, int num_chunks,
                               const int* per_request, int num_long, void* q_in, void* k_end, float* A, float* D, int H, int dim,
                               int vdim, float tau, float q_scale, const int* segments, int num_segments, float* seg_state,
-                              float* seg_decay, const float* head_decay, void* stream) {
+                              float* seg_decay, const float* head_decay, const float* lower, const float* z_bias, int tokens,
+                              void* stream) {
     if (num_chunks <= 0 || num_long <= 0) return kOk;
+    if (lower != nullptr && (z == nullptr || head_decay != nullptr || q_scale != 1.f || tokens <= 0)) return kBadSize;
     if (H <= 0 || dim <= 0 || vdim <= 0 || !(tau > 0.f) || dim % 16) return kBadSize;
     if (dim > 256) return kTooLarge;
     cudaStream_t st = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
+    const bool split = lower != nullptr;
+    const size_t plane = split ? (size_t)tokens * H * dim : 0;
     {
         const size_t smem = (size_t)3 * kChunk * dim * sizeof(float);
         static size_t have = 0;
         ensure_dynamic_smem(gla_chunk_prepare_kernel, smem, have);
         gla_chunk_prepare_kernel<<<dim3(num_chunks, H), 128, smem, st>>>((const bf*)q, (const bf*)k, row_stride, z, cu, chunks,
-                                                                        (bf*)q_in, (bf*)k_end, A, D, H, dim, 1.f / tau, q_scale, head_decay);
+                                                                        (bf*)q_in, (bf*)k_end, A, D, H, dim, 1.f / tau, q_scale, head_decay,
+                                                                        BoundedGate{lower, z_bias}, plane);
         const int rc = launch_status();
         if (rc != 0) return rc;
     }
     const size_t smem = ((size_t)2 * kChunk * (dim + 8) + (size_t)dim * (kScanCols + 8) + (size_t)kChunk * (kScanCols + 8)) * sizeof(bf)
-                        + ((size_t)kChunk * kChunk + dim) * sizeof(float);
+                        + ((size_t)kChunk * kChunk + dim) * sizeof(float)
+                        + (split ? ((size_t)2 * kChunk * (dim + 8) + (size_t)dim * (kScanCols + 8)) * sizeof(bf) : 0);
     dim3 grid((vdim + kScanCols - 1) / kScanCols, H, num_long);
-#define LB_SCAN(MT_, MODE_, LIST_) { static size_t have = 0; ensure_dynamic_smem(gla_chunk_scan_kernel<MT_, MODE_>, smem, have); \
-        gla_chunk_scan_kernel<MT_, MODE_><<<grid, 128, smem, st>>>((const bf*)q_in, (const bf*)k_end, (const bf*)v, row_stride, A, D, o, \
-            state, cu, start_pos, slots, LIST_, H, dim, vdim, seg_state, seg_decay); }
-#define LB_SCAN_MODE(MODE_, LIST_) { if (dim <= 64) LB_SCAN(1, MODE_, LIST_) else if (dim <= 128) LB_SCAN(2, MODE_, LIST_) else LB_SCAN(4, MODE_, LIST_) }
+#define LB_SCAN(MT_, MODE_, SPLIT_, LIST_) { static size_t have = 0; ensure_dynamic_smem(gla_chunk_scan_kernel<MT_, MODE_, SPLIT_>, smem, have); \
+        gla_chunk_scan_kernel<MT_, MODE_, SPLIT_><<<grid, 128, smem, st>>>((const bf*)q_in, (const bf*)k_end, (const bf*)v, row_stride, A, D, o, \
+            state, cu, start_pos, slots, LIST_, H, dim, vdim, seg_state, seg_decay, plane); }
+#define LB_SCAN_MT(MODE_, SPLIT_, LIST_) { if (dim <= 64) LB_SCAN(1, MODE_, SPLIT_, LIST_) else if (dim <= 128) LB_SCAN(2, MODE_, SPLIT_, LIST_) else LB_SCAN(4, MODE_, SPLIT_, LIST_) }
+#define LB_SCAN_MODE(MODE_, LIST_) { if (split) LB_SCAN_MT(MODE_, true, LIST_) else LB_SCAN_MT(MODE_, false, LIST_) }
     if (segments == nullptr || num_segments <= 0) {
         LB_SCAN_MODE(0, per_request)
         return launch_status();
@@ -485,6 +581,7 @@ extern "C" int lb_gla_chunked(const void* q, const void* k, const void* v, long 
     if (rc != 0) return rc;
     LB_SCAN_MODE(2, segments)
 #undef LB_SCAN_MODE
+#undef LB_SCAN_MT
 #undef LB_SCAN
     return launch_status();
 }

@@ -6,7 +6,10 @@
 //                     n / groups neighbours) whose best member scores highest; the `top` best are chosen; their
 //                     weights are s * scale (no correction, no renormalisation).  With `sigmoid_scores` = 2 the
 //                     logits themselves are ranked and the chosen ones' weights are the softmax over the chosen
-//                     logits only (times scale).  `bias` (may be null) is added to the logits.  Writes the dense weights [T, n]
+//                     logits only (times scale).  `bias` (may be null) is added to the logits.  With `pair_groups` a
+//                     group's score is the sum of its two largest members instead of its largest; with `normalize` the
+//                     chosen weights are divided by their sum + 1e-20; `gates` further rows of W_r behind the n outputs
+//                     are no experts: the dense weights' last `gates` columns are the sigmoids of their logits.  Writes the dense weights [T, n + gates]
 //                     (0 where not chosen), the chosen indices and weights [T, top], and per token the summed
 //                     weight of the chosen identity experts (the last n - experts outputs).
 //  moe_activation   : y[t, e, i] = w[t, e] * g~ * sigmoid(act_alpha * g~) * (u~ + 1),  g~ = min(g, limit),
@@ -31,14 +34,16 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
         const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ correction,
         float* __restrict__ dense, int* __restrict__ chosen, float* __restrict__ chosen_w,
         float* __restrict__ id_weight, int tokens, int width, int n, int experts, int top,
-        int groups, int keep, float scale, int sigmoid_scores, const float* __restrict__ bias) {
+        int groups, int keep, float scale, int sigmoid_scores, const float* __restrict__ bias, int pair_groups, int normalize,
+        int gates) {
     __shared__ float z[kRouteMax];
     __shared__ float c[kRouteMax];
     __shared__ unsigned char ok[kRouteMax];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x;
     const T* hr = h + (size_t)t * width;
-    for (int e = warp; e < n; e += kRouteWarps) {
+    const int nd = n + gates;                              // columns of the dense weights
+    for (int e = warp; e < nd; e += kRouteWarps) {
         const float* wr = w_router + (size_t)e * width;
         float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
         int k = lane;
@@ -51,7 +56,10 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
         }
         for (; k < width; k += 32) a0 += to_f32(hr[k]) * wr[k];
         const float a = warp_sum((a0 + a1) + (a2 + a3));
-        if (lane == 0) z[e] = a + (bias != nullptr ? bias[e] : 0.f);
+        if (lane == 0) {
+            if (e < n) z[e] = a + (bias != nullptr ? bias[e] : 0.f);
+            else dense[(size_t)t * nd + e] = 1.f / (1.f + expf(-a));
+        }
     }
     __syncthreads();
     if (warp != 0) return;
@@ -74,19 +82,24 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
         // meet in a score that has rounded to 1
         c[e] = (sigmoid_scores && correction == nullptr) ? logit : s + (correction != nullptr ? correction[e] : 0.f);
         ok[e] = 0;
-        dense[(size_t)t * n + e] = 0.f;
+        dense[(size_t)t * nd + e] = 0.f;
     }
     __syncwarp();
     if (lane != 0) return;
-    // the groups that stay: `keep` times the group whose best member is largest (ties: the lower index)
+    // the groups that stay: `keep` times the group whose best member (or best two) is largest (ties: the lower index)
     const int per = n / groups;
     for (int r = 0; r < keep; ++r) {
         int best_g = -1;
         float best = -INFINITY;
         for (int g = 0; g < groups; ++g) {
             if (ok[g * per]) continue;
-            float gm = -INFINITY;
-            for (int i = 0; i < per; ++i) gm = fmaxf(gm, c[g * per + i]);
+            float gm = -INFINITY, second = -INFINITY;
+            for (int i = 0; i < per; ++i) {
+                const float v = c[g * per + i];
+                if (v > gm) { second = gm; gm = v; }
+                else second = fmaxf(second, v);
+            }
+            if (pair_groups && per > 1) gm += second;
             if (best_g < 0 || gm > best) { best = gm; best_g = g; }
         }
         if (best_g < 0) break;
@@ -114,38 +127,47 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
             if (e < 0) continue;
             const float wgt = chosen_w[(size_t)t * top + r] / total * scale;
             chosen_w[(size_t)t * top + r] = wgt;
-            dense[(size_t)t * n + e] = wgt;
+            dense[(size_t)t * nd + e] = wgt;
             if (e >= experts) idw += wgt;
         }
         id_weight[t] = idw;
         return;
     }
+    float total = 0.f;
     for (int r = 0; r < top; ++r) {
         int best_e = -1;
         float best = -INFINITY;
         for (int e = 0; e < n; ++e)
             if (ok[e] == 1 && (best_e < 0 || c[e] > best)) { best = c[e]; best_e = e; }
-        if (best_e < 0) { chosen[(size_t)t * top + r] = -1; chosen_w[(size_t)t * top + r] = 0.f; continue; }
-        ok[best_e] = 2;
-        const float wgt = z[best_e] * scale;
-        dense[(size_t)t * n + best_e] = wgt;
         chosen[(size_t)t * top + r] = best_e;
+        if (best_e < 0) { chosen_w[(size_t)t * top + r] = 0.f; continue; }
+        ok[best_e] = 2;
+        total += z[best_e];
+    }
+    const float factor = normalize ? scale / (total + 1e-20f) : scale;
+    for (int r = 0; r < top; ++r) {
+        const int e = chosen[(size_t)t * top + r];
+        if (e < 0) continue;
+        const float wgt = z[e] * factor;
+        dense[(size_t)t * nd + e] = wgt;
         chosen_w[(size_t)t * top + r] = wgt;
-        if (best_e >= experts) idw += wgt;
+        if (e >= experts) idw += wgt;
     }
     id_weight[t] = idw;
 }
 
 extern "C" int lb_moe_route(const void* h, const float* w_router, const float* correction, float* dense, int* chosen,
                             float* chosen_w, float* id_weight, int tokens, int width, int n, int experts, int top, int groups,
-                            int keep, float scale, int sigmoid_scores, const float* bias, int dtype, void* stream) {
+                            int keep, float scale, int sigmoid_scores, const float* bias, int pair_groups, int normalize, int gates,
+                            int dtype, void* stream) {
     if (tokens <= 0) return kOk;
     if (n <= 0 || experts < 0 || experts > n || top <= 0 || top > n || groups <= 0 || n % groups || keep <= 0 || keep > groups)
         return kBadSize;
     if (n > kRouteMax) return kTooLarge;
-    if (sigmoid_scores < 0 || sigmoid_scores > 2) return kBadSize;
+    if (sigmoid_scores < 0 || sigmoid_scores > 2 || gates < 0 || (sigmoid_scores == 2 && normalize)) return kBadSize;
     LB_DISPATCH_DTYPE(dtype, moe_route_kernel<T><<<tokens, kRouteWarps * 32, 0, (cudaStream_t)stream>>>(
-        (const T*)h, w_router, correction, dense, chosen, chosen_w, id_weight, tokens, width, n, experts, top, groups, keep, scale, sigmoid_scores, bias));
+        (const T*)h, w_router, correction, dense, chosen, chosen_w, id_weight, tokens, width, n, experts, top, groups, keep, scale, sigmoid_scores, bias,
+        pair_groups, normalize, gates));
     return launch_status();
 }
 

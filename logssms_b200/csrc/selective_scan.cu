@@ -1,0 +1,290 @@
+// Selective scan with a decay of its own for every (channel, state): the recurrence of Mamba's first form.
+//
+//   dt_t[c]   = softplus(w_t[c] + dt_bias[c])           w_t: the step's projection (32-bit, as handed in or made here)
+//   S[c, n]  <- exp(dt_t[c] A[c, n]) S[c, n] + dt_t[c] x_t[c] B_t[n]            A = -exp(A_log); S float32
+//   y_t[c]    = (sum_n S[c, n] C_t[n] + D[c] x_t[c]) * silu(z_t[c])             (uses the updated state)
+//
+// x, B, C and the gate z are activations; step size, decays, state and sums are float32 in every dtype.  The decays
+// are exp2(dt * A log2(e)), one per (token, channel, state): the exponential unit bounds the kernel on long portions.
+//
+//  A CTA of 128 threads owns 128 / LN neighbouring channels of one request; LN lanes of a warp share a channel, each
+//  with NPT neighbouring states in registers.  Tokens go through in blocks of TB: x, dt, z of the CTA's channels and the
+//  block's B and C travel to registers while the block before is computed, then to shared memory, where the step
+//  size, its product with x and D x are worked out once per (token, channel); the loop over the tokens touches shared
+//  memory and registers only; the outputs leave through shared memory in rows of neighbouring channels.
+//
+//  selective_scan          : a request's tokens from its slot's state to its slot's state (a request that starts at
+//                            position 0 starts from zeros whatever the slot holds).  With `dt_w` the step's
+//                            low-rank projection rides along: w = dt_w low_t, the LN lanes of a channel sharing its row.
+//  selective_scan_segments : long portions cut into segments that run side by side, two launches.  The first runs every
+//                            request's first segment from the slot's state with its outputs, and every later segment
+//                            but the last from zero, without outputs, leaving its end state and the sum of its step
+//                            sizes (the product of its decays is exp(A * sum)).  In the second every later segment
+//                            joins the segments before it into its start state and runs with outputs; the last one
+//                            leaves the request's state in its slot.
+#include "lb200/common.cuh"
+using namespace lb200;
+
+namespace {
+constexpr int kThreads = 128;
+constexpr float kLog2e = 1.4426950408889634f;
+
+struct ScanArgs {
+    const void* x; long x_stride;          // [tokens, inner] view
+    const float* w;                        // [tokens, inner] the step's projection, or null: made from `low` and `dt_w`
+    const void* low; long low_stride;      // [tokens, rank + 2 * n] view: low-rank step | B | C
+    const void* dt_w;                      // [inner, rank]
+    const float* dt_bias; const float* A_log; const float* D;
+    const void* gate; long gate_stride;    // z: [tokens, inner] view
+    float* state;                          // [slots, inner, n]
+    void* y;                               // [tokens, inner]
+    const int* cu; const int* start_pos; const int* slots;
+    const int* list;                       // requests to run, or (segments) int32 [items, 4]
+    int inner, n, rank;
+    int seg_tokens; float* seg_state; float* seg_dt;
+};
+
+__device__ __forceinline__ float ex2(float v) {
+    float r;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(v));
+    return r;
+}
+__device__ __forceinline__ float softplus_f(float v) { return v > 20.f ? v : log1pf(expf(v)); }
+
+// PASS 0: whole portions; 1, 2: the two launches over segments
+template <typename T, int LN, int NPT, int TB, int PASS>
+__global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
+    constexpr int CH = kThreads / LN, NP = LN * NPT;
+    constexpr int KX = (TB * CH + kThreads - 1) / kThreads, KB = (TB * 2 * NP + kThreads - 1) / kThreads;
+    __shared__ __align__(16) float Bs[TB][NP], Cs[TB][NP];
+    __shared__ float dts[TB][CH], us[TB][CH], ys[TB][CH];
+    const int ch = threadIdx.x / LN, ln = threadIdx.x % LN;
+    const int c0 = blockIdx.x * CH, c = c0 + ch;
+    const bool c_ok = c < a.inner;
+    int b, first, last, seg = 0;
+    bool with_out = true, last_seg = true;
+    if (PASS == 0) {
+        b = a.list != nullptr ? a.list[blockIdx.y] : blockIdx.y;
+        if (b < 0) return;
+        first = a.cu[b];
+        last = a.cu[b + 1];
+    } else {
+        b = a.list[4 * blockIdx.y];
+        if (b < 0) return;
+        const int t0 = a.list[4 * blockIdx.y + 3], begin = a.cu[b], len = a.cu[b + 1] - begin;
+        seg = t0 / a.seg_tokens;
+        last_seg = t0 + a.seg_tokens >= len;
+        if (PASS == 1 ? (seg > 0 && last_seg) : seg == 0) return;
+        first = begin + t0;
+        last = begin + min(len, t0 + a.seg_tokens);
+        with_out = PASS == 2 || seg == 0;
+    }
+    if (first >= last) return;
+    float A2[NPT], S[NPT];
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) {
+        const int s = ln * NPT + i;
+        A2[i] = (c_ok && s < a.n) ? -expf(a.A_log[(size_t)c * a.n + s]) * kLog2e : 0.f;
+        S[i] = 0.f;
+    }
+    float* slot_state = a.state + ((size_t)a.slots[b] * a.inner + (c_ok ? c : 0)) * a.n;
+    if (PASS != 2) {
+        if (seg == 0 && a.start_pos[b] > 0 && c_ok) {
+#pragma unroll
+            for (int i = 0; i < NPT; ++i) if (ln * NPT + i < a.n) S[i] = slot_state[ln * NPT + i];
+        }
+    } else if (c_ok) {
+        // the segments before this one, joined in order (the first one's end state holds what the slot held)
+        for (int g = 0; g < seg; ++g) {
+            const size_t item = blockIdx.y - seg + g;
+            const float sum = g == 0 ? 0.f : a.seg_dt[item * a.inner + c];
+            const float* e = a.seg_state + (item * a.inner + c) * a.n;
+#pragma unroll
+            for (int i = 0; i < NPT; ++i)
+                if (ln * NPT + i < a.n) S[i] = (g == 0 ? 0.f : ex2(sum * A2[i]) * S[i]) + e[ln * NPT + i];
+        }
+    }
+    const T* x = (const T*)a.x;
+    const T* low = (const T*)a.low;
+    const T* gate = (const T*)a.gate;
+    float rx[KX], rw[KX], rz[KX], rb[KB];
+    auto fetch = [&](int t0) {
+        const int nt = min(TB, last - t0);
+#pragma unroll
+        for (int k = 0; k < KX; ++k) {
+            const int i = threadIdx.x + k * kThreads, t = i / CH, cc = c0 + i % CH;
+            rx[k] = rw[k] = rz[k] = 0.f;
+            if (t < nt && cc < a.inner) {
+                rx[k] = to_f32(x[(size_t)(t0 + t) * a.x_stride + cc]);
+                if (a.w != nullptr) rw[k] = a.w[(size_t)(t0 + t) * a.inner + cc];
+                if (with_out) rz[k] = to_f32(gate[(size_t)(t0 + t) * a.gate_stride + cc]);
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < KB; ++k) {
+            const int i = threadIdx.x + k * kThreads, t = i / (2 * NP), r = i % (2 * NP);
+            const int s = r < NP ? r : r - NP;
+            rb[k] = (t < nt && s < a.n) ? to_f32(low[(size_t)(t0 + t) * a.low_stride + a.rank + (r < NP ? 0 : a.n) + s]) : 0.f;
+        }
+    };
+    fetch(first);
+    float dt_sum = 0.f;
+    for (int t0 = first; t0 < last; t0 += TB) {
+        const int nt = min(TB, last - t0);
+        __syncthreads();                                   // the block before has left shared memory
+        if (a.w == nullptr) {
+            // w = dt_w low: the lanes of a channel share its row of dt_w
+            for (int t = 0; t < nt; ++t) {
+                float acc = 0.f;
+                if (c_ok)
+                    for (int r = ln; r < a.rank; r += LN)
+                        acc += to_f32(((const T*)a.dt_w)[(size_t)c * a.rank + r]) * to_f32(low[(size_t)(t0 + t) * a.low_stride + r]);
+#pragma unroll
+                for (int off = 1; off < LN; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+                if (ln == 0) dts[t][ch] = acc;
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int k = 0; k < KX; ++k) {
+            const int i = threadIdx.x + k * kThreads, t = i / CH, cl = i % CH;
+            if (t < TB) {
+                const int cc = c0 + cl;
+                float dt = 0.f, d = 0.f;
+                if (t < nt && cc < a.inner) {
+                    dt = softplus_f((a.w != nullptr ? rw[k] : dts[t][cl]) + a.dt_bias[cc]);
+                    d = a.D[cc];
+                }
+                dts[t][cl] = dt;
+                us[t][cl] = dt * rx[k];
+                ys[t][cl] = d * rx[k];
+            }
+        }
+#pragma unroll
+        for (int k = 0; k < KB; ++k) {
+            const int i = threadIdx.x + k * kThreads, t = i / (2 * NP), r = i % (2 * NP);
+            if (t < TB) {
+                if (r < NP) Bs[t][r] = rb[k];
+                else Cs[t][r - NP] = rb[k];
+            }
+        }
+        float z[KX];
+#pragma unroll
+        for (int k = 0; k < KX; ++k) z[k] = rz[k];
+        if (t0 + TB < last) fetch(t0 + TB);
+        __syncthreads();
+        if (with_out) {
+#pragma unroll 4
+            for (int t = 0; t < nt; ++t) {
+                const float dt = dts[t][ch], u = us[t][ch];
+                float acc = 0.f;
+#pragma unroll
+                for (int i = 0; i < NPT; i += 4) {
+                    const float4 bv = *reinterpret_cast<const float4*>(&Bs[t][ln * NPT + i]);
+                    const float4 cv = *reinterpret_cast<const float4*>(&Cs[t][ln * NPT + i]);
+                    S[i] = ex2(dt * A2[i]) * S[i] + u * bv.x;
+                    S[i + 1] = ex2(dt * A2[i + 1]) * S[i + 1] + u * bv.y;
+                    S[i + 2] = ex2(dt * A2[i + 2]) * S[i + 2] + u * bv.z;
+                    S[i + 3] = ex2(dt * A2[i + 3]) * S[i + 3] + u * bv.w;
+                    acc += S[i] * cv.x + S[i + 1] * cv.y + S[i + 2] * cv.z + S[i + 3] * cv.w;
+                }
+#pragma unroll
+                for (int off = 1; off < LN; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
+                if (ln == 0) ys[t][ch] += acc;
+            }
+            __syncthreads();
+#pragma unroll
+            for (int k = 0; k < KX; ++k) {
+                const int i = threadIdx.x + k * kThreads, t = i / CH, cc = c0 + i % CH;
+                if (t < nt && cc < a.inner)
+                    ((T*)a.y)[(size_t)(t0 + t) * a.inner + cc] = from_f32<T>(ys[t][i % CH] * (sizeof(T) == 2 ? silu_fast(z[k]) : silu_f(z[k])));
+            }
+        } else {
+#pragma unroll 4
+            for (int t = 0; t < nt; ++t) {
+                const float dt = dts[t][ch], u = us[t][ch];
+                dt_sum += dt;
+#pragma unroll
+                for (int i = 0; i < NPT; i += 4) {
+                    const float4 bv = *reinterpret_cast<const float4*>(&Bs[t][ln * NPT + i]);
+                    S[i] = ex2(dt * A2[i]) * S[i] + u * bv.x;
+                    S[i + 1] = ex2(dt * A2[i + 1]) * S[i + 1] + u * bv.y;
+                    S[i + 2] = ex2(dt * A2[i + 2]) * S[i + 2] + u * bv.z;
+                    S[i + 3] = ex2(dt * A2[i + 3]) * S[i + 3] + u * bv.w;
+                }
+            }
+        }
+    }
+    if (!c_ok) return;
+    float* dst = slot_state;
+    if (PASS == 1 && !last_seg) {
+        dst = a.seg_state + ((size_t)blockIdx.y * a.inner + c) * a.n;
+        if (ln == 0) a.seg_dt[(size_t)blockIdx.y * a.inner + c] = dt_sum;
+    } else if (PASS == 2 && !last_seg) {
+        return;
+    }
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) if (ln * NPT + i < a.n) dst[ln * NPT + i] = S[i];
+}
+
+template <typename T, int LN, int NPT, int TB>
+int launch_sized(const ScanArgs& a, int items, bool segmented, cudaStream_t st) {
+    constexpr int CH = kThreads / LN;
+    dim3 grid((a.inner + CH - 1) / CH, items);
+    if (!segmented) {
+        selective_scan_kernel<T, LN, NPT, TB, 0><<<grid, kThreads, 0, st>>>(a);
+        return launch_status();
+    }
+    selective_scan_kernel<T, LN, NPT, TB, 1><<<grid, kThreads, 0, st>>>(a);
+    const int rc = launch_status();
+    if (rc != 0) return rc;
+    selective_scan_kernel<T, LN, NPT, TB, 2><<<grid, kThreads, 0, st>>>(a);
+    return launch_status();
+}
+
+template <typename T>
+int launch(const ScanArgs& a, int items, bool segmented, cudaStream_t st) {
+    if (a.n <= 4) return launch_sized<T, 1, 4, 4>(a, items, segmented, st);
+    if (a.n <= 8) return launch_sized<T, 2, 4, 8>(a, items, segmented, st);
+    if (a.n <= 16) return launch_sized<T, 4, 4, 16>(a, items, segmented, st);
+    if (a.n <= 32) return launch_sized<T, 8, 4, 16>(a, items, segmented, st);
+    if (a.n <= 64) return launch_sized<T, 8, 8, 16>(a, items, segmented, st);
+    if (a.n <= 128) return launch_sized<T, 16, 8, 8>(a, items, segmented, st);
+    if (a.n <= 256) return launch_sized<T, 32, 8, 8>(a, items, segmented, st);
+    return kTooLarge;
+}
+
+bool sizes_ok(const ScanArgs& a) {
+    return a.inner > 0 && a.n > 0 && a.rank >= 0 && a.x_stride >= a.inner && a.gate_stride >= a.inner && a.low_stride >= a.rank + 2 * (long)a.n
+           && (a.w != nullptr || a.dt_w != nullptr);
+}
+}  // namespace
+
+// w: float32 [tokens, inner] (the step's projection without its bias), or null with dt_w [inner, rank] in the activation
+// dtype; state sizes up to 256; `requests` counts `list` (int32 request indices, -1: nothing) or, without a list, the batch.
+extern "C" int lb_selective_scan(const void* x, long x_stride, const float* w, const void* low, long low_stride, const void* dt_w,
+                                 const float* dt_bias, const float* A_log, const float* D, const void* gate, long gate_stride,
+                                 float* state, void* y, const int* cu, const int* start_pos, const int* slots, const int* list,
+                                 int requests, int inner, int n, int rank, int dtype, void* stream) {
+    if (requests <= 0) return kOk;
+    ScanArgs a{x, x_stride, w, low, low_stride, dt_w, dt_bias, A_log, D, gate, gate_stride, state, y, cu, start_pos, slots, list,
+               inner, n, rank, 0, nullptr, nullptr};
+    if (!sizes_ok(a) || requests > 65535) return kBadSize;
+    LB_DISPATCH_DTYPE(dtype, return launch<T>(a, requests, false, (cudaStream_t)stream));
+    return kOk;
+}
+
+// segments: int32 [items, 4] (request, -, -, first token within its portion), a request's segments of seg_tokens tokens one
+// after the other; request -1: nothing.  seg_state: float32 scratch [items, inner, n]; seg_dt: float32 scratch [items, inner].
+extern "C" int lb_selective_scan_segments(const void* x, long x_stride, const float* w, const void* low, long low_stride,
+                                          const float* dt_bias, const float* A_log, const float* D, const void* gate, long gate_stride,
+                                          float* state, void* y, const int* cu, const int* start_pos, const int* slots,
+                                          const int* segments, int items, int seg_tokens, float* seg_state, float* seg_dt, int inner,
+                                          int n, int rank, int dtype, void* stream) {
+    if (items <= 0) return kOk;
+    ScanArgs a{x, x_stride, w, low, low_stride, nullptr, dt_bias, A_log, D, gate, gate_stride, state, y, cu, start_pos, slots, segments,
+               inner, n, rank, seg_tokens, seg_state, seg_dt};
+    if (!sizes_ok(a) || items > 65535 || seg_tokens <= 0) return kBadSize;
+    LB_DISPATCH_DTYPE(dtype, return launch<T>(a, items, true, (cudaStream_t)stream));
+    return kOk;
+}

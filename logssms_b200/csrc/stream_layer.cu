@@ -6,6 +6,10 @@
 //                     x_out = v (may be x itself), h = N(v) * w rounded to the activation dtype (what the next
 //                     sublayer's products read; N may be "none": h is v rounded)
 //   stream_add_many : v = x + sum_i s_i * y_i (up to four addends, a scalar each), x_out = v in place, h = N(v) * w
+//   stream_add_conv_step : stream_add_many for a decode batch (row t is the single new token of request t) whose normed row
+//                     also passes a short causal convolution per channel before it is stored: with u = N(v) * w rounded,
+//                       h = sum_j cw[c, j] * u_(t - taps + 1 + j)
+//                     from the request's saved inputs, which are shifted in place (zeros for a request at position 0)
 //   stream_pair_rows: [x rounded | x0] side by side, the input of a product over the stream and the rows it began as
 //   side_gate       : a = gelu_tanh(z) * e for the products z [tokens, dim] of a side input's gate (see below), for
 //                     steps of many tokens, whose two small products go to the library
@@ -152,6 +156,61 @@ extern "C" int lb_stream_add_many(float* x, const void* y0, const void* y1, cons
         static size_t have = 0;
         ensure_dynamic_smem(stream_add_many_kernel<T>, smem, have);
         stream_add_many_kernel<T><<<rows, threads, smem, (cudaStream_t)stream>>>(x, a, w, eps, (T*)h_out, H, kind);
+    });
+    return launch_status();
+}
+
+// cw: float32 [H, taps]; conv_state: [slots, H, taps - 1] in the activation dtype
+template <typename T>
+__global__ void stream_add_conv_step_kernel(float* x, Addends a, const float* __restrict__ w, float eps, const float* __restrict__ cw,
+                                            int taps, T* conv_state, const int* __restrict__ slots, const int* __restrict__ start_pos,
+                                            T* __restrict__ h_out, int H, int kind) {
+    extern __shared__ float row[];
+    __shared__ float red[32];
+    const size_t base = (size_t)blockIdx.x * H;
+    T* st = conv_state + (size_t)slots[blockIdx.x] * H * (taps - 1);
+    const bool fresh = start_pos[blockIdx.x] <= 0;
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        float v = x[base + c];
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+            if (i < a.n) v += a.s[i] * to_f32(((const T*)a.y[i])[base + c]);
+        row[c] = v;
+        if (a.n > 0) x[base + c] = v;
+    }
+    __syncthreads();
+    float mean, inv;
+    row_stats(row, H, kind, eps, red, mean, inv);
+    for (int c = threadIdx.x; c < H; c += blockDim.x) {
+        const T u = from_f32<T>((row[c] - mean) * inv * (w != nullptr ? w[c] : 1.f));
+        const float* cwr = cw + (size_t)c * taps;
+        T* sc = st + (size_t)c * (taps - 1);
+        float acc = 0.f;
+        for (int j = 0; j + 1 < taps; ++j) {
+            const T old = fresh ? from_f32<T>(0.f) : sc[j];
+            acc += to_f32(old) * cwr[j];
+            if (j > 0) sc[j - 1] = old;
+        }
+        acc += to_f32(u) * cwr[taps - 1];
+        if (taps > 1) sc[taps - 2] = u;
+        h_out[base + c] = from_f32<T>(acc);
+    }
+}
+
+extern "C" int lb_stream_add_conv_step(float* x, const void* y0, const void* y1, const void* y2, const void* y3, float s0, float s1,
+                                       float s2, float s3, int n, const float* w, float eps, const float* cw, int taps, void* conv_state,
+                                       const int* slots, const int* start_pos, void* h_out, int rows, int H, int kind, int dtype,
+                                       void* stream) {
+    if (rows <= 0) return kOk;
+    if (H <= 0 || (size_t)H * sizeof(float) > 160 * 1024 || kind < kLayerNorm || kind > kNoNorm || n < 0 || n > 4 || taps < 1) return kBadSize;
+    const int threads = H >= 2048 ? 1024 : (H >= 512 ? 512 : 128);
+    const size_t smem = (size_t)H * sizeof(float);
+    const Addends a = {{y0, y1, y2, y3}, {s0, s1, s2, s3}, n};
+    LB_DISPATCH_DTYPE(dtype, {
+        static size_t have = 0;
+        ensure_dynamic_smem(stream_add_conv_step_kernel<T>, smem, have);
+        stream_add_conv_step_kernel<T><<<rows, threads, smem, (cudaStream_t)stream>>>(x, a, w, eps, cw, taps, (T*)conv_state, slots,
+                                                                                      start_pos, (T*)h_out, H, kind);
     });
     return launch_status();
 }

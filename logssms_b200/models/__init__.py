@@ -49,4 +49,8 @@ from ..config.zarisun import ARCHITECTURE as _ZARISUN, ZarisunConfig  # noqa: E4
 
 register_architecture(_ZARISUN, ZarisunConfig)
 
+from ..config.dimudra import ARCHITECTURE as _DIMUDRA, DimudraConfig  # noqa: E402
+
+register_architecture(_DIMUDRA, DimudraConfig)
+
 __all__ = ["Architecture", "DecoderModel", "build_model", "register_architecture"]

@@ -29,11 +29,13 @@ class DecoderModel(Part):
         # parts that several layers share and whose tensors are stored at the model's root (a second embedding table that
         # every layer reads a slice of): a layer puts them into `shared["model_parts"]` under their checkpoint prefix
         self.model_parts = dict(shared.get("model_parts", {}))
-        # products over the stream and the embedding's output that open a run of layers (`ScheduleEntry.opens`)
-        from ..parts.block import StreamInput
-        self.stream_inputs = [StreamInput(s, perturb_init) for s in getattr(spec, "stream_inputs", ())]
+        # what mixes the embedding's output into the stream again as a run of layers opens (`ScheduleEntry.opens`): a product
+        # over both, or their sum
+        from ..parts.block import STREAM_INPUTS
+        self.stream_inputs = [STREAM_INPUTS[s.kind](s, perturb_init) for s in getattr(spec, "stream_inputs", ())]
         for s, part in zip(getattr(spec, "stream_inputs", ()), self.stream_inputs):
-            self.model_parts[s.name] = part
+            if part.param_specs():
+                self.model_parts[s.name] = part
         self.schedule = spec.resolved_schedule()
         for e in self.schedule:
             if not 0 <= e.layer < len(self.layers):
@@ -109,7 +111,9 @@ class DecoderModel(Part):
             else:
                 x = self.embedding.forward(ctx.token_ids)
         residual = None
-        x0 = x.act if (self.stream_inputs and isinstance(x, K.StreamRows)) else None     # the embedding's output, kept for them
+        x0 = x.act if (self.stream_inputs and isinstance(x, K.StreamRows)) else None     # the embedding's rows, kept for them
+        x0_scale = getattr(self.embedding, "stream_scale", 1.0)                          # ... and what they are multiplied by
+        joined = False                             # the block before has added the embedding's output already
         tap = ctx.extras.get("layer_tap")          # debugging: called with (run index, the stream after that layer run)
         for i, e in enumerate(self.schedule):
             # a block may hand its output on already joined with the residual (`SummedRows`) where the norm that
@@ -123,11 +127,19 @@ class DecoderModel(Part):
                                                            "takes_scaled_rows", False)
             # ... or, on a 32-bit stream, already normed by that norm (the kernel that closes the block does it on the way)
             ctx.extras["next_input_norm"] = getattr(nxt, "input_norm", None)
-            # (not where a product over the stream comes between this block and the next)
-            ctx.extras["next_opens"] = i + 1 < len(self.schedule) and self.schedule[i + 1].opens is not None
-            if e.opens is not None:
+            # ... and, in a decode step, convolved by that block's input convolution
+            conv = getattr(nxt, "input_conv", None)
+            ctx.extras["next_input_conv"] = None if conv is None else (conv, self.schedule[i + 1].cache)
+            # (not where a product over the stream comes between this block and the next; a mere sum may join in the kernel
+            # that closes this block, except where a tap wants the stream as it is before)
+            if e.opens is not None and not joined:
                 with nvtx_range("stream input"):
-                    x = self.stream_inputs[e.opens].forward(x, x0)
+                    x = self.stream_inputs[e.opens].forward(x, x0, x0_scale)
+            opens = self.schedule[i + 1].opens if i + 1 < len(self.schedule) else None
+            joined = (opens is not None and getattr(self.stream_inputs[opens], "is_addend", False) and tap is None
+                      and getattr(self.layers[e.layer], "joins_opening", False))
+            ctx.extras["next_opens"] = opens is not None and not joined
+            ctx.extras["next_addend"] = (x0, x0_scale) if joined else None
             if PROFILER.nvtx:                      # named ranges per layer (and per part inside it) for a timeline
                 with nvtx_range(f"layer {e.layer}"):
                     x, residual = self.layers[e.layer].forward(x, residual, ctx, e.cache, e.writes_cache)
@@ -138,7 +150,8 @@ class DecoderModel(Part):
         ctx.extras.pop("next_norm_takes_summed", None)
         ctx.extras.pop("next_norm_takes_scaled", None)
         ctx.extras.pop("next_input_norm", None)
-        ctx.extras.pop("next_opens", None)
+        for key in ("next_opens", "next_input_conv", "next_addend"):
+            ctx.extras.pop(key, None)
         return x, residual
 
     def logits(self, x: torch.Tensor, residual, rows: torch.Tensor) -> torch.Tensor:

@@ -121,12 +121,13 @@ class StreamRows:
     """A residual stream that is kept in 32-bit whatever the activation dtype: `f32` [rows, width] is the stream, `act`
     its copy rounded to the activation dtype, which the next sublayer's products read (in a float32 engine both are one
     tensor).  Post-norm blocks hand these from layer to layer; a norm with `takes_stream_rows = True` normalises them."""
-    __slots__ = ("f32", "act", "normed_by")
+    __slots__ = ("f32", "act", "normed_by", "convolved")
 
-    def __init__(self, f32, act, normed_by=None):
+    def __init__(self, f32, act, normed_by=None, convolved=False):
         # `normed_by`: on a pre-norm stream `act` may already be the output of the norm that reads the stream next
-        # (the kernel that closed the layer before made it on the way); it then names that norm
-        self.f32, self.act, self.normed_by = f32, act, normed_by
+        # (the kernel that closed the layer before made it on the way); it then names that norm.  `convolved`: `act` has
+        # also passed the input convolution of the block that reads it next
+        self.f32, self.act, self.normed_by, self.convolved = f32, act, normed_by, convolved
 
     @property
     def shape(self):

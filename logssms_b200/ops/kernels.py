@@ -1094,20 +1094,33 @@ def _gla_decay_checks(z, head_decay, T: int, H: int, dk: int) -> None:
               "a fixed decay per head is float32 [H] and comes without z")
 
 
+def _gla_gate_checks(lower, z_bias, z, head_decay, q_scale: float, H: int, dk: int) -> None:
+    if lower is None:
+        _need(z_bias is None, "a bias of the gate comes with its lower bound")
+        return
+    _need(z is not None and head_decay is None and q_scale == 1.0, "a gate with a lower bound comes from z, without another scale")
+    for t, name in ((lower, "lower"), (z_bias, "z_bias")):
+        _need(t is None or (t.is_cuda and t.dtype == torch.float32 and t.shape == (H * dk,) and t.is_contiguous()), f"{name} must be float32 [H*key_dim]")
+
+
 def gla_scan(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor,
              slots: torch.Tensor, num_requests: int, num_heads: int, key_dim: int, value_dim: int, tau: float,
              q_scale: float, request_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
-             head_decay: torch.Tensor | None = None) -> torch.Tensor:
+             head_decay: torch.Tensor | None = None, lower: torch.Tensor | None = None,
+             z_bias: torch.Tensor | None = None) -> torch.Tensor:
     """Token-by-token recurrence S <- diag(sigmoid(z)^(1/tau)) S + k v^T, o = S^T (q * q_scale) per head over every
     request's tokens.  qkv: [tokens, >= 2*H*key_dim + H*value_dim] with columns q | k | v first (unit column stride);
     z: float32 [tokens, H*key_dim]; state: float32 [slots, H, key_dim, value_dim], updated in place.  Returns float32
     [tokens, H*value_dim].  With `head_decay` (float32 [H]) every key channel of head h decays by head_decay[h] at every
-    token, and z (then None) is not read."""
-    _cuda(qkv, z, state, cu_seqlens, start_pos, slots, request_list, head_decay)
+    token, and z (then None) is not read.  With `lower` (float32 [H*key_dim]; `z_bias` float32 [H*key_dim] is added to z) the
+    decay is a = lower + (1 - lower) sigmoid(z), the key is 1 - a, q passes silu first, and qkv holds the columns q | v."""
+    _cuda(qkv, z, state, cu_seqlens, start_pos, slots, request_list, head_decay, lower, z_bias)
     H, dk, dv = num_heads, key_dim, value_dim
     T = qkv.shape[0]
-    _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= H * (2 * dk + dv), "qkv must hold the columns q | k | v")
+    keys = 0 if lower is not None else H * dk            # columns of k
+    _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= H * (dk + dv) + keys, "qkv must hold the columns q | k | v")
     _gla_decay_checks(z, head_decay, T, H, dk)
+    _gla_gate_checks(lower, z_bias, z, head_decay, q_scale, H, dk)
     _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dk, dv),
           "the state must be contiguous float32 [slots, H, key_dim, value_dim]")
     for t, name in ((cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (slots, "slots")):
@@ -1120,9 +1133,11 @@ def gla_scan(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seqlens
     item, base = qkv.element_size(), qkv.data_ptr()
     stride = qkv.stride(0) if T > 1 else qkv.shape[1]
     f = _fn("gla", "lb_gla_scan", [c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_int, c_void_p])
-    _check(f(base, base + H * dk * item, base + 2 * H * dk * item, stride, _ptr(z), _ptr(o), _ptr(state), _ptr(cu_seqlens),
-             _ptr(start_pos), _ptr(slots), _ptr(request_list), n, H, dk, dv, tau, q_scale, _ptr(head_decay), _code(qkv), _stream()),
+                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int,
+                                   c_void_p])
+    _check(f(base, base + H * dk * item, base + (H * dk + keys) * item, stride, _ptr(z), _ptr(o), _ptr(state), _ptr(cu_seqlens),
+             _ptr(start_pos), _ptr(slots), _ptr(request_list), n, H, dk, dv, tau, q_scale, _ptr(head_decay), _ptr(lower), _ptr(z_bias),
+             _code(qkv), _stream()),
            "gla_scan", f"(key_dim {dk}, value_dim {dv})")
     return o
 
@@ -1141,25 +1156,30 @@ def gla_chunked(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seql
                 slots: torch.Tensor, chunks: torch.Tensor, num_chunks: int, per_request: torch.Tensor, num_long: int,
                 num_heads: int, key_dim: int, value_dim: int, tau: float, q_scale: float, out: torch.Tensor,
                 segments: torch.Tensor | None = None, segment_requests: torch.Tensor | None = None,
-                head_decay: torch.Tensor | None = None) -> torch.Tensor:
+                head_decay: torch.Tensor | None = None, lower: torch.Tensor | None = None,
+                z_bias: torch.Tensor | None = None) -> torch.Tensor:
     """The recurrence of `gla_scan` over the long portions of a step in chunks of `GLA_CHUNK` tokens on the tensor cores
     (see `csrc/gla.cu`); the rows of the other requests in `out` (float32 [tokens, H*value_dim]) are left alone.
     `chunks`, `per_request`: the work lists of `StepContext.long_portion_chunks(GLA_CHUNK)`.  With `segments` and
     `segment_requests` (`StepContext.long_portion_segments`) every request's segments run side by side, twice, with a
-    pass over their states between: for steps whose few long portions would leave most of the GPU idle."""
-    _cuda(qkv, z, state, cu_seqlens, start_pos, slots, chunks, per_request, out, head_decay)
+    pass over their states between: for steps whose few long portions would leave most of the GPU idle.  `lower`, `z_bias`:
+    as for `gla_scan`; the products' operands are then handed to the tensor cores as two bfloat16 terms each."""
+    _cuda(qkv, z, state, cu_seqlens, start_pos, slots, chunks, per_request, out, head_decay, lower, z_bias)
     H, dk, dv = num_heads, key_dim, value_dim
     T = qkv.shape[0]
     _need(gla_chunked_ok(qkv, dk), "gla_chunked takes bfloat16 operands with key channels a multiple of 16 up to 256")
-    _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= H * (2 * dk + dv), "qkv must hold the columns q | k | v")
+    keys = 0 if lower is not None else H * dk            # columns of k
+    _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] >= H * (dk + dv) + keys, "qkv must hold the columns q | k | v")
     _gla_decay_checks(z, head_decay, T, H, dk)
+    _gla_gate_checks(lower, z_bias, z, head_decay, q_scale, H, dk)
     _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (H, dk, dv),
           "the state must be contiguous float32 [slots, H, key_dim, value_dim]")
     _need(out.dtype == torch.float32 and out.shape == (T, H * dv) and out.is_contiguous(), "out must be contiguous float32 [tokens, H*value_dim]")
     for t, name in ((cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (slots, "slots"), (chunks, "chunks"), (per_request, "per_request")):
         _i32(t, name)
-    q_in = torch.empty((T, H, dk), dtype=torch.bfloat16, device=qkv.device)
-    k_end = torch.empty((T, H, dk), dtype=torch.bfloat16, device=qkv.device)
+    planes = 1 if lower is None else 2
+    q_in = torch.empty((planes, T, H, dk), dtype=torch.bfloat16, device=qkv.device)
+    k_end = torch.empty((planes, T, H, dk), dtype=torch.bfloat16, device=qkv.device)
     A = torch.empty((T, H, GLA_CHUNK), dtype=torch.float32, device=qkv.device)
     D = torch.empty((max(num_chunks, 1), H, dk), dtype=torch.float32, device=qkv.device)
     seg_state = seg_decay = None
@@ -1175,11 +1195,11 @@ def gla_chunked(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seql
     item, base = qkv.element_size(), qkv.data_ptr()
     f = _fn("gla", "lb_gla_chunked", [c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                      c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p])
-    _check(f(base, base + H * dk * item, base + 2 * H * dk * item, qkv.stride(0) if T > 1 else qkv.shape[1], _ptr(z), _ptr(out),
+                                      c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+    _check(f(base, base + H * dk * item, base + (H * dk + keys) * item, qkv.stride(0) if T > 1 else qkv.shape[1], _ptr(z), _ptr(out),
              _ptr(state), _ptr(cu_seqlens), _ptr(start_pos), _ptr(slots), _ptr(chunks), num_chunks, _ptr(per_request), num_long,
              _ptr(q_in), _ptr(k_end), _ptr(A), _ptr(D), H, dk, dv, tau, q_scale, _ptr(segments), n_seg, _ptr(seg_state),
-             _ptr(seg_decay), _ptr(head_decay), _stream()), "gla_chunked", f"(key_dim {dk}, value_dim {dv})", launches=2 if segments is None else 4)
+             _ptr(seg_decay), _ptr(head_decay), _ptr(lower), _ptr(z_bias), T, _stream()), "gla_chunked", f"(key_dim {dk}, value_dim {dv})", launches=2 if segments is None else 4)
     return out
 
 
@@ -1192,21 +1212,23 @@ def gla_segmented_pays(num_tokens: int, num_long: int, num_heads: int, value_dim
     return num_tokens >= 2 * GLA_SEGMENT * GLA_CHUNK and num_long * num_heads * -(-value_dim // 32) < _SM_COUNT
 
 
-def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, eps: float, num_heads: int,
-                  sigmoid_gate: bool = False) -> torch.Tensor:
+def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tensor, eps: float, num_heads: int,
+                  sigmoid_gate: bool = False, out_dtype: torch.dtype | None = None) -> torch.Tensor:
     """RMSNorm of every head's float32 output with one weight [value_dim] for all heads, times silu(gate) (or, with
     `sigmoid_gate`, sigmoid(gate)); the result has the gate's dtype.  `gate` may be a column view of a wider matrix.  With
-    `num_heads` 1 it is the gated norm over the whole row."""
+    `num_heads` 1 it is the gated norm over the whole row.  `gate` None: the norm alone, in `out_dtype`."""
     _cuda(o, gate, weight)
     rows, width = o.shape
     dv = width // num_heads
     _need(o.dtype == torch.float32 and o.is_contiguous() and width == num_heads * dv, "o must be contiguous float32 [rows, H*value_dim]")
-    _need(gate.shape == o.shape and gate.stride(1) == 1, "gate must match o, unit column stride")
+    _need(gate is not None or out_dtype is not None, "without a gate the result's dtype must be given")
+    _need(gate is None or (gate.shape == o.shape and gate.stride(1) == 1), "gate must match o, unit column stride")
     _need(weight.dtype == torch.float32 and weight.shape == (dv,) and weight.is_contiguous(), "weight must be float32 [value_dim]")
-    out = torch.empty((rows, width), dtype=gate.dtype, device=o.device)
+    out = torch.empty((rows, width), dtype=out_dtype if gate is None else gate.dtype, device=o.device)
     f = _fn("gla", "lb_gla_norm_gate", [c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p])
-    _check(f(_ptr(o), _ptr(gate), gate.stride(0) if rows > 1 else gate.shape[1], _ptr(weight), _ptr(out), rows, num_heads, dv,
-             eps, int(sigmoid_gate), _code(gate), _stream()), "gla_norm_gate")
+    stride = 0 if gate is None else (gate.stride(0) if rows > 1 else gate.shape[1])
+    _check(f(_ptr(o), _ptr(gate), stride, _ptr(weight), _ptr(out), rows, num_heads, dv, eps, int(sigmoid_gate), _code(out), _stream()),
+           "gla_norm_gate")
     return out
 
 
@@ -1391,27 +1413,32 @@ def latent_attention_wide(qa: torch.Tensor, q_rot: torch.Tensor, c_cache: torch.
 
 # --------------------------------------------------------------------------- routed feed-forward
 def moe_route(h: torch.Tensor, w_router: torch.Tensor, correction: torch.Tensor | None, num_experts: int, top: int, groups: int,
-              keep: int, scale: float, sigmoid_scores: bool = False, bias: torch.Tensor | None = None, chosen_softmax: bool = False):
+              keep: int, scale: float, sigmoid_scores: bool = False, bias: torch.Tensor | None = None, chosen_softmax: bool = False,
+              pair_groups: bool = False, normalize: bool = False, gates: int = 0):
     """(dense weights float32 [T, n], chosen int32 [T, top], their weights float32 [T, top], identity weight float32 [T]):
     see `csrc/moe.cu`.  `w_router` float32 [n, width]; outputs num_experts .. n-1 are identity experts.  Scores are the
     softmax over all outputs, or with `sigmoid_scores` the sigmoid of each; `correction` (may be None) moves the choice only.
     With `chosen_softmax` the logits themselves are ranked and the weights are the softmax over the chosen logits alone.
-    `bias` (float32 [n], may be None) is added to the logits."""
+    `bias` (float32 [n], may be None) is added to the logits.  `pair_groups`: a group's score is the sum of its two largest
+    choice scores (else its largest).  `normalize`: the chosen weights are divided by their sum + 1e-20.  The last `gates` rows
+    of `w_router` are no router outputs: the dense weights get `gates` further columns, the sigmoids of their products."""
     _cuda(h, w_router, correction, bias)
-    _need(bias is None or (bias.dtype == torch.float32 and bias.shape == (w_router.shape[0],) and bias.is_contiguous()), "router bias float32 [n]")
+    _need(bias is None or (bias.dtype == torch.float32 and bias.shape == (w_router.shape[0] - gates,) and bias.is_contiguous()), "router bias float32 [n]")
+    _need(not (chosen_softmax and normalize), "the softmax over the chosen logits is normalized already")
     _need(not (chosen_softmax and (sigmoid_scores or correction is not None)), "the softmax over the chosen logits takes no other score")
     T, width = h.shape
-    n = w_router.shape[0]
+    n = w_router.shape[0] - gates
     _need(h.is_contiguous() and w_router.dtype == torch.float32 and w_router.is_contiguous() and w_router.shape[1] == width
           and (correction is None or (correction.dtype == torch.float32 and correction.shape == (n,))),
           "router weight float32 [n, width], correction float32 [n]")
-    dense = torch.empty((T, n), dtype=torch.float32, device=h.device)
+    dense = torch.empty((T, n + gates), dtype=torch.float32, device=h.device)
     chosen = torch.empty((T, top), dtype=torch.int32, device=h.device)
     chosen_w = torch.empty((T, top), dtype=torch.float32, device=h.device)
     idw = torch.empty((T,), dtype=torch.float32, device=h.device)
-    f = _fn("moe", "lb_moe_route", [c_void_p] * 7 + [c_int] * 7 + [c_float, c_int, c_void_p, c_int, c_void_p])
+    f = _fn("moe", "lb_moe_route", [c_void_p] * 7 + [c_int] * 7 + [c_float, c_int, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(h), _ptr(w_router), _ptr(correction), _ptr(dense), _ptr(chosen), _ptr(chosen_w), _ptr(idw), T, width, n,
-             num_experts, top, groups, keep, scale, 2 if chosen_softmax else int(sigmoid_scores), _ptr(bias), _code(h), _stream()), "moe_route",
+             num_experts, top, groups, keep, scale, 2 if chosen_softmax else int(sigmoid_scores), _ptr(bias), int(pair_groups),
+             int(normalize), gates, _code(h), _stream()), "moe_route",
            f"({n} outputs, top {top}, {groups} groups)")
     return dense, chosen, chosen_w, idw
 
@@ -1430,13 +1457,13 @@ def moe_activation(gate_up: torch.Tensor, dense: torch.Tensor | None, num_expert
     T = gate_up.shape[0]
     ff = gate_up.shape[1] // (2 * num_experts)
     _need(gate_up.dim() == 2 and gate_up.stride(1) == 1 and gate_up.shape[1] == 2 * num_experts * ff, "gate_up must be [T, experts*2*ff], unit column stride")
-    _need(dense is None or (dense.dtype == torch.float32 and dense.is_contiguous() and dense.shape[0] == T and dense.shape[1] >= num_experts),
-          "dense weights float32 [T, n]")
+    _need(dense is None or (dense.dtype == torch.float32 and dense.stride(1) == 1 and dense.shape[0] == T and dense.shape[1] >= num_experts),
+          "dense weights float32 [T, n] (a column view is fine)")
     y = out if out is not None else torch.empty((T, num_experts * ff), dtype=gate_up.dtype, device=gate_up.device)
     _need(y.shape == (T, num_experts * ff) and y.dtype == gate_up.dtype and y.stride(1) == 1, "out must be [T, experts*ff] of gate_up's dtype")
     f = _fn("moe", "lb_moe_activation", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_long, c_long,
                                          c_int, c_void_p])
-    _check(f(_ptr(gate_up), _ptr(dense), _ptr(y), T, num_experts, ff, 0 if dense is None else dense.shape[1], limit, act_alpha,
+    _check(f(_ptr(gate_up), _ptr(dense), _ptr(y), T, num_experts, ff, 0 if dense is None else max(dense.stride(0), dense.shape[1]), limit, act_alpha,
              EXPERT_MODES[mode], gate_up.stride(0) if T > 1 else max(gate_up.stride(0), gate_up.shape[1]),
              y.stride(0) if T > 1 else max(y.stride(0), y.shape[1]), _code(gate_up), _stream()), "moe_activation")
     return y
@@ -1688,6 +1715,37 @@ def rownorm_prepare(qk: torch.Tensor, num_heads: int, num_kv_heads: int, head_di
     return q
 
 
+QK_NORMS = {"none": 0, "row": 1, "head": 2}
+
+
+def qk_prepare(qkv: torch.Tensor, num_heads: int, num_kv_heads: int, head_dim: int, value_dim: int, positions: torch.Tensor,
+               slot_mapping: torch.Tensor, table: torch.Tensor, norm: str, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
+               eps: float, k_cache: torch.Tensor, v_cache: torch.Tensor, write_kv: bool = True) -> torch.Tensor:
+    """Queries [tokens, heads, head_dim] from qkv = [tokens, q | k | v] (further columns may follow in the same rows): q and k
+    normed by the root mean square of their whole row ("row"; weights float32 per column of the row), of every head ("head";
+    weights float32 [head_dim]) or not at all ("none"), weights may be None; then rotated in halves over every head's first
+    `table.shape[1]` columns (table: float32 [positions, n], cos | sin of n/2 pairs, column i with column i + n/2; n = 0: no
+    rotation).  Keys and values go to the caches at the tokens' slots.  Norms and rotation are 32-bit."""
+    _cuda(qkv, positions, slot_mapping, table, q_weight, k_weight, k_cache, v_cache)
+    _i32(positions, "positions"); _i32(slot_mapping, "slot_mapping")
+    T = qkv.shape[0]
+    nq, nk, nv = num_heads * head_dim, num_kv_heads * head_dim, num_kv_heads * value_dim
+    _need(qkv.dim() == 2 and qkv.stride(1) == 1 and qkv.shape[1] == nq + nk + nv, "qkv must be [tokens, q | k | v] with unit column stride")
+    _need(k_cache.dtype == v_cache.dtype == qkv.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+          and k_cache.shape[2:] == (num_kv_heads, head_dim) and v_cache.shape[2:] == (num_kv_heads, value_dim), "caches must be [pages, page, kv_heads, dim]")
+    for w, n in ((q_weight, nq), (k_weight, nk)):
+        n = head_dim if norm == "head" else n
+        _need(w is None or (norm != "none" and w.dtype == torch.float32 and w.shape == (n,) and w.is_contiguous()), f"norm weights must be float32 [{n}]")
+    _need(table.dtype == torch.float32 and table.dim() == 2 and table.is_contiguous(), "the rotation table must be contiguous float32")
+    q = torch.empty((T, num_heads, head_dim), dtype=qkv.dtype, device=qkv.device)
+    f = _fn("attention_pooled", "lb_qk_prepare", [c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_int, c_int, c_void_p, c_void_p, c_int,
+                                                  c_float, c_void_p, c_void_p, c_void_p] + [c_int] * 7 + [c_void_p])
+    _check(f(_ptr(qkv), qkv.stride(0) if T > 1 else max(qkv.stride(0), qkv.shape[1]), _ptr(positions), _ptr(slot_mapping), _ptr(table),
+             table.shape[1], max(table.shape[0], 1), _ptr(q_weight), _ptr(k_weight), QK_NORMS[norm], eps, _ptr(q), _ptr(k_cache),
+             _ptr(v_cache), T, num_heads, num_kv_heads, head_dim, value_dim, int(write_kv), _code(qkv), _stream()), "qk_prepare")
+    return q
+
+
 def head_gate(o: torch.Tensor, gate: torch.Tensor, num_heads: int) -> torch.Tensor:
     """o [tokens, heads * width] (contiguous) times sigmoid(gate[t, h]) per token and head, in place.  gate: [tokens, heads]
     logits in float32 or o's dtype (a column view is fine)."""
@@ -1727,41 +1785,49 @@ def _rows(t: torch.Tensor | None) -> int:
     return 1 if t is None else max(t.shape[0], 1)
 
 
-def _score_extras(num_heads: int, pool: int, pooled_table, slopes, sinks) -> None:
+def _score_extras(num_heads: int, pool: int, pooled_table, slopes, sinks, gate=None, like=None) -> None:
     """Checks of the options that the pooled-attention kernels share.  `slopes[h] * (i - j)` is taken off the scaled score of
-    query i (head h) and token j; `exp(sinks[h])` joins the softmax's denominator with no key and no value."""
+    query i (head h) and token j; `exp(sinks[h])` joins the softmax's denominator with no key and no value; `gate` (logits of
+    `like`'s shape and dtype, a column view is fine): every output column is multiplied by sigmoid of its logit."""
     _need(pool >= 0 and (pool == 0 or pooled_table is not None), "pooled blocks need their caches and table (pool 0: none)")
     for t, name in ((slopes, "slopes"), (sinks, "sinks")):
         _need(t is None or (t.is_cuda and t.dtype == torch.float32 and t.shape == (num_heads,) and t.is_contiguous()),
               f"{name} must be float32 [heads] on the device")
+    _need(gate is None or (gate.is_cuda and gate.shape == like.shape and gate.dtype == like.dtype and gate.stride(1) == 1),
+          "gate logits must match the output, unit column stride")
+
+
+def _gate_stride(gate) -> int:
+    return 0 if gate is None else max(gate.stride(0), gate.shape[1])
 
 
 def pooled_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, kp_cache: torch.Tensor, vp_cache: torch.Tensor,
                      block_table: torch.Tensor, pooled_table: torch.Tensor, token_req: torch.Tensor, positions: torch.Tensor,
                      v_table: torch.Tensor, scale: float, window: int, pool: int, token_list: torch.Tensor | None = None,
-                     out: torch.Tensor | None = None, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> torch.Tensor:
+                     out: torch.Tensor | None = None, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                     gate: torch.Tensor | None = None) -> torch.Tensor:
     """[tokens, heads * value_dim]: attention of every (listed) token over its window's tokens and the pooled blocks
     behind it, a warp per (token, head), everything in float32; the summed values are turned back by the query's position.
     `pool` 0: no blocks (the pooled caches and their table may be None); `v_table` None: values are not rotated; `slopes`,
-    `sinks` (float32 per query head, may be None): see `_score_extras`."""
+    `sinks` (float32 per query head, may be None), `gate`: see `_score_extras`."""
     _cuda(q, k_cache, v_cache, kp_cache, vp_cache, block_table, pooled_table, token_req, positions, v_table, token_list)
     for t, name in ((block_table, "block_table"), (pooled_table, "pooled_table"), (token_req, "token_req"), (positions, "positions")):
         if t is not None:
             _i32(t, name)
     T, H, dim = q.shape
-    _score_extras(H, pool, pooled_table, slopes, sinks)
     G, vdim = v_cache.shape[2], v_cache.shape[3]
     _need(q.is_contiguous() and q.dtype == k_cache.dtype, "queries must be contiguous [tokens, heads, dim] in the cache's dtype")
     if out is None:
         out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
+    _score_extras(H, pool, pooled_table, slopes, sinks, gate, out)
     n = T if token_list is None else token_list.numel()
     f = _fn("attention_pooled", "lb_pooled_attention", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                         c_void_p, c_int, c_int, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p])
+            + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(token_req), _ptr(positions), _ptr(token_list), n, _ptr(v_table),
              _width(v_table), _rows(v_table), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool, _ptr(slopes),
-             _ptr(sinks), _code(q), _stream()), "pooled_attention", f"(dim {dim}, value dim {vdim})")
+             _ptr(sinks), _ptr(gate), _gate_stride(gate), _code(q), _stream()), "pooled_attention", f"(dim {dim}, value dim {vdim})")
     return out
 
 
@@ -1794,7 +1860,7 @@ def pooled_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
                           block_table: torch.Tensor, pooled_table: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor,
                           positions: torch.Tensor, tiles: torch.Tensor, v_table: torch.Tensor, scale: float, window: int, pool: int,
                           out: torch.Tensor, splits: int = 1, slopes: torch.Tensor | None = None,
-                          sinks: torch.Tensor | None = None) -> torch.Tensor:
+                          sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """The same attention for the long portions' runs of `pooled_attention_tile_q()` tokens (work list of
     `StepContext.long_portion_tiles`) on the tensor cores; writes those tokens' rows of `out` [tokens, heads * value_dim].
     With `splits` > 1 that many CTAs share a run's keys and a merge follows, which also writes the rows that no run covers
@@ -1805,18 +1871,18 @@ def pooled_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
         if t is not None:
             _i32(t, name)
     T, H, dim = q.shape
-    _score_extras(H, pool, pooled_table, slopes, sinks)
+    _score_extras(H, pool, pooled_table, slopes, sinks, gate, out)
     G, vdim = v_cache.shape[2], v_cache.shape[3]
     _need(q.is_contiguous() and q.dtype == torch.bfloat16 and k_cache.dtype == torch.bfloat16 and out.dtype == torch.bfloat16
           and out.is_contiguous() and out.shape == (T, H * vdim), "the tensor-core form takes contiguous bfloat16 tensors")
     partial = torch.empty((T, H, splits, vdim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
     f = _fn("attention_pooled", "lb_pooled_attention_tile", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                              c_void_p, c_int, c_void_p, c_int, c_int, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p])
+            + [c_float, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(cu_seqlens), _ptr(start_pos), _ptr(tiles), tiles.shape[0], _ptr(positions), T,
              _ptr(v_table), _width(v_table), _rows(v_table), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool,
-             _ptr(partial), splits, _ptr(slopes), _ptr(sinks), _stream()),
+             _ptr(partial), splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), _stream()),
            "pooled_attention_tile", f"(dim {dim}, value dim {vdim})", launches=2 if splits > 1 else 1)
     return out
 
@@ -1835,7 +1901,8 @@ def pooled_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
                            block_table: torch.Tensor, pooled_table: torch.Tensor, token_req: torch.Tensor, positions: torch.Tensor,
                            v_table: torch.Tensor, scale: float, window: int, pool: int, splits: int,
                            token_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
-                           slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None) -> torch.Tensor:
+                           slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
+                           gate: torch.Tensor | None = None) -> torch.Tensor:
     """The attention of `pooled_attention` with every token's keys cut into `splits` ranges that run side by side and all
     query heads of a key/value head in one CTA; a merge kernel joins the ranges (two launches)."""
     _cuda(q, k_cache, v_cache, kp_cache, vp_cache, block_table, pooled_table, token_req, positions, v_table, token_list)
@@ -1843,20 +1910,100 @@ def pooled_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
         if t is not None:
             _i32(t, name)
     T, H, dim = q.shape
-    _score_extras(H, pool, pooled_table, slopes, sinks)
     G, vdim = v_cache.shape[2], v_cache.shape[3]
     _need(q.is_contiguous() and q.dtype == k_cache.dtype, "queries must be contiguous [tokens, heads, dim] in the cache's dtype")
     if out is None:
         out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
+    _score_extras(H, pool, pooled_table, slopes, sinks, gate, out)
     n = T if token_list is None else token_list.numel()
     partial = torch.empty((n, H, splits, vdim + 2), dtype=torch.float32, device=q.device)
     f = _fn("attention_pooled", "lb_pooled_attention_split", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                               c_void_p, c_int, c_int, c_void_p, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_int, c_void_p])
+            + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(token_req), _ptr(positions), _ptr(token_list), n, _ptr(v_table),
              _width(v_table), _rows(v_table), _ptr(partial), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool,
-             splits, _ptr(slopes), _ptr(sinks), _code(q), _stream()), "pooled_attention_split", f"(dim {dim}, value dim {vdim}, {splits} ranges)", launches=2)
+             splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), _code(q), _stream()), "pooled_attention_split", f"(dim {dim}, value dim {vdim}, {splits} ranges)", launches=2)
+    return out
+
+
+# --------------------------------------------------------------------------- selective scan (a decay per channel and state)
+def _selective_checks(x, low, dt_bias, A_log, D, gate, state, y, rank: int) -> tuple[int, int]:
+    T, inner = x.shape
+    n = A_log.shape[1]
+    _need(x.stride(1) == 1, "x must be rows with unit column stride")
+    _need(low.shape == (T, rank + 2 * n) and low.stride(1) == 1 and low.dtype == x.dtype, "low must be [tokens, rank | state | state] of x's dtype")
+    _need(A_log.dtype == torch.float32 and A_log.shape == (inner, n) and A_log.is_contiguous(), "A_log must be float32 [inner, state]")
+    for t, name in ((dt_bias, "dt_bias"), (D, "D")):
+        _need(t.dtype == torch.float32 and t.shape == (inner,) and t.is_contiguous(), f"{name} must be float32 [inner]")
+    _need(gate.shape == (T, inner) and gate.stride(1) == 1 and gate.dtype == x.dtype, "gate must be a [tokens, inner] view of x's dtype")
+    _need(state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (inner, n), "the state must be contiguous float32 [slots, inner, state]")
+    _need(y.shape == (T, inner) and y.dtype == x.dtype and y.is_contiguous(), "out must be contiguous [tokens, inner] of x's dtype")
+    return inner, n
+
+
+def _row_stride(t: torch.Tensor) -> int:
+    return t.stride(0) if t.shape[0] > 1 else max(t.stride(0), t.shape[1])
+
+
+def selective_scan(x: torch.Tensor, w: torch.Tensor | None, low: torch.Tensor, dt_w: torch.Tensor | None, dt_bias: torch.Tensor,
+                   A_log: torch.Tensor, D: torch.Tensor, gate: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor,
+                   start_pos: torch.Tensor, slots: torch.Tensor, num_requests: int, rank: int, *,
+                   request_list: torch.Tensor | None = None, out: torch.Tensor | None = None) -> torch.Tensor:
+    """dt = softplus(w + dt_bias); S <- exp(-dt exp(A_log)) S + dt x B, y = (S C + D x) silu(gate) per channel (`inner` of
+    them) with `state` values each, token by token over every (listed) request's tokens.  x, gate: [tokens, inner] views; low:
+    [tokens, rank | B | C] view; w: float32 [tokens, inner], or None: it is then made in the kernel from low's first `rank`
+    columns and `dt_w` [inner, rank].  state: float32 [slots, inner, state], updated in place.  Returns y (other requests' rows
+    of `out` are left alone)."""
+    _cuda(x, w, low, dt_w, dt_bias, A_log, D, gate, state, cu_seqlens, start_pos, slots, request_list, out)
+    y = out if out is not None else torch.empty((x.shape[0], x.shape[1]), dtype=x.dtype, device=x.device)
+    inner, n = _selective_checks(x, low, dt_bias, A_log, D, gate, state, y, rank)
+    _need(w is None or (w.dtype == torch.float32 and w.shape == (x.shape[0], inner) and w.is_contiguous()), "w must be contiguous float32 [tokens, inner]")
+    _need(w is not None or (dt_w is not None and dt_w.shape == (inner, rank) and dt_w.dtype == x.dtype and dt_w.is_contiguous()),
+          "without w the step's weights [inner, rank] come in x's dtype")
+    for t, name in ((cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (slots, "slots")):
+        _i32(t, name)
+    requests = num_requests
+    if request_list is not None:
+        _i32(request_list, "request_list")
+        requests = request_list.numel()
+    f = _fn("selective_scan", "lb_selective_scan", [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
+                                                    c_long] + [c_void_p] * 6 + [c_int] * 5 + [c_void_p])
+    _check(f(_ptr(x), _row_stride(x), _ptr(w), _ptr(low), _row_stride(low), _ptr(dt_w), _ptr(dt_bias), _ptr(A_log), _ptr(D), _ptr(gate),
+             _row_stride(gate), _ptr(state), _ptr(y), _ptr(cu_seqlens), _ptr(start_pos), _ptr(slots), _ptr(request_list), requests, inner, n,
+             rank, _code(x), _stream()), "selective_scan", f"(inner {inner}, state {n})")
+    return y
+
+
+SELECTIVE_CHUNK = 64          # tokens; a segment is so many chunks of so many tokens
+SELECTIVE_SEGMENT = 4
+
+
+def selective_segmented_pays(num_tokens: int, num_long: int, inner: int, state: int) -> bool:
+    """Should the long portions run as segments side by side?  When the CTAs of whole portions would leave most of the GPU
+    idle (a channel takes ceil(state / 4) lanes or fewer) and the portions are long enough to be cut."""
+    lanes = 1 << max(0, (min(-(-state // 4), 32) - 1).bit_length())
+    return num_tokens >= 2 * SELECTIVE_SEGMENT * SELECTIVE_CHUNK and num_long * inner * lanes // 32 < 8 * 4 * _SM_COUNT
+
+
+def selective_scan_segments(x: torch.Tensor, w: torch.Tensor, low: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
+                            gate: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor, slots: torch.Tensor,
+                            segments: torch.Tensor, rank: int, out: torch.Tensor) -> torch.Tensor:
+    """The recurrence of `selective_scan` over the long portions of a step with every portion's segments of SELECTIVE_SEGMENT *
+    SELECTIVE_CHUNK tokens side by side (`segments`: `StepContext.long_portion_segments` of those sizes), in two launches."""
+    _cuda(x, w, low, dt_bias, A_log, D, gate, state, cu_seqlens, start_pos, slots, segments, out)
+    inner, n = _selective_checks(x, low, dt_bias, A_log, D, gate, state, out, rank)
+    _need(w.dtype == torch.float32 and w.shape == (x.shape[0], inner) and w.is_contiguous(), "w must be contiguous float32 [tokens, inner]")
+    for t, name in ((cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (slots, "slots"), (segments, "segments")):
+        _i32(t, name)
+    items = segments.shape[0]
+    seg_state = torch.empty((max(items, 1), inner, n), dtype=torch.float32, device=x.device)
+    seg_dt = torch.empty((max(items, 1), inner), dtype=torch.float32, device=x.device)
+    f = _fn("selective_scan", "lb_selective_scan_segments", [c_void_p, c_long, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p,
+                                                             c_long] + [c_void_p] * 6 + [c_int, c_int, c_void_p, c_void_p] + [c_int] * 4 + [c_void_p])
+    _check(f(_ptr(x), _row_stride(x), _ptr(w), _ptr(low), _row_stride(low), _ptr(dt_bias), _ptr(A_log), _ptr(D), _ptr(gate), _row_stride(gate),
+             _ptr(state), _ptr(out), _ptr(cu_seqlens), _ptr(start_pos), _ptr(slots), _ptr(segments), items, SELECTIVE_SEGMENT * SELECTIVE_CHUNK,
+             _ptr(seg_state), _ptr(seg_dt), inner, n, rank, _code(x), _stream()), "selective_scan_segments", f"(inner {inner}, state {n})", launches=2)
     return out
 
 
@@ -2036,6 +2183,36 @@ def stream_add_many(x: torch.Tensor, addends, weight: torch.Tensor | None, eps: 
     _check(f(_ptr(x), *ptrs, *scales, len(ys), _ptr(weight), eps, _ptr(h), rows, H, NORM_KINDS[kind], _DTYPE_CODE[act_dtype], _stream()),
            "stream_add_many", f"(width {H})")
     return x, h
+
+
+def stream_add_conv_step(x: torch.Tensor, addends, weight: torch.Tensor | None, eps: float, kind: str, conv_weight: torch.Tensor,
+                         conv_state: torch.Tensor | None, slots: torch.Tensor, start_pos: torch.Tensor, act_dtype: torch.dtype) -> torch.Tensor:
+    """`stream_add_many` for a decode batch (every row the single new token of its own request) whose normed rows also pass a
+    short causal convolution per channel: `conv_weight` float32 [width, taps] over the request's last taps - 1 normed rows
+    (`conv_state` [slots, width, taps - 1] in `act_dtype`, shifted in place; None with one tap) and this one.  Returns the
+    convolved rows."""
+    rows, H = x.shape
+    ys = [y for y, _ in addends]
+    _cuda(x, weight, conv_weight, conv_state, slots, start_pos, *ys)
+    taps = conv_weight.shape[1]
+    _need(x.dtype == torch.float32 and x.is_contiguous(), "the stream must be contiguous float32")
+    _need(len(addends) <= 4, "at most four addends join the stream in one kernel")
+    for y in ys:
+        _need(y.shape == x.shape and y.dtype == act_dtype and y.is_contiguous(), "an addend must match the stream's shape")
+    _need(weight is None or (weight.dtype == torch.float32 and weight.shape == (H,) and weight.is_contiguous()), "weight must be float32 [width]")
+    _need(conv_weight.dtype == torch.float32 and conv_weight.shape == (H, taps) and conv_weight.is_contiguous(), "conv weight must be float32 [width, taps]")
+    _need((taps == 1 and conv_state is None) or (conv_state is not None and conv_state.dtype == act_dtype and conv_state.is_contiguous()
+                                                 and conv_state.shape[1:] == (H, taps - 1)), "conv state must be [slots, width, taps - 1] of the activation dtype")
+    _i32(slots, "slots"); _i32(start_pos, "start_pos")
+    _need(slots.numel() >= rows and start_pos.numel() >= rows, "one slot and start per row")
+    h = torch.empty((rows, H), dtype=act_dtype, device=x.device)
+    ptrs = [_ptr(y) for y in ys] + [None] * (4 - len(ys))
+    scales = [float(s) for _, s in addends] + [0.0] * (4 - len(ys))
+    f = _fn("stream_layer", "lb_stream_add_conv_step", [c_void_p] * 5 + [c_float] * 4 + [c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
+                                                        c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
+    _check(f(_ptr(x), *ptrs, *scales, len(ys), _ptr(weight), eps, _ptr(conv_weight), taps, _ptr(conv_state), _ptr(slots), _ptr(start_pos),
+             _ptr(h), rows, H, NORM_KINDS[kind], _DTYPE_CODE[act_dtype], _stream()), "stream_add_conv_step", f"(width {H}, {taps} taps)")
+    return h
 
 
 def stream_pair_rows(x: torch.Tensor, x0: torch.Tensor) -> torch.Tensor:

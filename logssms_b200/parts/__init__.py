@@ -15,8 +15,11 @@ from .conv_attention import ConvAttention
 from .lightning import LightningAttention
 from .sink_attention import MixerPair, SinkAttention
 from .moe import GLU
+from .mamba import Mamba
+from .hgrn2 import HGRN2
+from .gated_attention import GatedAttention
 from .embedding import BareLMHead, Embedding, LMHead, NormedEmbedding, PairEmbedding, StreamEmbedding
-from .block import ParallelStreamBlock, PostNormBlock, PreNormParallelBlock, PreNormStreamBlock, StreamInput, TokenSideInput, OutNormStreamBlock
+from .block import ParallelStreamBlock, PostNormBlock, PreNormParallelBlock, PreNormStreamBlock, StreamInput, TokenSideInput, OutNormStreamBlock, InputConv, StreamAdd
 
 __all__ = ["MATRIX", "TABLE", "VECTOR", "ParamSpec", "Part", "Runtime", "StepContext", "RMSNorm",
            "RotaryEmbedding", "inverse_frequencies", "Attention", "Mamba2", "GatedMLP", "Embedding", "LMHead",
@@ -24,4 +27,4 @@ __all__ = ["MATRIX", "TABLE", "VECTOR", "ParamSpec", "Part", "Runtime", "StepCon
            "PairEmbedding", "BareLMHead", "LayerNorm", "MinGRU", "PooledWindowAttention", "ClampedGLU", "NormedEmbedding",
            "PreNormStreamBlock", "TokenSideInput", "ChannelDelta", "LightningAttention", "MixerPair", "SinkAttention", "GLU",
            "StreamEmbedding", "ParallelStreamBlock", "StreamInput", "GatedDelta", "ConvAttention", "OutNormStreamBlock",
-           "RampRotaryEmbedding", "ramp_frequencies"]
+           "RampRotaryEmbedding", "ramp_frequencies", "Mamba", "HGRN2", "GatedAttention", "InputConv", "StreamAdd"]

@@ -324,6 +324,42 @@ class TokenSideInput(Part):
                              s.eps, nw, neps, nkind, act_dtype)
 
 
+class InputConv(Part):
+    """What a block's mixer reads instead of the normed rows h: h + conv(h), conv a causal convolution over time per channel (no
+    bias, zeros before the sequence's start).  The last taps - 1 rows h are per-request state of the block's cache layer.  h
+    itself is one more on the last tap (added when the weight arrives), so it is one convolution: a kernel of its own for prompt
+    portions, part of the kernel that closes the block before in a decode step (`K.stream_add_conv_step`).
+    Tensor: the taps [width, taps], under the part's own name."""
+    kernels = ("conv", "stream_layer")
+    STATE = "input_conv"
+
+    def __init__(self, width: int, taps: int):
+        if not 1 <= taps <= 8:
+            raise ValueError("an input convolution takes 1 .. 8 taps")
+        self.width, self.taps = width, taps
+        self.weight: torch.Tensor | None = None
+
+    def param_specs(self):
+        from .base import VECTOR, ParamSpec, normal_init
+        return {"": ParamSpec((self.width, self.taps), VECTOR, normal_init(0.3))}
+
+    def bind(self, t):
+        self.weight = t[""].clone()
+        self.weight[:, -1] += 1.0
+
+    def state_needs(self) -> tuple:
+        from ..cache import StateNeed
+        return (StateNeed(self.STATE, (self.width, self.taps - 1), None),) if self.taps > 1 else ()
+
+    def state(self, ctx, cache_layer: int):
+        return ctx.cache.states[cache_layer][self.STATE] if self.taps > 1 else None
+
+    def forward(self, h: torch.Tensor, ctx, cache_layer: int) -> torch.Tensor:
+        C = self.width
+        return K.causal_conv1d(h, self.weight, None, self.state(ctx, cache_layer), ctx.cu_seqlens, ctx.start_pos, ctx.slots,
+                               ctx.num_requests, ctx.max_len, (C, C), (1.0, 1.0, 1.0), activation="none")
+
+
 @BLOCKS.register("prenorm_stream")
 class PreNormStreamBlock(Part):
     """Pre-norm block on a 32-bit stream (`K.StreamRows`): x <- x + s1 * mixer(norm1(x)); with a feed-forward
@@ -332,7 +368,12 @@ class PreNormStreamBlock(Part):
 
     Three kernels besides the sublayers' own: the mixer's output joins the stream and norm2 reads it in one
     (`K.stream_add_norm`); the feed-forward's output joins, the side input is added and the NEXT block's first norm
-    reads the result in one (`K.stream_side`); norm1 runs alone only where the block before could not do it."""
+    reads the result in one (`K.stream_side`); norm1 runs alone only where the block before could not do it.
+
+    A mixer of several branches hands back several outputs with a scale each; they join in one kernel (`K.stream_add_many`), in
+    blocks without `layer_scale` and side input.  With `input_conv` the mixer reads h + conv(h) (`InputConv`); in a decode step
+    the kernel that closes the block before makes that too.  Where the embedding's output is added before the next block, it
+    joins in the closing kernel as one more addend."""
 
     def __init__(self, spec, perturb_init: bool = False, shared: dict | None = None):
         self.spec = spec
@@ -350,6 +391,9 @@ class PreNormStreamBlock(Part):
             if norm is not None and not hasattr(norm, "norm_kind"):
                 raise ValueError("prenorm_stream blocks need norms with a form on a 32-bit stream (`norm_kind`)")
         self.side = None if spec.side is None else TokenSideInput(spec.side, perturb_init, shared)
+        self.input_conv = InputConv(spec.mixer_norm.size, spec.input_conv) if getattr(spec, "input_conv", 0) else None
+        self._plain = not spec.layer_scale and spec.side is None        # nothing but sums between the sublayers
+        self.joins_opening = self._plain      # forward() adds `ctx.extras["next_addend"]` to the stream as it closes the block
         self._jitter = 0.3 if perturb_init else 0.0
         self.scale_mixer = self.scale_ff = None
 
@@ -377,10 +421,16 @@ class PreNormStreamBlock(Part):
             kids[s.feed_forward_name] = self.feed_forward
         if self.side is not None:
             kids[s.side_name] = self.side
+        if self.input_conv is not None:
+            kids[s.input_conv_name] = self.input_conv
         return kids
 
     def cache_needs(self):
-        return self.mixer.cache_needs()
+        need = self.mixer.cache_needs()
+        if self.input_conv is None:
+            return need
+        from dataclasses import replace
+        return replace(need, states=need.states + self.input_conv.state_needs())
 
     def setup(self, rt) -> None:
         self.mixer.setup(rt)
@@ -396,17 +446,27 @@ class PreNormStreamBlock(Part):
             h = x.act
         else:
             _, h = K.stream_add_norm(stream, None, None, self.mixer_norm.weight, self.mixer_norm.eps, self.mixer_norm.norm_kind, act)
+        if self.input_conv is not None and not x.convolved:
+            h = self.input_conv.forward(h, ctx, cache_layer)
         with nvtx_range(self.spec.mixer.spec.kind):
             y = self.mixer.forward(h, ctx, cache_layer, writes_cache)
+        if isinstance(y, list) and not self._plain:
+            raise ValueError("a mixer of several branches goes without layer scales and side input")
         scale = self.scale_mixer
         if self.feed_forward is not None:
-            _, h = K.stream_add_norm(stream, y, scale, self.ff_norm.weight, self.ff_norm.eps, self.ff_norm.norm_kind, act)
+            n = self.ff_norm
+            if isinstance(y, list):
+                _, h = K.stream_add_many(stream, y, n.weight, n.eps, n.norm_kind, act)
+            else:
+                _, h = K.stream_add_norm(stream, y, scale, n.weight, n.eps, n.norm_kind, act)
             with nvtx_range(self.spec.feed_forward.kind):
                 y = self.feed_forward.forward(h)
             scale = self.scale_ff
         # what is left to join the stream (y with its scale) joins in the kernel that closes the block
         nxt = ctx.extras.get("next_input_norm")
-        nxt = nxt if hasattr(nxt, "norm_kind") else None
+        nxt = nxt if hasattr(nxt, "norm_kind") and not ctx.extras.get("next_opens") else None
+        if self._plain:
+            return self._close(stream, y, nxt, ctx, act), None
         if self.side is not None:
             _, h = self.side.close(stream, y, scale, ctx.token_ids, nxt, act)
         elif nxt is not None:
@@ -417,6 +477,26 @@ class PreNormStreamBlock(Part):
         if h is None:
             return K.StreamRows(stream, x.act[:0]), None
         return K.StreamRows(stream, h, normed_by=nxt), None
+
+    def _close(self, stream, y, nxt, ctx, act):
+        """x += what is left (each with a scalar), then what the next block reads: its norm, and in a decode step its input
+        convolution."""
+        joins = _addends(y)
+        if ctx.extras.get("next_addend") is not None:
+            joins.append(ctx.extras["next_addend"])
+        while len(joins) > 4:
+            K.stream_add_many(stream, joins[:4], None, 0.0, "rmsnorm", act)
+            joins = joins[4:]
+        if nxt is None:
+            K.stream_add_many(stream, joins, None, 0.0, "rmsnorm", act)
+            return K.StreamRows(stream, stream.new_empty((0, stream.shape[1]), dtype=act))
+        conv, layer = ctx.extras.get("next_input_conv") or (None, None)
+        if conv is not None and ctx.max_len == 1:
+            h = K.stream_add_conv_step(stream, joins, nxt.weight, nxt.eps, nxt.norm_kind, conv.weight, conv.state(ctx, layer), ctx.slots,
+                                       ctx.start_pos, act)
+            return K.StreamRows(stream, h, normed_by=nxt, convolved=True)
+        _, h = K.stream_add_many(stream, joins, nxt.weight, nxt.eps, nxt.norm_kind, act)
+        return K.StreamRows(stream, h, normed_by=nxt)
 
 
 class StreamInput(Part):
@@ -437,11 +517,32 @@ class StreamInput(Part):
     def bind(self, t):
         self.weight = t[""]
 
-    def forward(self, x, x0: torch.Tensor):
+    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0):
         if not isinstance(x, K.StreamRows):
             raise ValueError("a stream input mixes a 32-bit stream (`StreamRows`) with the rows it began as")
+        if x0_scale != 1.0:
+            raise ValueError("a stream input reads rows that carry no multiplier")
         y = K.linear(K.stream_pair_rows(x.f32, x0), self.weight, out_f32=True)
         return K.StreamRows(y, x0[:0])
+
+
+class StreamAdd(Part):
+    """x <- x + x0_scale * x0 on a 32-bit stream, x0 the embedding's rows (in the activation dtype): the embedding's output is
+    added once more.  A block that closes with `joins_opening` does it in its closing kernel instead.  No tensors."""
+    kernels = ("stream_layer",)
+    is_addend = True
+
+    def __init__(self, spec, perturb_init: bool = False):
+        self.spec = spec
+
+    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0):
+        if not isinstance(x, K.StreamRows):
+            raise ValueError("the embedding's output is added to a 32-bit stream (`StreamRows`)")
+        K.stream_add_many(x.f32, [(x0, x0_scale)], None, 0.0, "rmsnorm", x0.dtype)
+        return K.StreamRows(x.f32, x0[:0])
+
+
+STREAM_INPUTS = {"product": StreamInput, "add": StreamAdd}
 
 
 def _addends(y, scale: float = 1.0) -> list:

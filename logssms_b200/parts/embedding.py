@@ -66,19 +66,18 @@ class PairEmbedding(Part):
 
 @EMBEDDINGS.register("stream_embedding")
 class StreamEmbedding(Part):
-    """The token's row of the table as the first value of a 32-bit stream (`K.StreamRows`); the rows themselves, in the
-    activation dtype, stay at hand as the stream's `act` (a model whose layers mix them in again reads them there).
-    Tensor: `embed`."""
+    """The token's row of the table, times `multiplier` in 32-bit, as the first value of a 32-bit stream (`K.StreamRows`); the rows
+    themselves, in the activation dtype and without the multiplier, stay at hand as the stream's `act` (a model whose layers mix
+    them in again reads them there, and their factor as `stream_scale`).  Tensor: `embed`."""
     kernels = ("embed", "norm")
 
     def __init__(self, vocab_size: int, hidden_size: int, multiplier: float = 1.0):
-        if multiplier != 1.0:
-            raise ValueError("a stream embedding has no multiplier")
-        self.vocab_size, self.hidden_size = vocab_size, hidden_size
+        self.vocab_size, self.hidden_size, self.stream_scale = vocab_size, hidden_size, float(multiplier)
         self.weight = self.bad_ids = None
 
     def param_specs(self):
-        return {"embed": ParamSpec((self.vocab_size, self.hidden_size), MATRIX, normal_init(1.0))}
+        # random weights: rows of unit size once they are multiplied
+        return {"embed": ParamSpec((self.vocab_size, self.hidden_size), MATRIX, normal_init(1.0 / max(abs(self.stream_scale), 1e-3)))}
 
     def bind(self, t):
         self.weight = t["embed"]
@@ -86,7 +85,7 @@ class StreamEmbedding(Part):
 
     def forward(self, ids: torch.Tensor):
         rows = K.embed_gather(self.weight, ids, 1.0, self.bad_ids)
-        return K.StreamRows(K.scale(rows, 1.0, to_f32=True), rows)
+        return K.StreamRows(K.scale(rows, self.stream_scale, to_f32=True), rows)
 
 
 @EMBEDDINGS.register("normed_embedding")

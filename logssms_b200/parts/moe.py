@@ -114,7 +114,10 @@ class RoutedMLP(Part):
     `spec.expert = "silu"` weighted at the "output": w down(silu(gate h) * up h).  With `spec.shared_size` > 0 one more expert
     of that form and size (tensors shared.gate, shared.up, shared.down) runs for every token with weight 1: its gate and up
     rows lie behind the routed experts' in the one stacked product, its activations behind theirs, and its down matrix
-    behind theirs, so the one stacked down product adds it too."""
+    behind theirs, so the one stacked down product adds it too.  With `spec.shared_gate` its weight is sigmoid(shared.sg h), one
+    number per token: shared.sg is one more row of the router's matrix, whose kernel leaves that weight behind the experts'.
+    `spec.group_score = "pair"` ranks groups by the sum of their two best members; `spec.normalize` divides the chosen weights by
+    their sum."""
     kernels = ("moe", "linear_skinny", "gemm_tcgen05")
 
     def __init__(self, spec, perturb_init: bool = False, shared: dict | None = None):
@@ -125,6 +128,10 @@ class RoutedMLP(Part):
             raise ValueError("the softmax over the chosen outputs goes without correction, identity experts and groups")
         if getattr(spec, "shared_size", 0) and spec.num_identity:
             raise ValueError("a shared expert goes without identity experts")
+        if spec.shared_gate and not spec.shared_size:
+            raise ValueError("a gate of the shared expert needs a shared expert")
+        if spec.group_score not in ("best", "pair"):
+            raise ValueError(f"routed_mlp scores groups by their best member or pair, not {spec.group_score!r}")
         self.spec = spec
         self.shared_size = int(getattr(spec, "shared_size", 0))
         self.mode = {("clamped", "output"): "clamped", ("silu", "input"): "silu_input", ("silu", "output"): "silu"}.get((spec.expert, spec.weigh))
@@ -145,6 +152,8 @@ class RoutedMLP(Part):
             specs["shared.gate"] = ParamSpec((self.shared_size, s.hidden_size), MATRIX, fan)
             specs["shared.up"] = ParamSpec((self.shared_size, s.hidden_size), MATRIX, fan)
             specs["shared.down"] = ParamSpec((s.hidden_size, self.shared_size), MATRIX, normal_init(2.0 * self.shared_size ** -0.5))
+        if s.shared_gate:
+            specs["shared.sg"] = ParamSpec((1, s.hidden_size), VECTOR, normal_init(1.5 * s.hidden_size ** -0.5))
         for e in range(s.num_experts):
             specs[f"e{e}.gate"] = ParamSpec((s.expert_size, s.hidden_size), MATRIX, fan)
             specs[f"e{e}.up"] = ParamSpec((s.expert_size, s.hidden_size), MATRIX, fan)
@@ -154,6 +163,8 @@ class RoutedMLP(Part):
     def bind(self, t):
         s = self.spec
         self.router, self.correction, self.router_bias = t["router"], t.get("correction"), t.get("router.b")
+        if s.shared_gate:
+            self.router = torch.cat([self.router, t["shared.sg"]], 0).contiguous()
         shared = [t["shared.gate"], t["shared.up"]] if self.shared_size else []
         self.gate_up = torch.cat([t[f"e{e}.{n}"] for e in range(s.num_experts) for n in ("gate", "up")] + shared, 0).contiguous()
         self.down = torch.cat([t[f"e{e}.down"] for e in range(s.num_experts)] + ([t["shared.down"]] if self.shared_size else []), 1).contiguous()
@@ -165,7 +176,8 @@ class RoutedMLP(Part):
         s = self.spec
         dense, _, _, id_weight = K.moe_route(x, self.router, self.correction, s.num_experts, s.top, s.num_groups,
                                              s.keep_groups, s.route_scale, sigmoid_scores=s.score == "sigmoid",
-                                             bias=self.router_bias, chosen_softmax=s.score == "softmax_chosen")
+                                             bias=self.router_bias, chosen_softmax=s.score == "softmax_chosen",
+                                             pair_groups=s.group_score == "pair", normalize=s.normalize, gates=int(s.shared_gate))
         if s.num_experts == 0:
             return torch.zeros_like(x), x, id_weight
         gate_up = K.linear(x, self.gate_up)
@@ -174,7 +186,8 @@ class RoutedMLP(Part):
             routed = s.num_experts * s.expert_size
             y = torch.empty((x.shape[0], routed + self.shared_size), dtype=gate_up.dtype, device=gate_up.device)
             K.moe_activation(gate_up[:, :2 * routed], dense, s.num_experts, s.limit, s.act_alpha, mode=self.mode, out=y[:, :routed])
-            K.moe_activation(gate_up[:, 2 * routed:], None, 1, s.limit, s.act_alpha, mode=self.mode, out=y[:, routed:])
+            K.moe_activation(gate_up[:, 2 * routed:], dense[:, s.num_experts:] if s.shared_gate else None, 1, s.limit, s.act_alpha,
+                             mode=self.mode, out=y[:, routed:])
         else:
             y = K.moe_activation(gate_up, dense, s.num_experts, s.limit, s.act_alpha, mode=self.mode)
         out = K.linear(y, self.down)

@@ -26,16 +26,22 @@ class RMSNorm(Part):
         # `offset`: the norm multiplies by offset + the stored weight (1.0: a weight that is stored around zero); the sum is
         # made once, in 32-bit, when the weight arrives
         self.offset = float(getattr(spec, "offset", 0.0))
+        # `scalar`: the stored weight is one number, spread over all coordinates when it arrives
+        self.scalar = bool(getattr(spec, "scalar", False))
         self._jitter = 0.1 if perturb_init else 0.0
         self.weight: torch.Tensor | None = None
 
     def param_specs(self):
+        shape = () if self.scalar else (self.size,)
         if self.offset != 0.0:
-            return {self.param_name: ParamSpec((self.size,), VECTOR, normal_init(self._jitter))}
-        return {self.param_name: ParamSpec((self.size,), VECTOR, ones_init(self._jitter))}
+            return {self.param_name: ParamSpec(shape, VECTOR, normal_init(self._jitter))}
+        return {self.param_name: ParamSpec(shape, VECTOR, ones_init(self._jitter))}
 
     def bind(self, t):
-        self.weight = t[self.param_name] if self.offset == 0.0 else t[self.param_name] + self.offset
+        w = t[self.param_name]
+        if self.scalar:
+            w = w.reshape(1).expand(self.size).contiguous()
+        self.weight = w if self.offset == 0.0 else w + self.offset
 
     def post(self, stream, y, skip_scale: float = 1.0, *, extra=None, row_scale=None):
         """Post-norm on a 32-bit stream: norm(skip_scale * stream + y [+ row_scale[t] * extra]) as `K.StreamRows`."""
