@@ -840,8 +840,34 @@ ZARISUN_SIZES = {
     "w1024": (_zarisun_config(1024, 8, 2, 64, 128, 256, 32, 1024, 2048, 32768), PUPOPEL_SIZES["w1024"][0]),
     "w2048": (_zarisun_config(2048, 16, 4, 128, 128, 512, 64, 2048, 8192, 65536), PUPOPEL_SIZES["w2048"][0]),
 }
+
+
+def _dimudra_config(width: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, window: int, state: int, experts: int, top: int,
+                    expert_ff: int, shared_ff: int, vocab: int) -> dict:
+    """Layer sizes that resemble a real model's, every mixer once and HGRN2 twice: a pair of attention over a window and a selective
+    scan of twice the width, linear attention whose forget gate decides what is written, rotary attention over all keys; routed
+    feed-forwards in groups with a gated shared expert; a loop of one pass (the closest model's layers run once too)."""
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": key_dim, "vdim": key_dim, "scale": key_dim ** -0.5}
+    pair = {"type": "parallel", "mixer": {"left": {**attention, "mask": {"size": window}},
+                                          "right": {"inner": 2 * width, "state": state, "dt_rank": width // 16, "conv": 4},
+                                          "left_scale": 1.0, "right_scale": 1.0}}
+    hgrn = {"type": "hgrn2", "mixer": {"heads": heads, "dim": key_dim, "vdim": value_dim}}
+    rotary = {"type": "attention", "mixer": {**attention, "rot": {"base": 10000.0, "dims": key_dim // 2}}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": shared_ff}}
+    return {"architecture": "Dimudra", "layers": [{**m, "mlp": moe} for m in (pair, hgrn, rotary, hgrn)], "canon": {"taps": 4},
+            "embedding": {"scale": 16.0}, "loop": {"start": 1, "stop": 3, "times": 1}, "norm": {"eps": 1e-5}, "vocab": vocab, "width": width}
+
+
+# Dimudra beside Pupopel (the closest existing model: a 32-bit stream, a pair of softmax attention and a linear recurrence side by
+# side, a recurrent mixer with a matrix state per head, routed feed-forwards with a shared expert computed over all experts) at the
+# same width, depth, vocabulary, head and expert sizes
+DIMUDRA_SIZES = {
+    "w1024": (_dimudra_config(1024, 8, 2, 64, 128, 1024, 16, 8, 2, 1024, 1024, 32768), PUPOPEL_SIZES["w1024"][0]),
+    "w2048": (_dimudra_config(2048, 16, 4, 128, 128, 2048, 16, 16, 4, 1408, 1408, 65536), PUPOPEL_SIZES["w2048"][0]),
+}
 DESIGNS = {"dudurax": (DESIGN_SIZES, "falcon_h1"), "kuvazen": (KUVAZEN_SIZES, "dudurax"), "pupopel": (PUPOPEL_SIZES, "dudurax"),
-           "zarisun": (ZARISUN_SIZES, "pupopel")}
+           "zarisun": (ZARISUN_SIZES, "pupopel"), "dimudra": (DIMUDRA_SIZES, "pupopel")}
 
 
 def _design_point(cfg: dict, vocab: int, K: int, W: int, batch: int, context: int) -> dict:
@@ -914,7 +940,7 @@ def _design_point(cfg: dict, vocab: int, K: int, W: int, batch: int, context: in
 
 def run_design(args) -> dict:
     """`--design NAME`: that design at a few layer sizes beside the closest existing model at the same width and depth
-    (Dudurax beside Falcon-H1, Kuvazen and Pupopel beside Dudurax, Zarisun beside Pupopel)."""
+    (Dudurax beside Falcon-H1, Kuvazen and Pupopel beside Dudurax, Zarisun and Dimudra beside Pupopel)."""
     table, beside = DESIGNS[args.design]
     sizes = {}
     for name, (new, closest) in table.items():
@@ -975,7 +1001,7 @@ def main() -> int:
     ap.add_argument("--reference-timeout", type=int, default=900, help="seconds the reference arm may take")
     ap.add_argument("--probe", choices=["decode", "prefill", "mixed"], default=None,
                     help="a short run of one kind of step for a profiler (see profiles/); prints no benchmark line")
-    ap.add_argument("--design", choices=["dudurax", "kuvazen", "pupopel", "zarisun"], default=None,
+    ap.add_argument("--design", choices=["dudurax", "kuvazen", "pupopel", "zarisun", "dimudra"], default=None,
                     help="prefill and decode of another design at a few layer sizes beside the closest existing model "
                          "(one JSON line of its own; the default workload is untouched)")
     args = ap.parse_args()

@@ -19,7 +19,8 @@
 //                     multiplied by the weight (gate and up are linear in it).  Without weights (`dense` null, one
 //                     expert) it is the activation of a dense gated layer.  Modes `kSiluOutput` and `kGeluOutput`:
 //                     y = w * silu(g) * u and y = w * gelu_tanh(g) * u.  Input and output rows may be column views
-//                     of wider matrices (row strides in elements).
+//                     of wider matrices (row strides in elements).  `tail_ff` > 0: behind the experts' columns lies one
+//                     more expert of that size (input gate | up, output), whose weight is dense column `tail_gate`, or 1.
 //  moe_add_identity : out += id_weight[t] * h
 //  gelu_tanh        : 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 #include "lb200/common.cuh"
@@ -28,41 +29,79 @@ using namespace lb200;
 constexpr int kRouteMax = 256;        // router outputs
 constexpr int kRouteWarps = 16;       // warps of a token's CTA: each takes every sixteenth router output
 
-// grid (tokens)
-template <typename T>
+// the index of the largest v[i] among those with ok[i] (ties: the lower index), -1 if there is none; by one warp, all lanes get it
+__device__ __forceinline__ int warp_best(const float* v, const unsigned char* ok, int n) {
+    unsigned key = 0, at = 0xffffffffu;                    // floats as unsigned integers of the same order; 0: none
+    for (int i = threadIdx.x & 31; i < n; i += 32) {
+        const unsigned bits = __float_as_uint(v[i]);
+        const unsigned k = ok[i] ? ((bits & 0x80000000u) ? ~bits : bits | 0x80000000u) : 0u;
+        if (k > key) { key = k; at = i; }
+    }
+    const unsigned best = __reduce_max_sync(0xffffffffu, key);
+    if (best == 0) return -1;
+    return (int)__reduce_min_sync(0xffffffffu, key == best ? at : 0xffffffffu);
+}
+
+// four consecutive values as floats
+__device__ __forceinline__ float4 four(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 four(const __nv_bfloat16* p) {
+    const uint2 v = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&v.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// grid (ceil(tokens / kTok)): a CTA takes kTok neighbouring tokens, so that a row of W_r is read once for all of them; its warps
+// share the rows, then warp k chooses for token k.  VEC: four columns at a time (width a multiple of 4, rows 16-byte aligned).
+template <typename T, int kTok, bool VEC>
 __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
         const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ correction,
         float* __restrict__ dense, int* __restrict__ chosen, float* __restrict__ chosen_w,
         float* __restrict__ id_weight, int tokens, int width, int n, int experts, int top,
         int groups, int keep, float scale, int sigmoid_scores, const float* __restrict__ bias, int pair_groups, int normalize,
         int gates) {
-    __shared__ float z[kRouteMax];
-    __shared__ float c[kRouteMax];
-    __shared__ unsigned char ok[kRouteMax];
+    __shared__ float zs[kTok][kRouteMax], cs[kTok][kRouteMax], gss[kTok][kRouteMax], shares[kTok][kRouteMax];
+    __shared__ int pickeds[kTok][kRouteMax];
+    __shared__ unsigned char oks[kTok][kRouteMax], goks[kTok][kRouteMax];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int t = blockIdx.x;
-    const T* hr = h + (size_t)t * width;
+    const int first = blockIdx.x * kTok;
     const int nd = n + gates;                              // columns of the dense weights
     for (int e = warp; e < nd; e += kRouteWarps) {
         const float* wr = w_router + (size_t)e * width;
-        float a0 = 0.f, a1 = 0.f, a2 = 0.f, a3 = 0.f;
-        int k = lane;
-#pragma unroll 2
-        for (; k + 96 < width; k += 128) {
-            a0 += to_f32(hr[k]) * wr[k];
-            a1 += to_f32(hr[k + 32]) * wr[k + 32];
-            a2 += to_f32(hr[k + 64]) * wr[k + 64];
-            a3 += to_f32(hr[k + 96]) * wr[k + 96];
+        float acc[kTok];
+#pragma unroll
+        for (int k = 0; k < kTok; ++k) acc[k] = 0.f;
+        if (VEC) {
+#pragma unroll 4
+            for (int c = lane * 4; c < width; c += 128) {
+                const float4 wv = four(wr + c);
+#pragma unroll
+                for (int k = 0; k < kTok; ++k) {
+                    const float4 hv = four(h + (size_t)min(first + k, tokens - 1) * width + c);
+                    acc[k] += (hv.x * wv.x + hv.y * wv.y) + (hv.z * wv.z + hv.w * wv.w);
+                }
+            }
+        } else {
+            for (int c = lane; c < width; c += 32) {
+                const float wv = wr[c];
+#pragma unroll
+                for (int k = 0; k < kTok; ++k) acc[k] += to_f32(h[(size_t)min(first + k, tokens - 1) * width + c]) * wv;
+            }
         }
-        for (; k < width; k += 32) a0 += to_f32(hr[k]) * wr[k];
-        const float a = warp_sum((a0 + a1) + (a2 + a3));
-        if (lane == 0) {
-            if (e < n) z[e] = a + (bias != nullptr ? bias[e] : 0.f);
-            else dense[(size_t)t * nd + e] = 1.f / (1.f + expf(-a));
+#pragma unroll
+        for (int k = 0; k < kTok; ++k) {
+            const float a = warp_sum(acc[k]);
+            if (lane == 0 && first + k < tokens) {
+                if (e < n) zs[k][e] = a + (bias != nullptr ? bias[e] : 0.f);
+                else dense[(size_t)(first + k) * nd + e] = 1.f / (1.f + expf(-a));
+            }
         }
     }
     __syncthreads();
-    if (warp != 0) return;
+    const int t = first + warp;
+    if (warp >= kTok || t >= tokens) return;
+    float *z = zs[warp], *c = cs[warp], *gs = gss[warp], *share = shares[warp];
+    int* picked = pickeds[warp];
+    unsigned char *ok = oks[warp], *gok = goks[warp];
     const bool chosen_softmax = sigmoid_scores == 2;
     float mx = 0.f, sum = 1.f;
     if (sigmoid_scores == 0) {
@@ -85,75 +124,56 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
         dense[(size_t)t * nd + e] = 0.f;
     }
     __syncwarp();
-    if (lane != 0) return;
     // the groups that stay: `keep` times the group whose best member (or best two) is largest (ties: the lower index)
     const int per = n / groups;
+    for (int g = lane; g < groups; g += 32) {
+        float gm = -INFINITY, second = -INFINITY;
+        for (int i = 0; i < per; ++i) {
+            const float v = c[g * per + i];
+            if (v > gm) { second = gm; gm = v; }
+            else second = fmaxf(second, v);
+        }
+        gs[g] = (pair_groups && per > 1) ? gm + second : gm;
+        gok[g] = 1;
+    }
+    __syncwarp();
     for (int r = 0; r < keep; ++r) {
-        int best_g = -1;
-        float best = -INFINITY;
-        for (int g = 0; g < groups; ++g) {
-            if (ok[g * per]) continue;
-            float gm = -INFINITY, second = -INFINITY;
-            for (int i = 0; i < per; ++i) {
-                const float v = c[g * per + i];
-                if (v > gm) { second = gm; gm = v; }
-                else second = fmaxf(second, v);
-            }
-            if (pair_groups && per > 1) gm += second;
-            if (best_g < 0 || gm > best) { best = gm; best_g = g; }
-        }
+        const int best_g = warp_best(gs, gok, groups);
         if (best_g < 0) break;
-        for (int i = 0; i < per; ++i) ok[best_g * per + i] = 1;
+        for (int i = lane; i < per; i += 32) ok[best_g * per + i] = 1;
+        if (lane == 0) gok[best_g] = 0;
+        __syncwarp();
     }
-    float idw = 0.f;
-    if (chosen_softmax) {
-        // the `top` largest logits, then the softmax over them alone
-        float best_all = -INFINITY, total = 0.f;
-        for (int r = 0; r < top; ++r) {
-            int best_e = -1;
-            float best = -INFINITY;
-            for (int e = 0; e < n; ++e)
-                if (ok[e] == 1 && (best_e < 0 || c[e] > best)) { best = c[e]; best_e = e; }
-            chosen[(size_t)t * top + r] = best_e;
-            if (best_e < 0) { chosen_w[(size_t)t * top + r] = 0.f; continue; }
-            ok[best_e] = 2;
-            if (r == 0) best_all = best;
-            const float p = expf(best - best_all);
-            chosen_w[(size_t)t * top + r] = p;
-            total += p;
-        }
-        for (int r = 0; r < top; ++r) {
-            const int e = chosen[(size_t)t * top + r];
-            if (e < 0) continue;
-            const float wgt = chosen_w[(size_t)t * top + r] / total * scale;
-            chosen_w[(size_t)t * top + r] = wgt;
-            dense[(size_t)t * nd + e] = wgt;
-            if (e >= experts) idw += wgt;
-        }
-        id_weight[t] = idw;
-        return;
-    }
-    float total = 0.f;
+    // the `top` best of what stays: chosen_softmax weighs them by the softmax over their logits, the others by their scores
+    float idw = 0.f, total = 0.f, best_all = 0.f;
     for (int r = 0; r < top; ++r) {
-        int best_e = -1;
-        float best = -INFINITY;
-        for (int e = 0; e < n; ++e)
-            if (ok[e] == 1 && (best_e < 0 || c[e] > best)) { best = c[e]; best_e = e; }
-        chosen[(size_t)t * top + r] = best_e;
-        if (best_e < 0) { chosen_w[(size_t)t * top + r] = 0.f; continue; }
-        ok[best_e] = 2;
-        total += z[best_e];
+        const int e = warp_best(c, ok, n);
+        float part = 0.f;
+        if (e >= 0) {
+            if (r == 0) best_all = c[e];
+            part = chosen_softmax ? expf(c[e] - best_all) : z[e];
+        }
+        total += part;
+        __syncwarp();
+        if (lane == 0) {
+            if (e >= 0) ok[e] = 0;
+            chosen[(size_t)t * top + r] = e;
+            picked[r] = e;
+            share[r] = part;
+        }
+        __syncwarp();
     }
     const float factor = normalize ? scale / (total + 1e-20f) : scale;
-    for (int r = 0; r < top; ++r) {
-        const int e = chosen[(size_t)t * top + r];
-        if (e < 0) continue;
-        const float wgt = z[e] * factor;
-        dense[(size_t)t * nd + e] = wgt;
+    for (int r = lane; r < top; r += 32) {
+        const int e = picked[r];
+        const float wgt = e < 0 ? 0.f : (chosen_softmax ? share[r] / total * scale : share[r] * factor);
         chosen_w[(size_t)t * top + r] = wgt;
+        if (e < 0) continue;
+        dense[(size_t)t * nd + e] = wgt;
         if (e >= experts) idw += wgt;
     }
-    id_weight[t] = idw;
+    idw = warp_sum(idw);
+    if (lane == 0) id_weight[t] = idw;
 }
 
 extern "C" int lb_moe_route(const void* h, const float* w_router, const float* correction, float* dense, int* chosen,
@@ -165,9 +185,14 @@ extern "C" int lb_moe_route(const void* h, const float* w_router, const float* c
         return kBadSize;
     if (n > kRouteMax) return kTooLarge;
     if (sigmoid_scores < 0 || sigmoid_scores > 2 || gates < 0 || (sigmoid_scores == 2 && normalize)) return kBadSize;
-    LB_DISPATCH_DTYPE(dtype, moe_route_kernel<T><<<tokens, kRouteWarps * 32, 0, (cudaStream_t)stream>>>(
-        (const T*)h, w_router, correction, dense, chosen, chosen_w, id_weight, tokens, width, n, experts, top, groups, keep, scale, sigmoid_scores, bias,
-        pair_groups, normalize, gates));
+    const bool vec = width % 4 == 0 && ((uintptr_t)h & 7) == 0 && ((uintptr_t)w_router & 15) == 0 && (dtype == kBF16 || ((uintptr_t)h & 15) == 0);
+    const bool tile = tokens >= 4 * 148;                   // enough tokens for a CTA per four of them on every SM
+#define LB_ROUTE(TOK, V) LB_DISPATCH_DTYPE(dtype, moe_route_kernel<T, TOK, V><<<(tokens + TOK - 1) / TOK, kRouteWarps * 32, 0, (cudaStream_t)stream>>>( \
+        (const T*)h, w_router, correction, dense, chosen, chosen_w, id_weight, tokens, width, n, experts, top, groups, keep, scale, sigmoid_scores, bias, \
+        pair_groups, normalize, gates))
+    if (tile) { if (vec) { LB_ROUTE(4, true); } else { LB_ROUTE(4, false); } }
+    else { if (vec) { LB_ROUTE(1, true); } else { LB_ROUTE(1, false); } }
+#undef LB_ROUTE
     return launch_status();
 }
 
@@ -187,20 +212,23 @@ __device__ __forceinline__ float expert_act(float g, float u, float w, float lim
     return w * (g / (1.f + expf(-act_alpha * g)) * (u + 1.f));
 }
 
-// gu: [T, experts, 2, ff]; y: [T, experts, ff]; dense: [T, n] (null: weight 1)
+// gu: [T, experts, 2, ff] [2, tail_ff]; y: [T, experts, ff] [tail_ff]; dense: [T, n] (null: weight 1)
 template <typename T>
 __global__ void moe_activation_kernel(const T* __restrict__ gu, const float* __restrict__ dense, T* __restrict__ y,
                                       int experts, int ff, int n, float limit, float act_alpha, int mode, long in_stride,
-                                      long out_stride) {
+                                      long out_stride, int tail_ff, int tail_gate) {
     const size_t t = blockIdx.z;
     const int e = blockIdx.y;
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i >= ff) return;
-    const float w = dense != nullptr ? dense[t * n + e] : 1.f;
+    const bool tail = e == experts;
+    const int size = tail ? tail_ff : ff;
+    if (i >= size) return;
+    const int col = tail ? tail_gate : e;
+    const float w = (dense != nullptr && col >= 0) ? dense[t * n + col] : 1.f;
     float v = 0.f;
     if (w != 0.f) {
         const T* row = gu + t * in_stride + e * 2 * (size_t)ff;
-        v = expert_act(to_f32(row[i]), to_f32(row[ff + i]), w, limit, act_alpha, mode);
+        v = expert_act(to_f32(row[i]), to_f32(row[size + i]), w, limit, act_alpha, mode);
     }
     y[t * out_stride + e * (size_t)ff + i] = from_f32<T>(v);
 }
@@ -210,17 +238,19 @@ __global__ void moe_activation_kernel(const T* __restrict__ gu, const float* __r
 __global__ void __launch_bounds__(256) moe_activation_vec_kernel(const __nv_bfloat16* __restrict__ gu, const float* __restrict__ dense,
                                                                  __nv_bfloat16* __restrict__ y, int experts, int ff, int n,
                                                                  float limit, float act_alpha, int mode, long in_stride,
-                                                                 long out_stride) {
+                                                                 long out_stride, int tail_ff, int tail_gate) {
     const size_t t = blockIdx.x;
-    const int pieces = ff / 8;
-    for (int i = threadIdx.x; i < experts * pieces; i += blockDim.x) {
-        const int e = i / pieces, pc = i % pieces;
-        const float w = dense != nullptr ? dense[t * n + e] : 1.f;
+    const int pieces = ff / 8, all = experts * pieces;
+    for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < all + tail_ff / 8; i += gridDim.y * blockDim.x) {
+        const bool tail = i >= all;
+        const int e = tail ? experts : i / pieces, pc = tail ? i - all : i % pieces;
+        const int size = tail ? tail_ff : ff, col = tail ? tail_gate : e;
+        const float w = (dense != nullptr && col >= 0) ? dense[t * n + col] : 1.f;
         uint4 out = make_uint4(0, 0, 0, 0);
         if (w != 0.f) {
             const __nv_bfloat16* row = gu + t * in_stride + e * 2 * (size_t)ff;
             const uint4 gv = *reinterpret_cast<const uint4*>(row + pc * 8);
-            const uint4 uv = *reinterpret_cast<const uint4*>(row + ff + pc * 8);
+            const uint4 uv = *reinterpret_cast<const uint4*>(row + size + pc * 8);
             const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
             const __nv_bfloat162* u2 = reinterpret_cast<const __nv_bfloat162*>(&uv);
             __nv_bfloat162* o2 = reinterpret_cast<__nv_bfloat162*>(&out);
@@ -247,19 +277,23 @@ __global__ void __launch_bounds__(256) moe_activation_vec_kernel(const __nv_bflo
 }
 
 extern "C" int lb_moe_activation(const void* gu, const float* dense, void* y, int tokens, int experts, int ff, int n, float limit,
-                                 float act_alpha, int mode, long in_stride, long out_stride, int dtype, void* stream) {
+                                 float act_alpha, int mode, long in_stride, long out_stride, int tail_ff, int tail_gate, int dtype,
+                                 void* stream) {
     if (tokens <= 0 || experts <= 0) return kOk;
-    if (ff <= 0 || (dense != nullptr && n < experts) || experts > 65535 || mode < kClampedOutput || mode > kGeluOutput
-        || in_stride < 2 * (long)experts * ff || out_stride < (long)experts * ff)
+    if (ff <= 0 || (dense != nullptr && n < experts) || experts > 65534 || mode < kClampedOutput || mode > kGeluOutput || tail_ff < 0
+        || tail_gate >= n || in_stride < 2 * ((long)experts * ff + tail_ff) || out_stride < (long)experts * ff + tail_ff)
         return kBadSize;
-    if (dtype == kBF16 && ff % 8 == 0 && (((uintptr_t)gu | (uintptr_t)y) & 15) == 0 && in_stride % 8 == 0 && out_stride % 8 == 0) {
-        moe_activation_vec_kernel<<<tokens, 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, dense, (__nv_bfloat16*)y, experts, ff,
-                                                                          n, limit, act_alpha, mode, in_stride, out_stride);
+    if (dtype == kBF16 && ff % 8 == 0 && tail_ff % 8 == 0 && (((uintptr_t)gu | (uintptr_t)y) & 15) == 0 && in_stride % 8 == 0 && out_stride % 8 == 0) {
+        // few tokens: several CTAs share a token's columns
+        const int pieces = (experts * ff + tail_ff) / 8;
+        const int split = tokens >= 148 ? 1 : min(max(1, 296 / tokens), (pieces + 255) / 256);
+        moe_activation_vec_kernel<<<dim3(tokens, split), 256, 0, (cudaStream_t)stream>>>((const __nv_bfloat16*)gu, dense, (__nv_bfloat16*)y, experts, ff,
+                                                                          n, limit, act_alpha, mode, in_stride, out_stride, tail_ff, tail_gate);
         return launch_status();
     }
-    dim3 grid((ff + 127) / 128, experts, tokens);
+    dim3 grid((max(ff, tail_ff) + 127) / 128, experts + (tail_ff > 0), tokens);
     LB_DISPATCH_DTYPE(dtype, moe_activation_kernel<T><<<grid, 128, 0, (cudaStream_t)stream>>>(
-        (const T*)gu, dense, (T*)y, experts, ff, n, limit, act_alpha, mode, in_stride, out_stride));
+        (const T*)gu, dense, (T*)y, experts, ff, n, limit, act_alpha, mode, in_stride, out_stride, tail_ff, tail_gate));
     return launch_status();
 }
 

@@ -1447,25 +1447,28 @@ EXPERT_MODES = {"clamped": 0, "silu_input": 1, "silu": 2, "gelu_tanh": 3}
 
 
 def moe_activation(gate_up: torch.Tensor, dense: torch.Tensor | None, num_experts: int, limit: float, act_alpha: float,
-                   mode: str = "clamped", out: torch.Tensor | None = None) -> torch.Tensor:
+                   mode: str = "clamped", out: torch.Tensor | None = None, tail: int = 0, tail_gate: int = -1) -> torch.Tensor:
     """gate_up: [T, experts * 2 * ff] (per expert gate | up); returns [T, experts * ff] with every expert's gated
     activation and the token's weight for that expert (0 where the expert was not chosen).  Mode "clamped": weight *
     g~ sigmoid(act_alpha g~) (u~ + 1) with gate and up clamped at `limit`; "silu_input": silu(w g) * (w u), the expert on
     an input that was multiplied by the weight; "silu", "gelu_tanh": weight * act(g) * u.  `dense` None: every weight is 1 (a
-    dense gated layer: one expert).  `gate_up` and `out` ([T, experts * ff]) may be column views of wider matrices."""
+    dense gated layer: one expert).  `gate_up` and `out` ([T, experts * ff]) may be column views of wider matrices.  With `tail`
+    one more expert of that size follows the others in both; its weight is dense column `tail_gate` (-1: 1)."""
     _cuda(gate_up, dense, out)
     T = gate_up.shape[0]
-    ff = gate_up.shape[1] // (2 * num_experts)
-    _need(gate_up.dim() == 2 and gate_up.stride(1) == 1 and gate_up.shape[1] == 2 * num_experts * ff, "gate_up must be [T, experts*2*ff], unit column stride")
+    ff = (gate_up.shape[1] - 2 * tail) // (2 * num_experts)
+    cols = num_experts * ff + tail
+    _need(gate_up.dim() == 2 and gate_up.stride(1) == 1 and gate_up.shape[1] == 2 * cols, "gate_up must be [T, experts*2*ff], unit column stride")
+    _need(tail_gate < (0 if dense is None else dense.shape[1]), "the tail's weight is a column of the dense weights")
     _need(dense is None or (dense.dtype == torch.float32 and dense.stride(1) == 1 and dense.shape[0] == T and dense.shape[1] >= num_experts),
           "dense weights float32 [T, n] (a column view is fine)")
-    y = out if out is not None else torch.empty((T, num_experts * ff), dtype=gate_up.dtype, device=gate_up.device)
-    _need(y.shape == (T, num_experts * ff) and y.dtype == gate_up.dtype and y.stride(1) == 1, "out must be [T, experts*ff] of gate_up's dtype")
+    y = out if out is not None else torch.empty((T, cols), dtype=gate_up.dtype, device=gate_up.device)
+    _need(y.shape == (T, cols) and y.dtype == gate_up.dtype and y.stride(1) == 1, "out must be [T, experts*ff] of gate_up's dtype")
     f = _fn("moe", "lb_moe_activation", [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_int, c_long, c_long,
-                                         c_int, c_void_p])
+                                         c_int, c_int, c_int, c_void_p])
     _check(f(_ptr(gate_up), _ptr(dense), _ptr(y), T, num_experts, ff, 0 if dense is None else max(dense.stride(0), dense.shape[1]), limit, act_alpha,
              EXPERT_MODES[mode], gate_up.stride(0) if T > 1 else max(gate_up.stride(0), gate_up.shape[1]),
-             y.stride(0) if T > 1 else max(y.stride(0), y.shape[1]), _code(gate_up), _stream()), "moe_activation")
+             y.stride(0) if T > 1 else max(y.stride(0), y.shape[1]), tail, tail_gate, _code(gate_up), _stream()), "moe_activation")
     return y
 
 

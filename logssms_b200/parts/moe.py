@@ -181,15 +181,8 @@ class RoutedMLP(Part):
         if s.num_experts == 0:
             return torch.zeros_like(x), x, id_weight
         gate_up = K.linear(x, self.gate_up)
-        if self.shared_size:
-            # the routed experts' activations and the shared expert's side by side, as the stacked down matrix wants them
-            routed = s.num_experts * s.expert_size
-            y = torch.empty((x.shape[0], routed + self.shared_size), dtype=gate_up.dtype, device=gate_up.device)
-            K.moe_activation(gate_up[:, :2 * routed], dense, s.num_experts, s.limit, s.act_alpha, mode=self.mode, out=y[:, :routed])
-            K.moe_activation(gate_up[:, 2 * routed:], dense[:, s.num_experts:] if s.shared_gate else None, 1, s.limit, s.act_alpha,
-                             mode=self.mode, out=y[:, routed:])
-        else:
-            y = K.moe_activation(gate_up, dense, s.num_experts, s.limit, s.act_alpha, mode=self.mode)
+        y = K.moe_activation(gate_up, dense, s.num_experts, s.limit, s.act_alpha, mode=self.mode, tail=self.shared_size,
+                             tail_gate=s.num_experts if s.shared_gate else -1)
         out = K.linear(y, self.down)
         if s.num_identity == 0:
             return out

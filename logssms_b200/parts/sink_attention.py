@@ -103,7 +103,7 @@ class MixerPair(Part):
     """Two mixers side by side on the same input h: out_scale_left * left(h) + out_scale_right * right(h).  `forward` hands
     back the two outputs with their scales, as a list of (rows, scale): the kernel that joins the layer's sublayers to the
     stream adds them in 32-bit.  Both use the block's cache layer (at most one of them keeps keys and values; their state
-    names must differ).  Tensors: the two mixers' own, under their slots' names."""
+    names must differ).  In a captured step of few rows the right one runs beside the left one, on a stream to spare.  Tensors: the two mixers' own, under their slots' names."""
 
     def __init__(self, spec, perturb_init: bool = False, shared: dict | None = None):
         self.spec = spec
@@ -136,9 +136,20 @@ class MixerPair(Part):
             raise ValueError(f"state names clash inside a mixer pair: {names}")
         return CacheNeeds(kv=kv, states=tuple(states))
 
+    BESIDE_MAX_ROWS = 64      # with more rows each mixer's kernels fill the GPU by themselves
+
     def forward(self, x: torch.Tensor, ctx, cache_layer: int, writes_cache: bool = True):
+        results = [None, None]
+
+        def run(i: int) -> None:
+            results[i] = self.mixers[i].forward(x, ctx, cache_layer, writes_cache)
+        beside = ctx.fork() if x.shape[0] <= self.BESIDE_MAX_ROWS else None
+        run(0)
+        if beside is None:
+            run(1)
+        else:
+            beside(lambda: run(1))()
         outs = []
-        for slot, mixer in zip(self.slots, self.mixers):
-            y = mixer.forward(x, ctx, cache_layer, writes_cache)
+        for slot, y in zip(self.slots, results):
             outs += [(t, sc * slot.out_scale) for t, sc in y] if isinstance(y, list) else [(y, slot.out_scale)]
         return outs
