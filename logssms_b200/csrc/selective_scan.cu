@@ -107,24 +107,33 @@ __global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
     const T* x = (const T*)a.x;
     const T* low = (const T*)a.low;
     const T* gate = (const T*)a.gate;
-    float rx[KX], rw[KX], rz[KX], rb[KB];
+    // the element of a block that this thread stages: token threadIdx.x / CH (+ kThreads / CH per turn), channel cl
+    constexpr int TSTEP = kThreads / CH;
+    const int tl = threadIdx.x / CH, cl = threadIdx.x % CH;
+    const bool cl_ok = c0 + cl < a.inner;
+    const float cl_bias = cl_ok ? a.dt_bias[c0 + cl] : 0.f, cl_D = cl_ok ? a.D[c0 + cl] : 0.f;
+    // (raw values: converting them here would wait for them here)
+    T rx[KX], rz[KX], rb[KB];
+    float rw[KX];
+    const T zero = from_f32<T>(0.f);
     auto fetch = [&](int t0) {
         const int nt = min(TB, last - t0);
 #pragma unroll
         for (int k = 0; k < KX; ++k) {
-            const int i = threadIdx.x + k * kThreads, t = i / CH, cc = c0 + i % CH;
-            rx[k] = rw[k] = rz[k] = 0.f;
-            if (t < nt && cc < a.inner) {
-                rx[k] = to_f32(x[(size_t)(t0 + t) * a.x_stride + cc]);
-                if (a.w != nullptr) rw[k] = a.w[(size_t)(t0 + t) * a.inner + cc];
-                if (with_out) rz[k] = to_f32(gate[(size_t)(t0 + t) * a.gate_stride + cc]);
+            const int t = tl + k * TSTEP;
+            rx[k] = rz[k] = zero;
+            rw[k] = 0.f;
+            if (t < nt && cl_ok) {
+                rx[k] = x[(size_t)(t0 + t) * a.x_stride + c0 + cl];
+                if (a.w != nullptr) rw[k] = a.w[(size_t)(t0 + t) * a.inner + c0 + cl];
+                if (with_out) rz[k] = gate[(size_t)(t0 + t) * a.gate_stride + c0 + cl];
             }
         }
 #pragma unroll
         for (int k = 0; k < KB; ++k) {
             const int i = threadIdx.x + k * kThreads, t = i / (2 * NP), r = i % (2 * NP);
             const int s = r < NP ? r : r - NP;
-            rb[k] = (t < nt && s < a.n) ? to_f32(low[(size_t)(t0 + t) * a.low_stride + a.rank + (r < NP ? 0 : a.n) + s]) : 0.f;
+            rb[k] = (t < nt && s < a.n) ? low[(size_t)(t0 + t) * a.low_stride + a.rank + (r < NP ? 0 : a.n) + s] : zero;
         }
     };
     fetch(first);
@@ -147,57 +156,79 @@ __global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
         }
 #pragma unroll
         for (int k = 0; k < KX; ++k) {
-            const int i = threadIdx.x + k * kThreads, t = i / CH, cl = i % CH;
+            const int t = tl + k * TSTEP;
             if (t < TB) {
-                const int cc = c0 + cl;
-                float dt = 0.f, d = 0.f;
-                if (t < nt && cc < a.inner) {
-                    dt = softplus_f((a.w != nullptr ? rw[k] : dts[t][cl]) + a.dt_bias[cc]);
-                    d = a.D[cc];
-                }
+                const float xv = to_f32(rx[k]);
+                const float dt = (t < nt && cl_ok) ? softplus_f((a.w != nullptr ? rw[k] : dts[t][cl]) + cl_bias) : 0.f;
                 dts[t][cl] = dt;
-                us[t][cl] = dt * rx[k];
-                ys[t][cl] = d * rx[k];
+                us[t][cl] = dt * xv;
+                ys[t][cl] = cl_D * xv;
             }
         }
 #pragma unroll
         for (int k = 0; k < KB; ++k) {
             const int i = threadIdx.x + k * kThreads, t = i / (2 * NP), r = i % (2 * NP);
             if (t < TB) {
-                if (r < NP) Bs[t][r] = rb[k];
-                else Cs[t][r - NP] = rb[k];
+                if (r < NP) Bs[t][r] = to_f32(rb[k]);
+                else Cs[t][r - NP] = to_f32(rb[k]);
             }
         }
         float z[KX];
 #pragma unroll
-        for (int k = 0; k < KX; ++k) z[k] = rz[k];
+        for (int k = 0; k < KX; ++k) z[k] = to_f32(rz[k]);
         if (t0 + TB < last) fetch(t0 + TB);
         __syncthreads();
-        if (with_out) {
-#pragma unroll 4
-            for (int t = 0; t < nt; ++t) {
-                const float dt = dts[t][ch], u = us[t][ch];
-                float acc = 0.f;
+        // one token for this thread's states: its share of the output sum
+        auto step = [&](int t) {
+            const float dt = dts[t][ch], u = us[t][ch];
+            float acc = 0.f;
 #pragma unroll
-                for (int i = 0; i < NPT; i += 4) {
-                    const float4 bv = *reinterpret_cast<const float4*>(&Bs[t][ln * NPT + i]);
-                    const float4 cv = *reinterpret_cast<const float4*>(&Cs[t][ln * NPT + i]);
-                    S[i] = ex2(dt * A2[i]) * S[i] + u * bv.x;
-                    S[i + 1] = ex2(dt * A2[i + 1]) * S[i + 1] + u * bv.y;
-                    S[i + 2] = ex2(dt * A2[i + 2]) * S[i + 2] + u * bv.z;
-                    S[i + 3] = ex2(dt * A2[i + 3]) * S[i + 3] + u * bv.w;
-                    acc += S[i] * cv.x + S[i + 1] * cv.y + S[i + 2] * cv.z + S[i + 3] * cv.w;
-                }
+            for (int i = 0; i < NPT; i += 4) {
+                const float4 bv = *reinterpret_cast<const float4*>(&Bs[t][ln * NPT + i]);
+                const float4 cv = *reinterpret_cast<const float4*>(&Cs[t][ln * NPT + i]);
+                S[i] = ex2(dt * A2[i]) * S[i] + u * bv.x;
+                S[i + 1] = ex2(dt * A2[i + 1]) * S[i + 1] + u * bv.y;
+                S[i + 2] = ex2(dt * A2[i + 2]) * S[i + 2] + u * bv.z;
+                S[i + 3] = ex2(dt * A2[i + 3]) * S[i + 3] + u * bv.w;
+                acc += S[i] * cv.x + S[i + 1] * cv.y + S[i + 2] * cv.z + S[i + 3] * cv.w;
+            }
+            return acc;
+        };
+        if (with_out) {
+            if (nt == 1) {
+                float acc = step(0);
 #pragma unroll
                 for (int off = 1; off < LN; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
-                if (ln == 0) ys[t][ch] += acc;
+                if (ln == 0) ys[0][ch] += acc;
+            } else {
+                // G tokens at a time, their sums over the LN lanes taken together: at every halving a lane keeps one half of
+                // the tokens and hands the other half over, so that lane g (mod G) ends with token g's sum.  (Tokens behind the
+                // last one have dt = 0 and zero inputs: they change nothing.)
+                constexpr int G = LN < TB ? LN : TB;
+                for (int g0 = 0; g0 < nt; g0 += G) {
+                    float acc[G];
+#pragma unroll
+                    for (int g = 0; g < G; ++g) acc[g] = step(g0 + g);
+#pragma unroll
+                    for (int off = G / 2; off > 0; off >>= 1) {
+                        const bool upper = ln & off;
+#pragma unroll
+                        for (int g = 0; g < off; ++g) {
+                            const float mine = upper ? acc[g + off] : acc[g], other = upper ? acc[g] : acc[g + off];
+                            acc[g] = mine + __shfl_xor_sync(0xffffffffu, other, off);
+                        }
+                    }
+#pragma unroll
+                    for (int off = G; off < LN; off <<= 1) acc[0] += __shfl_xor_sync(0xffffffffu, acc[0], off);
+                    if (ln < G) ys[g0 + ln][ch] += acc[0];
+                }
             }
             __syncthreads();
 #pragma unroll
             for (int k = 0; k < KX; ++k) {
-                const int i = threadIdx.x + k * kThreads, t = i / CH, cc = c0 + i % CH;
-                if (t < nt && cc < a.inner)
-                    ((T*)a.y)[(size_t)(t0 + t) * a.inner + cc] = from_f32<T>(ys[t][i % CH] * (sizeof(T) == 2 ? silu_fast(z[k]) : silu_f(z[k])));
+                const int t = tl + k * TSTEP;
+                if (t < nt && cl_ok)
+                    ((T*)a.y)[(size_t)(t0 + t) * a.inner + c0 + cl] = from_f32<T>(ys[t][cl] * (sizeof(T) == 2 ? silu_fast(z[k]) : silu_f(z[k])));
             }
         } else {
 #pragma unroll 4

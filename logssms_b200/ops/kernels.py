@@ -1979,14 +1979,14 @@ def selective_scan(x: torch.Tensor, w: torch.Tensor | None, low: torch.Tensor, d
 
 
 SELECTIVE_CHUNK = 64          # tokens; a segment is so many chunks of so many tokens
-SELECTIVE_SEGMENT = 4
+SELECTIVE_SEGMENT = 2
 
 
 def selective_segmented_pays(num_tokens: int, num_long: int, inner: int, state: int) -> bool:
-    """Should the long portions run as segments side by side?  When the CTAs of whole portions would leave most of the GPU
-    idle (a channel takes ceil(state / 4) lanes or fewer) and the portions are long enough to be cut."""
-    lanes = 1 << max(0, (min(-(-state // 4), 32) - 1).bit_length())
-    return num_tokens >= 2 * SELECTIVE_SEGMENT * SELECTIVE_CHUNK and num_long * inner * lanes // 32 < 8 * 4 * _SM_COUNT
+    """Should the long portions run as segments side by side (nearly every token twice)?  When the portions are long enough to be
+    cut and whole portions would be fewer than three warps for every two of the GPU's schedulers."""
+    lanes = next(ln for n, ln in ((4, 1), (8, 2), (16, 4), (64, 8), (128, 16), (256, 32)) if state <= n)      # lanes per channel
+    return num_tokens >= 2 * SELECTIVE_SEGMENT * SELECTIVE_CHUNK and 2 * (num_long * inner * lanes // 32) < 3 * 4 * _SM_COUNT
 
 
 def selective_scan_segments(x: torch.Tensor, w: torch.Tensor, low: torch.Tensor, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,

@@ -248,8 +248,8 @@ def test_mamba_in_portions(dtype, inner, state, rank, conv):
 
 @pytest.mark.parametrize("inner, state, rank, conv", [(40, 16, 4, 4), (24, 7, 3, 3)])
 def test_mamba_carries_the_state_through_segments(inner, state, rank, conv):
-    """Portions long enough to be cut into segments that run side by side (their edges at 256 tokens), a portion that ends a
-    token behind an edge, beside a short request, and decoded tokens after them; some channels hardly decay."""
+    """Portions long enough to be cut into segments that run side by side (their edges at multiples of 128 tokens), a portion
+    that ends a token behind an edge, beside a short request, and decoded tokens after them; some channels hardly decay."""
     from logssms_b200.ops import kernels as K
     for dtype in DTYPES:
         part, stored, m = mamba_part(dtype, inner, state, rank, conv, seed=state)
@@ -317,7 +317,7 @@ def test_selective_scan_kernels_equal_the_recurrence(inner, n, rank):
         state = state.cuda()
         if form == "segments":
             y = torch.empty(T, inner, device="cuda")
-            segments, _ = segment_lists(lens, K.SELECTIVE_CHUNK, K.SELECTIVE_SEGMENT, cap_segments=7, cap_long=2)
+            segments, _ = segment_lists(lens, K.SELECTIVE_CHUNK, K.SELECTIVE_SEGMENT, cap_segments=10, cap_long=2)
             K.selective_scan_segments(xz[:, :inner], w.cuda().contiguous(), low, *common, state, *where, torch.from_numpy(segments).cuda(), rank, y)
         else:
             y = K.selective_scan(xz[:, :inner], w.cuda().contiguous() if form == "handed in" else None, low, dt_w.cuda().contiguous(), *common, state,
