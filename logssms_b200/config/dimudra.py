@@ -23,6 +23,9 @@ ARCHITECTURE = "Dimudra"
 MIXER_TYPES = ("parallel", "hgrn2", "attention")
 MAX_TAPS = 8              # taps the convolution kernels are built for
 MAX_STATE = 256           # states per channel the selective scan is built for
+MAX_KEY_DIM = 512         # key channels per head the linear attention's kernels are built for
+MAX_EXPERTS = 256         # router outputs the router's kernel is built for
+MAX_VALUE_DIM = 256       # value columns per head the attention's kernels are built for
 
 
 def _sub(raw: Mapping[str, Any], key: str, where: str) -> Mapping[str, Any]:
@@ -48,7 +51,8 @@ def _attention(m: Mapping[str, Any], where: str) -> None:
     if _positive(m, "heads", where) % _positive(m, "kv_heads", where):
         raise ConfigError(f"{where}heads must be a multiple of kv_heads")
     _positive(m, "dim", where)
-    _positive(m, "vdim", where)
+    if _positive(m, "vdim", where) > MAX_VALUE_DIM:
+        raise ConfigError(f"{where}vdim must be at most {MAX_VALUE_DIM}")
     require(m, "scale", float)
     if m.get("mask") is not None:
         _positive(_sub(m, "mask", where), "size", where + "mask.")
@@ -70,6 +74,8 @@ def _moe(mlp: Mapping[str, Any], where: str) -> None:
     _positive(_sub(mlp, "expert", where), "ff", where + "expert.")
     router = _sub(mlp, "router", where)
     experts = _positive(router, "experts", where + "router.")
+    if experts > MAX_EXPERTS:
+        raise ConfigError(f"{where}router.experts must be at most {MAX_EXPERTS}")
     if not 1 <= require(router, "top", int) <= experts:
         raise ConfigError(f"{where}router.top must lie within 1 .. experts")
     if router.get("groups") is not None:
@@ -121,6 +127,8 @@ class DimudraConfig:
             elif kind == "hgrn2":
                 for key in ("heads", "dim", "vdim"):
                     _positive(mixer, key, where + "mixer.")
+                if int(mixer["dim"]) > MAX_KEY_DIM:
+                    raise ConfigError(f"{where}mixer.dim must be at most {MAX_KEY_DIM}")
             elif kind == "attention":
                 _attention(mixer, where + "mixer.")
             else:

@@ -27,7 +27,9 @@
 using namespace lb200;
 
 constexpr int kRouteMax = 256;        // router outputs
-constexpr int kRouteWarps = 16;       // warps of a token's CTA: each takes every sixteenth router output
+// warps of a CTA, which share the router outputs: one token per CTA (few tokens) takes many, several tokens fewer with more
+// registers each, so that more loads are in flight
+constexpr int route_warps(int tok) { return tok == 1 ? 16 : 8; }
 
 // the index of the largest v[i] among those with ok[i] (ties: the lower index), -1 if there is none; by one warp, all lanes get it
 __device__ __forceinline__ int warp_best(const float* v, const unsigned char* ok, int n) {
@@ -53,7 +55,7 @@ __device__ __forceinline__ float4 four(const __nv_bfloat16* p) {
 // grid (ceil(tokens / kTok)): a CTA takes kTok neighbouring tokens, so that a row of W_r is read once for all of them; its warps
 // share the rows, then warp k chooses for token k.  VEC: four columns at a time (width a multiple of 4, rows 16-byte aligned).
 template <typename T, int kTok, bool VEC>
-__global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
+__global__ void __launch_bounds__(route_warps(kTok) * 32) moe_route_kernel(
         const T* __restrict__ h, const float* __restrict__ w_router, const float* __restrict__ correction,
         float* __restrict__ dense, int* __restrict__ chosen, float* __restrict__ chosen_w,
         float* __restrict__ id_weight, int tokens, int width, int n, int experts, int top,
@@ -65,7 +67,7 @@ __global__ void __launch_bounds__(kRouteWarps * 32) moe_route_kernel(
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int first = blockIdx.x * kTok;
     const int nd = n + gates;                              // columns of the dense weights
-    for (int e = warp; e < nd; e += kRouteWarps) {
+    for (int e = warp; e < nd; e += route_warps(kTok)) {
         const float* wr = w_router + (size_t)e * width;
         float acc[kTok];
 #pragma unroll
@@ -187,7 +189,7 @@ extern "C" int lb_moe_route(const void* h, const float* w_router, const float* c
     if (sigmoid_scores < 0 || sigmoid_scores > 2 || gates < 0 || (sigmoid_scores == 2 && normalize)) return kBadSize;
     const bool vec = width % 4 == 0 && ((uintptr_t)h & 7) == 0 && ((uintptr_t)w_router & 15) == 0 && (dtype == kBF16 || ((uintptr_t)h & 15) == 0);
     const bool tile = tokens >= 4 * 148;                   // enough tokens for a CTA per four of them on every SM
-#define LB_ROUTE(TOK, V) LB_DISPATCH_DTYPE(dtype, moe_route_kernel<T, TOK, V><<<(tokens + TOK - 1) / TOK, kRouteWarps * 32, 0, (cudaStream_t)stream>>>( \
+#define LB_ROUTE(TOK, V) LB_DISPATCH_DTYPE(dtype, moe_route_kernel<T, TOK, V><<<(tokens + TOK - 1) / TOK, route_warps(TOK) * 32, 0, (cudaStream_t)stream>>>( \
         (const T*)h, w_router, correction, dense, chosen, chosen_w, id_weight, tokens, width, n, experts, top, groups, keep, scale, sigmoid_scores, bias, \
         pair_groups, normalize, gates))
     if (tile) { if (vec) { LB_ROUTE(4, true); } else { LB_ROUTE(4, false); } }

@@ -58,6 +58,9 @@ def test_looped_schedule():
     (("layers", 0, "mixer", "right", "state"), 257, "at most"),
     (("layers", 0, "mixer", "right", "dt_rank"), 0, "positive"),
     (("layers", 1, "mixer", "vdim"), 0, "positive"),
+    (("layers", 1, "mixer", "dim"), 513, "at most"),
+    (("layers", 2, "mixer", "vdim"), 257, "at most"),
+    (("layers", 0, "mlp", "router", "experts"), 260, "at most"),
     (("layers", 2, "mixer", "rot", "dims"), 7, "even"),
     (("layers", 2, "mixer", "rot", "dims"), 18, "at most"),
     (("layers", 2, "mixer", "rot", "base"), 0.0, "positive"),
