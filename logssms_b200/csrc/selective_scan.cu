@@ -80,30 +80,27 @@ __global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
         with_out = PASS == 2 || seg == 0;
     }
     if (first >= last) return;
+    // the thread's decay rates and states, as 16-byte pieces where the state size fills the lanes exactly; the rates are worked
+    // out after the first block's loads are on their way too
     float A2[NPT], S[NPT];
+    const bool full = a.n == NP && (((uintptr_t)a.A_log | (uintptr_t)a.state) & 15) == 0;
+    auto load_states = [&](const float* row, float (&out)[NPT]) {
+        if (full) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) {
-        const int s = ln * NPT + i;
-        A2[i] = (c_ok && s < a.n) ? -expf(a.A_log[(size_t)c * a.n + s]) * kLog2e : 0.f;
-        S[i] = 0.f;
-    }
+            for (int i = 0; i < NPT; i += 4) {
+                const float4 v = *reinterpret_cast<const float4*>(row + ln * NPT + i);
+                out[i] = v.x; out[i + 1] = v.y; out[i + 2] = v.z; out[i + 3] = v.w;
+            }
+        } else {
+#pragma unroll
+            for (int i = 0; i < NPT; ++i) out[i] = ln * NPT + i < a.n ? row[ln * NPT + i] : 0.f;
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) A2[i] = S[i] = 0.f;
+    if (c_ok) load_states(a.A_log + (size_t)c * a.n, A2);
     float* slot_state = a.state + ((size_t)a.slots[b] * a.inner + (c_ok ? c : 0)) * a.n;
-    if (PASS != 2) {
-        if (seg == 0 && a.start_pos[b] > 0 && c_ok) {
-#pragma unroll
-            for (int i = 0; i < NPT; ++i) if (ln * NPT + i < a.n) S[i] = slot_state[ln * NPT + i];
-        }
-    } else if (c_ok) {
-        // the segments before this one, joined in order (the first one's end state holds what the slot held)
-        for (int g = 0; g < seg; ++g) {
-            const size_t item = blockIdx.y - seg + g;
-            const float sum = g == 0 ? 0.f : a.seg_dt[item * a.inner + c];
-            const float* e = a.seg_state + (item * a.inner + c) * a.n;
-#pragma unroll
-            for (int i = 0; i < NPT; ++i)
-                if (ln * NPT + i < a.n) S[i] = (g == 0 ? 0.f : ex2(sum * A2[i]) * S[i]) + e[ln * NPT + i];
-        }
-    }
+    if (PASS != 2 && seg == 0 && a.start_pos[b] > 0 && c_ok) load_states(slot_state, S);
     const T* x = (const T*)a.x;
     const T* low = (const T*)a.low;
     const T* gate = (const T*)a.gate;
@@ -137,17 +134,44 @@ __global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
         }
     };
     fetch(first);
+#pragma unroll
+    for (int i = 0; i < NPT; ++i) A2[i] = (c_ok && ln * NPT + i < a.n) ? -expf(A2[i]) * kLog2e : 0.f;
+    if (PASS == 2 && c_ok) {
+        // the segments before this one, joined in order (the first one's end state holds what the slot held)
+        for (int g = 0; g < seg; ++g) {
+            const size_t item = blockIdx.y - seg + g;
+            const float sum = g == 0 ? 0.f : a.seg_dt[item * a.inner + c];
+            float e[NPT];
+            load_states(a.seg_state + (item * a.inner + c) * a.n, e);
+#pragma unroll
+            for (int i = 0; i < NPT; ++i) S[i] = ex2(sum * A2[i]) * S[i] + e[i];
+        }
+    }
     float dt_sum = 0.f;
     for (int t0 = first; t0 < last; t0 += TB) {
         const int nt = min(TB, last - t0);
         __syncthreads();                                   // the block before has left shared memory
         if (a.w == nullptr) {
-            // w = dt_w low: the lanes of a channel share its row of dt_w
+            // w = dt_w low: the lanes of a channel share its row of dt_w, in pieces of 16 bytes where they are aligned
+            constexpr int E = 16 / sizeof(T);
+            const bool pieces = a.rank % E == 0 && a.low_stride % E == 0 && (((uintptr_t)a.dt_w | (uintptr_t)a.low) & 15) == 0;
             for (int t = 0; t < nt; ++t) {
                 float acc = 0.f;
-                if (c_ok)
-                    for (int r = ln; r < a.rank; r += LN)
-                        acc += to_f32(((const T*)a.dt_w)[(size_t)c * a.rank + r]) * to_f32(low[(size_t)(t0 + t) * a.low_stride + r]);
+                const T* wr = (const T*)a.dt_w + (size_t)(c_ok ? c : 0) * a.rank;
+                const T* lr = low + (size_t)(t0 + t) * a.low_stride;
+                if (c_ok) {
+                    if (pieces) {
+#pragma unroll 4
+                        for (int r = ln * E; r < a.rank; r += LN * E) {
+                            const uint4 wv = *reinterpret_cast<const uint4*>(wr + r), lv = *reinterpret_cast<const uint4*>(lr + r);
+                            const T *we = reinterpret_cast<const T*>(&wv), *le = reinterpret_cast<const T*>(&lv);
+#pragma unroll
+                            for (int e = 0; e < E; ++e) acc += to_f32(we[e]) * to_f32(le[e]);
+                        }
+                    } else {
+                        for (int r = ln; r < a.rank; r += LN) acc += to_f32(wr[r]) * to_f32(lr[r]);
+                    }
+                }
 #pragma unroll
                 for (int off = 1; off < LN; off <<= 1) acc += __shfl_xor_sync(0xffffffffu, acc, off);
                 if (ln == 0) dts[t][ch] = acc;
@@ -254,8 +278,13 @@ __global__ void __launch_bounds__(kThreads) selective_scan_kernel(ScanArgs a) {
     } else if (PASS == 2 && !last_seg) {
         return;
     }
+    if (full) {
 #pragma unroll
-    for (int i = 0; i < NPT; ++i) if (ln * NPT + i < a.n) dst[ln * NPT + i] = S[i];
+        for (int i = 0; i < NPT; i += 4) *reinterpret_cast<float4*>(dst + ln * NPT + i) = make_float4(S[i], S[i + 1], S[i + 2], S[i + 3]);
+    } else {
+#pragma unroll
+        for (int i = 0; i < NPT; ++i) if (ln * NPT + i < a.n) dst[ln * NPT + i] = S[i];
+    }
 }
 
 template <typename T, int LN, int NPT, int TB>
