@@ -39,22 +39,27 @@ class PagedTensor:
 
 @dataclass(frozen=True)
 class PagedNeed:
-    """What a cache layer keeps per token, in pages: named tensors; `window`: only the last so many tokens are read.
+    """What a cache layer keeps per token, in pages: named tensors; `window`: only the last so many tokens are read, and with
+    `keep_first` the sequence's first so many tokens besides (their pages stay for the request's life).
     `every` > 1: one entry per run of so many tokens instead of one per token (a summary of every block of tokens);
     entry number position // every lies where a token of that number would lie in a group of single tokens."""
     tensors: tuple[PagedTensor, ...]
     window: int | None = None
     every: int = 1
+    keep_first: int = 0
 
     def __post_init__(self):
+        if self.keep_first < 0 or (self.keep_first > 0 and self.window is None):
+            raise ValueError("a paged need keeps its first tokens beside a window")
         if self.every < 1 or (self.every > 1 and self.window is not None):
             raise ValueError("a paged need has one entry per `every` >= 1 tokens, and a window only with every = 1")
 
 
-def KVNeed(num_kv_heads: int, head_dim: int, window: int | None = None, value_head_dim: int | None = None) -> PagedNeed:
+def KVNeed(num_kv_heads: int, head_dim: int, window: int | None = None, value_head_dim: int | None = None,
+           keep_first: int = 0) -> PagedNeed:
     """Keys "k" and values "v" of [num_kv_heads, head_dim] per token (values of another head size if given)."""
     return PagedNeed((PagedTensor("k", (num_kv_heads, head_dim)),
-                      PagedTensor("v", (num_kv_heads, value_head_dim or head_dim))), window)
+                      PagedTensor("v", (num_kv_heads, value_head_dim or head_dim))), window, keep_first=keep_first)
 
 
 @dataclass(frozen=True)
@@ -92,7 +97,9 @@ class PageGroup:
                                             device=device) for t in need.tensors}
         self.block_table = np.full((max_requests + 1, max_pages_per_request), -1, dtype=np.int32)
         self.block_table[max_requests, :] = num_pages
-        self.first_page = np.zeros(max_requests, dtype=np.int64)     # pages below are given back (window)
+        self.kept_pages = -(-need.keep_first // page_size)            # a request's first pages, which no window gives back
+        # pages below are given back (window), except for the kept ones
+        self.first_page = np.zeros(max_requests, dtype=np.int64)
         self.num_pages_of = np.zeros(max_requests, dtype=np.int64)    # logical pages handed out so far
 
     def tensor(self, name: str, layer: int) -> torch.Tensor:
@@ -109,13 +116,19 @@ class PageGroup:
         """Pages that hold the entries of `length` tokens (a last, unfinished run of `every` tokens has its entry)."""
         return -(-(-(-length // self.need.every)) // self.page_size)
 
+    def held(self, row: int) -> list[tuple[int, int]]:
+        """Ranges of logical pages that a request holds: the kept first ones, and what the window has not given back."""
+        n, lo = int(self.num_pages_of[row]), int(self.first_page[row])
+        kept = min(self.kept_pages, lo, n)
+        return [(0, kept), (lo, n)] if kept > 0 else [(lo, n)]
+
     def lifetime_pages(self, total_len: int, max_step_tokens: int) -> int:
         """Most pages a request of `total_len` tokens holds at any time."""
         full = self.pages_for(total_len)
         if self.need.window is None:
             return full
         # live span while a step of `max_step_tokens` runs: window - 1 earlier keys + the step's tokens
-        return min(full, self.pages_for(self.need.window - 1 + max_step_tokens) + 1)
+        return min(full, self.pages_for(self.need.window - 1 + max_step_tokens) + 1 + self.kept_pages)
 
 
 @dataclass
@@ -269,7 +282,7 @@ class CacheManager:
                 if g.need.window is not None:
                     # pages the window has passed go back first; a request with a reservation may claim them again
                     oldest_needed = max(0, rc.length - g.need.window + 1)
-                    given_back = max(0, min(oldest_needed // g.page_size, have) - int(g.first_page[rc.row]))
+                    given_back = max(0, min(oldest_needed // g.page_size, have) - max(int(g.first_page[rc.row]), g.kept_pages))
                     if gi in rc.reserved:
                         reserved += given_back
                     else:
@@ -289,7 +302,7 @@ class CacheManager:
         g = self.groups[gi]
         oldest_needed = max(0, first_query_pos - g.need.window + 1)
         keep_from = min(oldest_needed // g.page_size, int(g.num_pages_of[rc.row]))
-        lo = int(g.first_page[rc.row])
+        lo = max(int(g.first_page[rc.row]), g.kept_pages)
         if keep_from > lo:
             pages = [int(p) for p in g.block_table[rc.row, lo:keep_from]]
             self._free_pages(gi, pages)
@@ -312,8 +325,7 @@ class CacheManager:
         if self.live.get(rc.row) is not rc:
             raise ValueError(f"request row {rc.row} released twice (or never admitted)")
         for gi, g in enumerate(self.groups):
-            lo, hi = int(g.first_page[rc.row]), int(g.num_pages_of[rc.row])
-            self._free_pages(gi, [int(p) for p in g.block_table[rc.row, lo:hi]])
+            self._free_pages(gi, [int(p) for lo, hi in g.held(rc.row) for p in g.block_table[rc.row, lo:hi]])
             g.block_table[rc.row, :] = -1
             g.first_page[rc.row] = 0
             g.num_pages_of[rc.row] = 0
@@ -348,15 +360,18 @@ class CacheManager:
             g.pool.check()
             seen: set[int] = set()
             for row, rc in self.live.items():
-                lo, hi = int(g.first_page[row]), int(g.num_pages_of[row])
-                pages = [int(p) for p in g.block_table[row, lo:hi]]
+                ranges = g.held(row)
+                pages = [int(p) for lo, hi in ranges for p in g.block_table[row, lo:hi]]
                 for p in pages:
                     if p < 0 or not g.pool.is_held(p):
                         raise AssertionError(f"group {gi}: row {row} lists page {p} that it does not hold")
                     if p in seen:
                         raise AssertionError(f"group {gi}: page {p} is held twice")
                     seen.add(p)
-                if (g.block_table[row, :lo] != -1).any() or (g.block_table[row, hi:] != -1).any():
+                outside = np.ones(g.block_table.shape[1], dtype=bool)
+                for lo, hi in ranges:
+                    outside[lo:hi] = False
+                if (g.block_table[row][outside] != -1).any():
                     raise AssertionError(f"group {gi}: row {row} has entries outside its live pages")
             if len(seen) != g.pool.num_held:
                 raise AssertionError(f"group {gi}: {g.pool.num_held - len(seen)} pages are held by nobody")

@@ -8,6 +8,7 @@ from .kuvazen import KuvazenConfig
 from .pupopel import PupopelConfig
 from .zarisun import ZarisunConfig
 from .dimudra import DimudraConfig
+from .fosupel import FosupelConfig
 
 __all__ = [
     "ConfigError", "architecture_of", "load_model_config", "make_model_config", "read_config_json", "require",
@@ -15,4 +16,5 @@ __all__ = [
     "RopeSpec", "ScheduleEntry", "FalconH1Config", "DuduraxConfig", "DenseMLPSpec", "GLASpec", "LatentAttentionSpec",
     "PostNormBlockSpec", "RoutedMLPSpec", "KuvazenConfig", "ClampedGLUSpec", "MinGRUSpec", "PooledWindowAttentionSpec",
     "StreamBlockSpec", "TokenSideSpec", "PupopelConfig", "ZarisunConfig", "DimudraConfig",
+    "FosupelConfig",
 ]

@@ -125,13 +125,14 @@ class LatentAttentionSpec:
     pairing: str = "halves"         # the rotation pairs column i with i + n/2 ("halves") or 2i with 2i + 1 ("neighbours")
     sink: bool = False              # a stored number per head joins the softmax's denominator as exp(sink_h)
     head_gate: bool = False         # a head's output is multiplied by sigmoid of a projection of the input, one number per head
+    column_gate: bool = False       # the same with one number per output column of every head
     own_latents: bool = True        # False: no down-projection; the layer reads the latents another layer cached
                                     # (the schedule gives it that layer's cache, `writes_cache=False`)
 
 
 @dataclass(frozen=True)
 class DenseMLPSpec:
-    """down(act(up(x))), no gate."""
+    """down(act(up(x))), no gate.  `activation`: "gelu_tanh", or "xielu" with two stored numbers."""
     hidden_size: int
     intermediate_size: int
     activation: str = "gelu_tanh"
@@ -286,6 +287,39 @@ class LightningAttentionSpec:
 
 
 @dataclass(frozen=True)
+class RetentionSpec:
+    """Linear attention over rotated queries and keys with one fixed decay per head: k times key_dim^-1/2 after the rotation (in
+    halves); S <- decay_h S + k v^T, o = S^T q; each head's o over its root mean square (no weight), times silu(gate projection),
+    then the output projection."""
+    hidden_size: int
+    num_heads: int
+    key_dim: int
+    value_dim: int
+    decay: tuple[float, ...]
+    norm_eps: float
+    position: RopeSpec | None = None
+    kind: str = "retention"
+
+
+@dataclass(frozen=True)
+class TalkingAttentionSpec:
+    """Grouped-query attention whose heads mix their softmax weights by a stored matrix before they are applied to the values:
+    rotation in halves; scores times `softmax_scale`; position i sees j <= i with i - j < window (None: every j <= i) or
+    j < keep_first; with `sink` a stored number per head joins the softmax's denominator (and is not mixed)."""
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    value_dim: int
+    softmax_scale: float
+    window: int | None = None
+    keep_first: int = 0
+    position: RopeSpec | None = None
+    sink: bool = True
+    kind: str = "talking_attention"
+
+
+@dataclass(frozen=True)
 class MixerPairSpec:
     """Two mixers side by side on the same input; the result is the sum of their outputs, each times its slot's
     `out_scale`.  At most one of them keeps keys and values."""
@@ -309,6 +343,7 @@ class GatedAttentionSpec:
     norm_eps: float
     window: int | None = None
     position: RopeSpec | None = None
+    keep_first: int = 0                 # the sequence's first so many tokens stay visible behind the window
     proj_bias: bool = False
     qk_norm: str = "none"
     sink_zero: bool = False
@@ -440,8 +475,9 @@ class OutNormBlockSpec:
 @dataclass(frozen=True)
 class StreamBlockSpec:
     """Pre-norm block on a 32-bit stream: x <- x + s1 * mixer(norm(x)); with a feed-forward x <- x + s2 * ff(norm(x))
-    (s1, s2: a stored scale per channel, when `layer_scale`); then, with `side`, the token's side input.  `input_conv` > 0: the
-    mixer reads h + conv(h) instead of the normed rows h, conv a causal convolution per channel of so many taps."""
+    (s1, s2: a stored scale per channel, when `layer_scale`, else both the number `residual_scale`); then, with `side`, the
+    token's side input.  `input_conv` > 0: the mixer reads h + conv(h) instead of the normed rows h, conv a causal convolution
+    per channel of so many taps."""
     prefix: str
     mixer: MixerSlot
     mixer_norm: NormSpec
@@ -456,6 +492,7 @@ class StreamBlockSpec:
     side_name: str = "side."
     input_conv: int = 0
     input_conv_name: str = "canon1"
+    residual_scale: float = 1.0
     kind: str = "prenorm_stream"
 
 
@@ -489,6 +526,16 @@ class StreamAddSpec:
 
 
 @dataclass(frozen=True)
+class StreamVectorSpec:
+    """x <- x + b_k on a 32-bit stream, the same vector for every row: row k of a table [count, width] stored at the model's root
+    under `name`, k the schedule entry's `turn`."""
+    hidden_size: int
+    name: str
+    count: int
+    kind: str = "vector"
+
+
+@dataclass(frozen=True)
 class ScheduleEntry:
     """One execution of a layer.  `layer` indexes `ModelSpec.layers` (a layer
     may appear in several entries: its weights then run more than once).
@@ -499,6 +546,7 @@ class ScheduleEntry:
     cache: int
     writes_cache: bool = True
     opens: int | None = None      # index into `ModelSpec.stream_inputs`: that input is applied right before this execution
+    turn: int = 0                 # the number of the pass that opens here, for an input that differs from pass to pass
 
 
 @dataclass(frozen=True)
@@ -518,6 +566,7 @@ class ModelSpec:
     lm_head_kind: str = "lm_head"           # registry.HEADS: built as cls(vocab_size, hidden_size, multiplier, tied_to)
     embedding_options: tuple[tuple[str, Any], ...] = ()    # further keyword arguments of the embedding's constructor
     stream_inputs: tuple[StreamInputSpec, ...] = ()         # see `ScheduleEntry.opens`
+    lm_head_options: tuple[tuple[str, Any], ...] = ()      # further keyword arguments of the head's constructor
 
     def resolved_schedule(self) -> tuple[ScheduleEntry, ...]:
         if self.schedule:

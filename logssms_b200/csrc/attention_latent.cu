@@ -7,7 +7,8 @@
 //
 //  latent_prepare   : per token: RMSNorm of the first `rank` columns of the down-projection -> cache "c";
 //                     rotation of its last `rot` columns -> cache "kr"; rotation of every head's query part, in place
-//  heads_matmul     : out[t, h, n] = sum_k a[t, h, k] * w[h, k, n]     (32-bit accumulation)
+//  heads_matmul     : out[t, h, n] = sum_k a[t, h, k] * w[h, k, n]     (32-bit accumulation), with gate logits
+//                     times sigmoid(g[t, h, n])
 //  latent_attention : softmax attention of listed tokens over their request's pages, keys j with
 //                     0 <= p - j < window (window 0: all earlier keys).  One warp per (token, head); the warps of a
 //                     CTA are heads of one token and share its key tiles in shared memory; scores, softmax weights
@@ -82,7 +83,8 @@ extern "C" int lb_latent_prepare(void* proj, long row_stride, int q_cols, int H,
 constexpr int kHmTokens = 8;
 template <typename T>
 __global__ void __launch_bounds__(128) heads_matmul_kernel(const T* __restrict__ a, long a_row, long a_head, const T* __restrict__ w,
-                                                           T* __restrict__ out, long o_row, long o_head, int tokens, int K, int N) {
+                                                           T* __restrict__ out, long o_row, long o_head, int tokens, int K, int N,
+                                                           const T* __restrict__ gate, long g_row) {
     extern __shared__ float as[];                    // [kHmTokens][K], then [4][kHmTokens][32] partial sums
     float* part = as + kHmTokens * K;
     const int h = blockIdx.y, t0 = blockIdx.z * kHmTokens;
@@ -112,15 +114,16 @@ __global__ void __launch_bounds__(128) heads_matmul_kernel(const T* __restrict__
     for (int i = threadIdx.x; i < nt * 32; i += blockDim.x) {
         const int tt = i >> 5, c = i & 31, nn = blockIdx.x * 32 + c;
         if (nn < N) {
-            const float sum = (part[tt * 32 + c] + part[(kHmTokens + tt) * 32 + c])
-                            + (part[(2 * kHmTokens + tt) * 32 + c] + part[(3 * kHmTokens + tt) * 32 + c]);
+            float sum = (part[tt * 32 + c] + part[(kHmTokens + tt) * 32 + c])
+                      + (part[(2 * kHmTokens + tt) * 32 + c] + part[(3 * kHmTokens + tt) * 32 + c]);
+            if (gate != nullptr) sum *= 1.f / (1.f + expf(-to_f32(gate[(size_t)(t0 + tt) * g_row + (size_t)h * N + nn])));
             out[(size_t)(t0 + tt) * o_row + (size_t)h * o_head + nn] = from_f32<T>(sum);
         }
     }
 }
 
 extern "C" int lb_heads_matmul(const void* a, long a_row, long a_head, const void* w, void* out, long o_row, long o_head,
-                               int tokens, int H, int K, int N, int dtype, void* stream) {
+                               int tokens, int H, int K, int N, const void* gate, long g_row, int dtype, void* stream) {
     if (tokens <= 0) return kOk;
     if (H <= 0 || K <= 0 || N <= 0) return kBadSize;
     const size_t smem = ((size_t)kHmTokens * K + 4 * kHmTokens * 32) * sizeof(float);
@@ -130,8 +133,32 @@ extern "C" int lb_heads_matmul(const void* a, long a_row, long a_head, const voi
         static size_t have = 0;
         ensure_dynamic_smem(heads_matmul_kernel<T>, smem, have);
         heads_matmul_kernel<T><<<grid, 128, smem, (cudaStream_t)stream>>>((const T*)a, a_row, a_head, (const T*)w, (T*)out,
-                                                                         o_row, o_head, tokens, K, N);
+                                                                         o_row, o_head, tokens, K, N, (const T*)gate, g_row);
     });
+    return launch_status();
+}
+
+// out[t, h, n] = a[t, h, n] * sigmoid(g[t, h * N + n]), two neighbouring columns per thread: the gate of a product that the library
+// made (its rows may lie head by head)
+__global__ void column_gate_kernel(const __nv_bfloat16* __restrict__ a, long a_row, long a_head, const __nv_bfloat16* __restrict__ gate,
+                                   long g_row, __nv_bfloat16* __restrict__ out, int width, int N, size_t total) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= total) return;
+    const size_t t = i / (width / 2);
+    const int c = (int)(i % (width / 2)) * 2, h = c / N;
+    const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(a + t * a_row + (size_t)h * a_head + (c - h * N)));
+    const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gate + t * g_row + c));
+    *reinterpret_cast<__nv_bfloat162*>(out + t * width + c) = __floats2bfloat162_rn(v.x / (1.f + expf(-g.x)), v.y / (1.f + expf(-g.y)));
+}
+
+// bfloat16; N even, even strides; out: contiguous [tokens, H * N]
+extern "C" int lb_column_gate(const void* a, long a_row, long a_head, const void* gate, long g_row, void* out, int tokens, int H, int N,
+                              void* stream) {
+    if (tokens <= 0) return kOk;
+    if (H <= 0 || N <= 0 || N % 2 || a_row % 2 || a_head % 2 || g_row % 2 || (((uintptr_t)a | (uintptr_t)gate | (uintptr_t)out) & 3)) return kBadSize;
+    const size_t total = (size_t)tokens * H * (N / 2);
+    column_gate_kernel<<<(unsigned)((total + 255) / 256), 256, 0, (cudaStream_t)stream>>>(
+        (const __nv_bfloat16*)a, a_row, a_head, (const __nv_bfloat16*)gate, g_row, (__nv_bfloat16*)out, H * N, N, total);
     return launch_status();
 }
 

@@ -16,6 +16,7 @@
 //   score of token j.  `sinks` (a number per query head): exp(sink_h) joins the softmax's denominator, with no key and no
 //   value.  Without rotation tables (`v_rot` = 0) values are summed as they are cached.  `gate` (a row of logits per token,
 //   one per output column): every output column is multiplied by sigmoid of its logit before it is rounded and stored.
+//   `keep` (with `pool` = 0): the sequence's first `keep` tokens stay visible behind the window, at their true positions.
 //
 //   pooled_prepare : per (token, head): rotate the query; rotate key and value and store them at the token's slot
 //   normed_prepare : per (token, head): RMS-norm the query and the key over the head's columns with a weight each
@@ -30,6 +31,9 @@
 //   pooled_attention_tile : bfloat16 prompt portions on the tensor cores: a CTA per (run of up to 64 neighbouring tokens
 //                           of a request, query head); the keys the run sees go through shared memory once for all
 //                           its queries (described at the kernel)
+//   talk_merge            : attention whose heads mix their softmax weights before they are applied to the values: the two
+//                           kernels above sum every head's weights over ALL key/value heads' values, and this one mixes
+//                           (described at the kernel)
 #include "lb200/common.cuh"
 using namespace lb200;
 
@@ -205,9 +209,10 @@ __device__ __forceinline__ long key_row(int kk, int blocks, int first, const int
     return page < 0 ? -1 : (long)page * page_size + e % page_size;
 }
 
-// blocks that lie wholly behind the window of position i (none without pooling)
-__device__ __forceinline__ int blocks_behind(int i, int window, int pool) {
-    return pool > 0 ? max(0, (i - window + 1) / pool) : 0;
+// what lies behind the window of position i and is seen all the same: blocks that are wholly behind it, or (without pooling)
+// the `keep` first tokens
+__device__ __forceinline__ int leading_keys(int i, int window, int pool, int keep) {
+    return pool > 0 ? max(0, (i - window + 1) / pool) : min(keep, max(0, i - window + 1));
 }
 
 // what the options add to an attention: a slope per head on the distance to a token, a sink per head in the denominator, a
@@ -217,6 +222,14 @@ struct ScoreExtras {
     const float* sinks;       // [Hq] or null
     const void* gate;         // [tokens, Hq * vdim] view of logits in the activation dtype, or null
     long gate_stride;
+    int keep;                 // first tokens that stay visible behind the window (0 with pooled blocks)
+};
+
+// Value columns of a CTA where every head's weights are summed over the values of ALL key/value heads (`width` = Hkv * their
+// size; the value rows of a token lie side by side in the cache): chunks of columns, a CTA each.  width 0: the columns of the
+// head's own key/value head.  A partial result is `stride` floats: maximum and sum first, the columns from `off` on.
+struct ValueSpan {
+    int width, stride, off;
 };
 
 template <typename T>
@@ -253,7 +266,7 @@ __global__ void __launch_bounds__(kWarps * 32) pooled_attention_kernel(
     const int* pages = block_table + (size_t)token_req[t] * table_width;
     const int* pooled_pages = pooled_table + (size_t)token_req[t] * pooled_width;
     const int first = max(0, pos - window + 1);
-    const int blocks = blocks_behind(pos, window, pool);
+    const int blocks = leading_keys(pos, window, pool, extras.keep);
     const int keys = blocks + (pos - first + 1);
     const float slope = extras.slopes != nullptr ? extras.slopes[head] : 0.f;
     float m = -INFINITY, l = 0.f, acc[kMaxValueRegs];
@@ -274,6 +287,7 @@ __global__ void __launch_bounds__(kWarps * 32) pooled_attention_kernel(
                 if (c < dim) a0 += qs[c] * to_f32(kr[c]);
                 s = a0 + a1;
                 if (!pooled) s -= slope * (float)(pos - (first + kk - blocks));
+                else if (extras.keep > 0) s -= slope * (float)(pos - kk);
             }
         }
         const float m_new = fmaxf(m, warp_max(s));
@@ -330,17 +344,18 @@ extern "C" int lb_pooled_attention(const void* q, const void* k_cache, const voi
                                    int pooled_width, const int* token_req, const int* positions, const int* token_list,
                                    int num_tokens, const float* v_table, int v_rot, int table_rows, void* out, int Hq, int Hkv,
                                    int dim, int vdim, int page_size, float scale, int window, int pool, const float* slopes,
-                                   const float* sinks, const void* gate, long gate_stride, int dtype, void* stream) {
+                                   const float* sinks, const void* gate, long gate_stride, int keep, int dtype, void* stream) {
     if (num_tokens <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || dim <= 0 || vdim <= 0 || page_size <= 0 || window <= 0 || pool < 0 || (v_rot & 1)
-        || v_rot > vdim || table_rows <= 0)
+        || v_rot > vdim || table_rows <= 0 || keep < 0 || (keep > 0 && pool > 0))
         return kBadSize;
+    if (keep > 0) { kp_cache = k_cache; vp_cache = v_cache; pooled_table = block_table; pooled_width = table_width; }
     if (vdim > 32 * kMaxValueRegs || (size_t)kWarps * dim * sizeof(float) > 48 * 1024) return kTooLarge;
     dim3 grid(num_tokens, (Hq + kWarps - 1) / kWarps);
     LB_DISPATCH_DTYPE(dtype, pooled_attention_kernel<T><<<grid, kWarps * 32, (size_t)kWarps * dim * sizeof(float), (cudaStream_t)stream>>>(
         (const T*)q, (const T*)k_cache, (const T*)v_cache, (const T*)kp_cache, (const T*)vp_cache, block_table, table_width,
         pooled_table, pooled_width, token_req, positions, token_list, v_table, v_rot, table_rows, (T*)out, Hq, Hkv, dim, vdim,
-        page_size, scale, window, pool, ScoreExtras{slopes, sinks, gate, gate_stride}));
+        page_size, scale, window, pool, ScoreExtras{slopes, sinks, gate, gate_stride, keep}));
     return launch_status();
 }
 
@@ -351,7 +366,7 @@ extern "C" int lb_pooled_attention(const void* q, const void* k_cache, const voi
 // the warp's 32 keys.  The four warps' partial (maximum, sum, weighted values) meet in shared memory and go to a
 // scratch buffer; `pooled_merge` joins the ranges, divides, turns the values back and stores.  All float32.
 constexpr int kSplitWarps = 4;
-constexpr int kSplitValueRegs = 4;        // value columns per lane: vdim <= 128
+constexpr int kSplitValueRegs = 4;        // value columns per lane: vdim <= 128 (the mixed form takes up to four times as many)
 
 template <typename T, int kPer>
 __device__ __forceinline__ void score_row(const T* __restrict__ kr, const float* __restrict__ qs, int dim, float (&s)[kPer]) {
@@ -377,22 +392,26 @@ __device__ __forceinline__ void score_row_vec(const __nv_bfloat16* __restrict__ 
     }
 }
 
-// grid (tokens, Hkv * ceil(per / kPer), splits); dynamic shared memory: kPer * dim floats (queries) + the warps' partial results
-// partial: float [tokens, Hq, splits, vdim + 2] (maximum, sum, weighted values)
-template <typename T, int kPer>
+// grid (tokens, chunks * Hkv * ceil(per / kPer), splits); dynamic shared memory: kPer * dim floats (queries) + the warps' partial
+// results; partial: float [tokens, Hq, splits, span.stride] (maximum, sum, weighted values).  `vdim`: the most value columns of a
+// CTA, kValueRegs per lane.
+template <typename T, int kPer, int kValueRegs>
 __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kernel(
         const T* __restrict__ q, const T* __restrict__ k_cache, const T* __restrict__ v_cache, const T* __restrict__ kp_cache,
         const T* __restrict__ vp_cache, const int* __restrict__ block_table, int table_width, const int* __restrict__ pooled_table,
         int pooled_width, const int* __restrict__ token_req, const int* __restrict__ positions, const int* __restrict__ token_list,
         float* __restrict__ partial, int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool, int splits,
-        ScoreExtras extras) {
+        ScoreExtras extras, ValueSpan span) {
     extern __shared__ __align__(16) float split_smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int slot = blockIdx.x;                                   // row of the scratch buffer
     const int t = token_list != nullptr ? token_list[slot] : slot;
     if (t < 0) return;
     const int per = Hq / Hkv, groups = (per + kPer - 1) / kPer;
-    const int g = blockIdx.y / groups, h0 = g * per + (blockIdx.y % groups) * kPer;
+    const int g = (blockIdx.y / groups) % Hkv, h0 = g * per + (blockIdx.y % groups) * kPer;
+    const int v_row = span.width > 0 ? span.width : Hkv * vdim;    // value elements of a token
+    const int v_col = span.width > 0 ? (blockIdx.y / (groups * Hkv)) * vdim : g * vdim;
+    const int cols = span.width > 0 ? min(vdim, span.width - v_col) : vdim;
     const int nh = min(kPer, g * per + per - h0);                  // query heads of this CTA
     const int split = blockIdx.z;
     float* qs = split_smem;                                        // [kPer][dim]
@@ -406,7 +425,7 @@ __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kerne
     const int* pages = block_table + (size_t)token_req[t] * table_width;
     const int* pooled_pages = pooled_table + (size_t)token_req[t] * pooled_width;
     const int first = max(0, pos - window + 1);
-    const int blocks = blocks_behind(pos, window, pool);
+    const int blocks = leading_keys(pos, window, pool, extras.keep);
     const int keys = blocks + (pos - first + 1);
     float slope[kPer];
 #pragma unroll
@@ -414,12 +433,12 @@ __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kerne
     const int chunk = ((keys + splits - 1) / splits + 31) / 32 * 32;
     const int k_begin = split * chunk, k_end = min(keys, k_begin + chunk);
     const bool vec = sizeof(T) == 2 && dim % 8 == 0;
-    float m[kPer], l[kPer], acc[kPer][kSplitValueRegs];
+    float m[kPer], l[kPer], acc[kPer][kValueRegs];
 #pragma unroll
     for (int h = 0; h < kPer; ++h) {
         m[h] = -INFINITY; l[h] = 0.f;
 #pragma unroll
-        for (int r = 0; r < kSplitValueRegs; ++r) acc[h][r] = 0.f;
+        for (int r = 0; r < kValueRegs; ++r) acc[h][r] = 0.f;
     }
     for (int k0 = k_begin + warp * 32; k0 < k_end; k0 += kSplitWarps * 32) {
         const int kk = k0 + lane;
@@ -433,8 +452,8 @@ __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kerne
             const T* kr = (pooled ? kp_cache : k_cache) + ((size_t)row * Hkv + g) * dim;
             if (vec) score_row_vec<kPer>(reinterpret_cast<const __nv_bfloat16*>(kr), qs, dim, s);
             else score_row<T, kPer>(kr, qs, dim, s);
-            if (!pooled) {
-                const float dist = (float)(pos - (first + kk - blocks));
+            if (!pooled || extras.keep > 0) {
+                const float dist = (float)(pos - (pooled ? kk : first + kk - blocks));
 #pragma unroll
                 for (int h = 0; h < kPer; ++h) s[h] -= slope[h] * dist;
             }
@@ -449,21 +468,21 @@ __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kerne
             l[h] = l[h] * corr + warp_sum(p[h]);
             m[h] = m_new;
 #pragma unroll
-            for (int r = 0; r < kSplitValueRegs; ++r) acc[h][r] *= corr;
+            for (int r = 0; r < kValueRegs; ++r) acc[h][r] *= corr;
         }
         const int n = min(32, k_end - k0);
         for (int j = 0; j < n; ++j) {
             const long rj = __shfl_sync(0xffffffffu, row, j);
             if (rj < 0) continue;
-            const T* vr = ((k0 + j) < blocks ? vp_cache : v_cache) + ((size_t)rj * Hkv + g) * vdim;
-            float vv[kSplitValueRegs];
+            const T* vr = ((k0 + j) < blocks ? vp_cache : v_cache) + (size_t)rj * v_row + v_col;
+            float vv[kValueRegs];
 #pragma unroll
-            for (int r = 0; r < kSplitValueRegs; ++r) { const int c = lane + 32 * r; vv[r] = c < vdim ? to_f32(vr[c]) : 0.f; }
+            for (int r = 0; r < kValueRegs; ++r) { const int c = lane + 32 * r; vv[r] = c < cols ? to_f32(vr[c]) : 0.f; }
 #pragma unroll
             for (int h = 0; h < kPer; ++h) {
                 const float pj = __shfl_sync(0xffffffffu, p[h], j);
 #pragma unroll
-                for (int r = 0; r < kSplitValueRegs; ++r) acc[h][r] += pj * vv[r];
+                for (int r = 0; r < kValueRegs; ++r) acc[h][r] += pj * vv[r];
             }
         }
     }
@@ -474,26 +493,27 @@ __global__ void __launch_bounds__(kSplitWarps * 32) pooled_attention_split_kerne
         float* dst = part + ((size_t)warp * kPer + h) * stride;
         if (lane == 0) { dst[0] = m[h]; dst[1] = l[h]; }
 #pragma unroll
-        for (int r = 0; r < kSplitValueRegs; ++r) { const int c = lane + 32 * r; if (c < vdim) dst[2 + c] = acc[h][r]; }
+        for (int r = 0; r < kValueRegs; ++r) { const int c = lane + 32 * r; if (c < cols) dst[2 + c] = acc[h][r]; }
     }
     __syncthreads();
     for (int h = warp; h < nh; h += kSplitWarps) {
         float mm = -INFINITY;
         for (int w = 0; w < kSplitWarps; ++w) mm = fmaxf(mm, part[((size_t)w * kPer + h) * stride]);
-        float ll = 0.f, o[kSplitValueRegs];
+        float ll = 0.f, o[kValueRegs];
 #pragma unroll
-        for (int r = 0; r < kSplitValueRegs; ++r) o[r] = 0.f;
+        for (int r = 0; r < kValueRegs; ++r) o[r] = 0.f;
         for (int w = 0; w < kSplitWarps; ++w) {
             const float* src = part + ((size_t)w * kPer + h) * stride;
             const float f = (src[0] == -INFINITY) ? 0.f : expf(src[0] - mm);
             ll += f * src[1];
 #pragma unroll
-            for (int r = 0; r < kSplitValueRegs; ++r) { const int c = lane + 32 * r; if (c < vdim) o[r] += f * src[2 + c]; }
+            for (int r = 0; r < kValueRegs; ++r) { const int c = lane + 32 * r; if (c < cols) o[r] += f * src[2 + c]; }
         }
-        float* dst = partial + (((size_t)slot * Hq + h0 + h) * splits + split) * stride;
-        if (lane == 0) { dst[0] = mm; dst[1] = ll; }
+        float* dst = partial + (((size_t)slot * Hq + h0 + h) * splits + split) * span.stride;
+        if (lane == 0 && (span.width == 0 || v_col == 0)) { dst[0] = mm; dst[1] = ll; }
+        dst += span.off + (span.width > 0 ? v_col : 0);
 #pragma unroll
-        for (int r = 0; r < kSplitValueRegs; ++r) { const int c = lane + 32 * r; if (c < vdim) dst[2 + c] = o[r]; }
+        for (int r = 0; r < kValueRegs; ++r) { const int c = lane + 32 * r; if (c < cols) dst[c] = o[r]; }
     }
 }
 
@@ -542,20 +562,20 @@ __global__ void __launch_bounds__(32) pooled_merge_kernel(const float* __restric
     }
 }
 
-template <typename T, int kPer>
+template <typename T, int kPer, int kValueRegs>
 static int launch_split(const void* q, const void* k_cache, const void* v_cache, const void* kp_cache, const void* vp_cache,
                         const int* block_table, int table_width, const int* pooled_table, int pooled_width, const int* token_req,
                         const int* positions, const int* token_list, int num_tokens, float* partial, int Hq, int Hkv, int dim, int vdim,
-                        int page_size, float scale, int window, int pool, int splits, ScoreExtras extras, void* stream) {
+                        int page_size, float scale, int window, int pool, int splits, ScoreExtras extras, ValueSpan span, void* stream) {
     const size_t smem = ((size_t)kPer * dim + (size_t)kSplitWarps * kPer * (vdim + 2)) * sizeof(float);
     static size_t have = 0;
-    ensure_dynamic_smem(pooled_attention_split_kernel<T, kPer>, smem, have);
-    const int per = Hq / Hkv;
-    dim3 grid(num_tokens, Hkv * ((per + kPer - 1) / kPer), splits);
-    pooled_attention_split_kernel<T, kPer><<<grid, kSplitWarps * 32, smem, (cudaStream_t)stream>>>(
+    ensure_dynamic_smem(pooled_attention_split_kernel<T, kPer, kValueRegs>, smem, have);
+    const int per = Hq / Hkv, chunks = span.width > 0 ? (span.width + vdim - 1) / vdim : 1;
+    dim3 grid(num_tokens, chunks * Hkv * ((per + kPer - 1) / kPer), splits);
+    pooled_attention_split_kernel<T, kPer, kValueRegs><<<grid, kSplitWarps * 32, smem, (cudaStream_t)stream>>>(
         (const T*)q, (const T*)k_cache, (const T*)v_cache, (const T*)kp_cache, (const T*)vp_cache, block_table, table_width,
         pooled_table, pooled_width, token_req, positions, token_list, partial, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits,
-        extras);
+        extras, span);
     return launch_status();
 }
 
@@ -566,24 +586,25 @@ extern "C" int lb_pooled_attention_split(const void* q, const void* k_cache, con
                                          int num_tokens, const float* v_table, int v_rot, int table_rows, float* partial, void* out,
                                          int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
                                          int splits, const float* slopes, const float* sinks, const void* gate, long gate_stride,
-                                         int dtype, void* stream) {
+                                         int keep, int dtype, void* stream) {
     if (num_tokens <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || dim <= 0 || dim % 4 || vdim <= 0 || page_size <= 0 || window <= 0 || pool < 0 || (v_rot & 1)
-        || v_rot > vdim || table_rows <= 0 || splits <= 0 || splits > 65535 || Hq > 65535)
+        || v_rot > vdim || table_rows <= 0 || splits <= 0 || splits > 65535 || Hq > 65535 || keep < 0 || (keep > 0 && pool > 0))
         return kBadSize;
     if (vdim > 32 * kSplitValueRegs || dim > 1024) return kTooLarge;
+    if (keep > 0) { kp_cache = k_cache; vp_cache = v_cache; pooled_table = block_table; pooled_width = table_width; }
     const int per = Hq / Hkv;
     int code;
-#define LB_SPLIT(PER) LB_DISPATCH_DTYPE(dtype, code = (launch_split<T, PER>(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, \
+#define LB_SPLIT(PER) LB_DISPATCH_DTYPE(dtype, code = (launch_split<T, PER, kSplitValueRegs>(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, \
         pooled_table, pooled_width, token_req, positions, token_list, num_tokens, partial, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits, \
-        ScoreExtras{slopes, nullptr, nullptr, 0}, stream)))
+        ScoreExtras{slopes, nullptr, nullptr, 0, keep}, ValueSpan{0, vdim + 2, 2}, stream)))
     if (per == 1) { LB_SPLIT(1); } else if (per == 2) { LB_SPLIT(2); } else { LB_SPLIT(4); }
 #undef LB_SPLIT
     if (code != 0) return code;
     dim3 grid(num_tokens, Hq);
     LB_DISPATCH_DTYPE(dtype, pooled_merge_kernel<T><<<grid, 32, 0, (cudaStream_t)stream>>>(partial, positions, token_list, v_table, v_rot,
                                                                                            table_rows, (T*)out, Hq, vdim, splits,
-                                                                                           ScoreExtras{nullptr, sinks, gate, gate_stride}));
+                                                                                           ScoreExtras{nullptr, sinks, gate, gate_stride, 0}));
     return launch_status();
 }
 
@@ -614,17 +635,22 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         int table_width, const int* __restrict__ pooled_table, int pooled_width, const int* __restrict__ cu,
         const int* __restrict__ start_pos, const int* __restrict__ tiles, const float* __restrict__ v_table, int v_rot,
         int table_rows, __nv_bfloat16* __restrict__ out, int Hq, int Hkv, int dim, int vdim, int page_size, float scale,
-        int window, int pool, float* __restrict__ partial, int splits, ScoreExtras extras) {
+        int window, int pool, float* __restrict__ partial, int splits, ScoreExtras extras, ValueSpan span) {
     extern __shared__ __align__(16) unsigned char tile_smem[];
     const int b = tiles[2 * blockIdx.x];
     if (b < 0) return;
     const int t0 = tiles[2 * blockIdx.x + 1];
-    const int head = blockIdx.y, g = head / (Hq / Hkv);
+    const int head = blockIdx.y % Hq, g = head / (Hq / Hkv);
+    const int v_row = span.width > 0 ? span.width : Hkv * vdim;     // value elements of a token
+    const int v_col = span.width > 0 ? (blockIdx.y / Hq) * vdim : g * vdim;
+    const int cols = span.width > 0 ? min(vdim, span.width - v_col) : vdim;
+    const int keep = extras.keep;
     const int n_q = min(kTileQ, cu[b + 1] - cu[b] - t0);
     const int row0 = cu[b] + t0, pos0 = start_pos[b] + t0;
     const int i_last = pos0 + n_q - 1;
     const int first = max(0, pos0 - window + 1);                    // the oldest token any query of the run sees
-    const int blocks = blocks_behind(i_last, window, pool);         // the blocks the last query sees
+    // the blocks the last query sees, or the kept tokens that lie behind every query's window
+    const int blocks = leading_keys(pool > 0 ? i_last : pos0, window, pool, keep);
     const float slope = extras.slopes != nullptr ? extras.slopes[head] : 0.f;
     const int keys = blocks + (i_last - first + 1);
     const int k_stride = dim + 8, v_stride = vdim + 8;              // elements; the pad staggers the banks
@@ -632,7 +658,7 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
     __nv_bfloat16* Ks0 = reinterpret_cast<__nv_bfloat16*>(tile_smem);
     __nv_bfloat16* Vs0 = Ks0 + 2 * kTileK * k_stride;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gq = lane >> 2, tq = lane & 3;
-    const int dsteps = dim / 16, vtiles = vdim / 8;
+    const int dsteps = dim / 16, vtiles = cols / 8;
     const int* pages = block_table + (size_t)b * table_width;
     const int* pooled_pages = pooled_table + (size_t)b * pooled_width;
 
@@ -658,10 +684,10 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
             }
         }
     }
-    const int nb_lo = blocks_behind(i_lo, window, pool), nb_hi = blocks_behind(i_hi, window, pool);
+    const int nb_lo = pool > 0 ? leading_keys(i_lo, window, pool, 0) : blocks, nb_hi = pool > 0 ? leading_keys(i_hi, window, pool, 0) : blocks;
     // what the warp's 16 rows can see at all: a chunk wholly outside is skipped
     const int iw0 = pos0 + warp * 16, iw1 = min(iw0 + 15, i_last);
-    const int nb_warp = blocks_behind(iw1, window, pool);
+    const int nb_warp = pool > 0 ? leading_keys(iw1, window, pool, 0) : blocks;
     float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
     float o[kValueTiles][4];
 #pragma unroll
@@ -676,9 +702,9 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         long row = -1;
         bool pooled = false;
         if (kk < keys) row = key_row(kk, blocks, first, pages, pooled_pages, page_size, pooled);
-        const int n = is_v ? vdim : dim;
+        const int n = is_v ? cols : dim;
         const __nv_bfloat16* src = is_v ? (pooled ? vp_cache : v_cache) : (pooled ? kp_cache : k_cache);
-        if (row >= 0) src += ((size_t)row * Hkv + g) * n;
+        if (row >= 0) src += is_v ? (size_t)row * v_row + v_col : ((size_t)row * Hkv + g) * dim;
         __nv_bfloat16* dst = is_v ? Vs0 + ((size_t)buf * kTileK + r) * v_stride : Ks0 + ((size_t)buf * kTileK + r) * k_stride;
         const uint32_t dst_addr = (uint32_t)__cvta_generic_to_shared(dst);
         const int bytes = row >= 0 ? 16 : 0;
@@ -704,7 +730,7 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
             if (k0 < blocks && k0 < nb_warp) any = true;
             if (c_last >= blocks) {
                 const int ja = first + max(k0, blocks) - blocks, jb = first + c_last - blocks;
-                if (jb > iw0 - window && ja <= iw1) any = true;
+                if ((jb > iw0 - window || ja < keep) && ja <= iw1) any = true;
             }
             if (!any || iw0 > i_last) continue;
         }
@@ -731,8 +757,8 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
                 bool seen = kk < keys && (hi ? r_hi : r_lo) < n_q;
                 float bias = 0.f;
                 if (seen) {
-                    if (kk < blocks) seen = kk < (hi ? nb_hi : nb_lo);
-                    else { const int j = first + kk - blocks; seen = j <= i && j > i - window; bias = slope * (float)(i - j); }
+                    if (kk < blocks) { seen = kk < (hi ? nb_hi : nb_lo); if (keep > 0) bias = slope * (float)(i - kk); }
+                    else { const int j = first + kk - blocks; seen = j <= i && (j > i - window || j < keep); bias = slope * (float)(i - j); }
                 }
                 const float v = seen ? sc[n][x] * scale - bias : -INFINITY;
                 sc[n][x] = v;
@@ -784,17 +810,19 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         }
     }
     if (partial != nullptr) {
-        const int stride = vdim + 2;
-        float* p_lo = partial + (((size_t)(row0 + r_lo) * Hq + head) * splits + blockIdx.z) * stride;
-        float* p_hi = partial + (((size_t)(row0 + r_hi) * Hq + head) * splits + blockIdx.z) * stride;
-        if (tq == 0 && r_lo < n_q) { p_lo[0] = m_lo; p_lo[1] = l_lo; }
-        if (tq == 0 && r_hi < n_q) { p_hi[0] = m_hi; p_hi[1] = l_hi; }
+        float* p_lo = partial + (((size_t)(row0 + r_lo) * Hq + head) * splits + blockIdx.z) * span.stride;
+        float* p_hi = partial + (((size_t)(row0 + r_hi) * Hq + head) * splits + blockIdx.z) * span.stride;
+        const bool with_sums = tq == 0 && (span.width == 0 || v_col == 0);
+        if (with_sums && r_lo < n_q) { p_lo[0] = m_lo; p_lo[1] = l_lo; }
+        if (with_sums && r_hi < n_q) { p_hi[0] = m_hi; p_hi[1] = l_hi; }
+        p_lo += span.off + (span.width > 0 ? v_col : 0);
+        p_hi += span.off + (span.width > 0 ? v_col : 0);
 #pragma unroll
-        for (int n = 0; n < kValueTiles; ++n) {
+        for (int n = 0; n < kValueTiles; ++n) {      // (even offsets and strides: 8-byte stores)
             if (n >= vtiles) continue;
             const int c = n * 8 + 2 * tq;
-            if (r_lo < n_q) { p_lo[2 + c] = o[n][0]; p_lo[3 + c] = o[n][1]; }
-            if (r_hi < n_q) { p_hi[2 + c] = o[n][2]; p_hi[3 + c] = o[n][3]; }
+            if (r_lo < n_q) *reinterpret_cast<float2*>(p_lo + c) = make_float2(o[n][0], o[n][1]);
+            if (r_hi < n_q) *reinterpret_cast<float2*>(p_hi + c) = make_float2(o[n][2], o[n][3]);
         }
         return;
     }
@@ -834,16 +862,16 @@ static int launch_tile(const void* q, const void* k_cache, const void* v_cache, 
                        const int* block_table, int table_width, const int* pooled_table, int pooled_width, const int* cu,
                        const int* start_pos, const int* tiles, int num_tiles, const float* v_table, int v_rot, int table_rows,
                        void* out, int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
-                       float* partial, int splits, ScoreExtras extras, void* stream) {
+                       float* partial, int splits, ScoreExtras extras, ValueSpan span, void* stream) {
     const size_t smem = (size_t)2 * kTileK * ((dim + 8) + (vdim + 8)) * sizeof(__nv_bfloat16);
     static size_t have = 0;
     ensure_dynamic_smem(pooled_attention_tile_kernel<kDimSteps, kValueTiles>, smem, have);
-    dim3 grid(num_tiles, Hq, splits);
+    dim3 grid(num_tiles, Hq * (span.width > 0 ? (span.width + vdim - 1) / vdim : 1), splits);
     pooled_attention_tile_kernel<kDimSteps, kValueTiles><<<grid, kTileThreads, smem, (cudaStream_t)stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (const __nv_bfloat16*)kp_cache,
         (const __nv_bfloat16*)vp_cache, block_table, table_width, pooled_table, pooled_width, cu, start_pos, tiles, v_table, v_rot,
-        table_rows, (__nv_bfloat16*)out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits > 1 ? partial : nullptr, splits,
-        extras);
+        table_rows, (__nv_bfloat16*)out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits > 1 || span.width > 0 ? partial : nullptr,
+        splits, extras, span);
     return launch_status();
 }
 
@@ -857,15 +885,17 @@ static int tile_dispatch(const void* q, const void* k_cache, const void* v_cache
                                         int pooled_width, const int* cu, const int* start_pos, const int* tiles, int num_tiles,
                                         const float* v_table, int v_rot, int table_rows, void* out, int Hq, int Hkv, int dim,
                                         int vdim, int page_size, float scale, int window, int pool, float* partial, int splits,
-                                        ScoreExtras extras, void* stream) {
+                                        ScoreExtras extras, ValueSpan span, void* stream) {
     if (num_tiles <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hq > 65535 || dim <= 0 || dim % 16 || vdim <= 0 || vdim % 8 || page_size <= 0 || window <= 0
-        || pool < 0 || (v_rot & 1) || v_rot > vdim || table_rows <= 0)
+        || pool < 0 || (v_rot & 1) || v_rot > vdim || table_rows <= 0 || extras.keep < 0 || (extras.keep > 0 && pool > 0)
+        || span.width % 8 || span.stride % 2 || span.off % 2)
         return kBadSize;
-    if (dim > 128 || vdim > 128 || splits < 1 || splits > 64 || (splits > 1 && partial == nullptr)) return kTooLarge;
+    if (dim > 128 || vdim > 128 || splits < 1 || splits > 64 || ((splits > 1 || span.width > 0) && partial == nullptr)) return kTooLarge;
+    if (extras.keep > 0) { kp_cache = k_cache; vp_cache = v_cache; pooled_table = block_table; pooled_width = table_width; }
 #define LB_TILE(DS, VT) return launch_tile<DS, VT>(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, pooled_table, \
         pooled_width, cu, start_pos, tiles, num_tiles, v_table, v_rot, table_rows, out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, \
-        partial, splits, extras, stream)
+        partial, splits, extras, span, stream)
     const int ds = dim / 16, vt = vdim / 8;
     if (ds <= 2) { if (vt <= 4) LB_TILE(2, 4); if (vt <= 8) LB_TILE(2, 8); if (vt <= 12) LB_TILE(2, 12); LB_TILE(2, 16); }
     if (ds <= 4) { if (vt <= 4) LB_TILE(4, 4); if (vt <= 8) LB_TILE(4, 8); if (vt <= 12) LB_TILE(4, 12); LB_TILE(4, 16); }
@@ -882,17 +912,150 @@ extern "C" int lb_pooled_attention_tile(const void* q, const void* k_cache, cons
                                         const int* positions, int tokens, const float* v_table, int v_rot, int table_rows, void* out,
                                         int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
                                         float* partial, int splits, const float* slopes, const float* sinks, const void* gate,
-                                        long gate_stride, void* stream) {
+                                        long gate_stride, int keep, void* stream) {
     // (with several CTAs per run the sink joins in the merge, once)
     const int code = tile_dispatch(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, pooled_table, pooled_width, cu,
                                    start_pos, tiles, num_tiles, v_table, v_rot, table_rows, out, Hq, Hkv, dim, vdim, page_size, scale,
-                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks, gate, gate_stride}, stream);
+                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks, gate, gate_stride, keep},
+                                   ValueSpan{0, vdim + 2, 2}, stream);
     if (code != 0 || splits <= 1 || num_tiles <= 0 || tokens <= 0) return code;
     dim3 grid(tokens, Hq);
     pooled_merge_kernel<__nv_bfloat16><<<grid, 32, 0, (cudaStream_t)stream>>>(partial, positions, nullptr, v_table, v_rot, table_rows,
                                                                             (__nv_bfloat16*)out, Hq, vdim, splits,
-                                                                            ScoreExtras{nullptr, sinks, gate, gate_stride});
+                                                                            ScoreExtras{nullptr, sinks, gate, gate_stride, 0});
     return launch_status();
+}
+
+// ------------------------------------------------------------------------------------------------ heads that mix their weights
+// With w_g(i, j) the softmax weights of head g (its denominator holds the sink, which has no weight of its own), head h of
+// key/value head c applies sum_g M[h, g] w_g(i, j) to the values of c.  The mix moves behind the sum over the keys:
+//     o_h(i) = sum_g M[h, g] U_gc(i),     U_gc(i) = sum_j w_g(i, j) v_c(j)
+// so the attention kernels above sum the weights of every head over the values of ALL key/value heads (`ValueSpan`) in one
+// ordinary online softmax, and leave (maximum, sum, weighted values) per key range; this kernel joins the ranges and the
+// sink, divides, and mixes, all in float32.
+// grid (tokens, Hkv, column blocks of kTalkCols), 256 threads: 256 / kTalkCols slices of the heads g share a column, their
+// sums meet in shared memory.  Dynamic shared memory: Hq * splits floats (what a range's sums are multiplied by).
+constexpr int kTalkOff = 8;               // floats in front of the value columns of a partial result
+constexpr int kTalkHeads = 8;             // output heads at a time
+template <typename T, int kTalkCols>
+__global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict__ partial, const int* __restrict__ token_list,
+                                                         const float* __restrict__ talk, const float* __restrict__ sinks,
+                                                         T* __restrict__ out, int Hq, int Hkv, int vdim, int splits) {
+    constexpr int kSlices = 256 / kTalkCols;
+    extern __shared__ float factor[];                          // [Hq][splits]
+    __shared__ float red[kSlices][kTalkHeads][kTalkCols];
+    const int slot = blockIdx.x, c = blockIdx.y, col0 = blockIdx.z * kTalkCols;
+    const int t = token_list != nullptr ? token_list[slot] : slot;
+    if (t < 0) return;
+    const int per = Hq / Hkv, stride = Hkv * vdim + kTalkOff;
+    const float* src = partial + (size_t)slot * Hq * splits * stride;
+    for (int g = threadIdx.x; g < Hq; g += blockDim.x) {
+        const float* s0 = src + (size_t)g * splits * stride;
+        float mm = sinks != nullptr ? sinks[g] : -INFINITY;
+        for (int s = 0; s < splits; ++s) mm = fmaxf(mm, s0[(size_t)s * stride]);
+        float ll = sinks != nullptr ? expf(sinks[g] - mm) : 0.f;
+        for (int s = 0; s < splits; ++s) {
+            const float m = s0[(size_t)s * stride], f = m == -INFINITY ? 0.f : expf(m - mm);
+            factor[g * splits + s] = f;
+            ll += f * s0[(size_t)s * stride + 1];
+        }
+        const float inv = ll > 0.f ? 1.f / ll : 0.f;
+        for (int s = 0; s < splits; ++s) factor[g * splits + s] *= inv;
+    }
+    __syncthreads();
+    const int slice = threadIdx.x / kTalkCols, col = threadIdx.x % kTalkCols;
+    const bool live = col0 + col < vdim;
+    const float* column = src + kTalkOff + c * vdim + col0 + (live ? col : 0);
+    for (int r0 = 0; r0 < per; r0 += kTalkHeads) {
+        const int nr = min(kTalkHeads, per - r0);
+        const float* mix = talk + (size_t)(c * per + r0) * Hq;
+        float acc[kTalkHeads];
+#pragma unroll
+        for (int r = 0; r < kTalkHeads; ++r) acc[r] = 0.f;
+        for (int g = slice; g < Hq; g += kSlices) {
+            float u = 0.f;
+            for (int s = 0; s < splits; ++s) {
+                const float f = factor[g * splits + s];
+                if (f != 0.f) u += f * column[((size_t)g * splits + s) * stride];     // (a range without keys holds no sums)
+            }
+#pragma unroll
+            for (int r = 0; r < kTalkHeads; ++r)
+                if (r < nr) acc[r] += mix[(size_t)r * Hq + g] * u;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int r = 0; r < kTalkHeads; ++r) red[slice][r][col] = acc[r];
+        __syncthreads();
+        for (int i = threadIdx.x; i < nr * kTalkCols; i += blockDim.x) {
+            const int r = i / kTalkCols, cc = i % kTalkCols;
+            if (col0 + cc >= vdim) continue;
+            float sum = 0.f;
+#pragma unroll
+            for (int s = 0; s < kSlices; ++s) sum += red[s][r][cc];
+            out[((size_t)t * Hq + c * per + r0 + r) * vdim + col0 + cc] = from_f32<T>(sum);
+        }
+    }
+}
+
+static int launch_talk_merge(const float* partial, const int* token_list, int tokens, const float* talk, const float* sinks, void* out,
+                             int Hq, int Hkv, int vdim, int splits, int dtype, void* stream) {
+    const size_t smem = (size_t)Hq * splits * sizeof(float);
+    if (smem > 96 * 1024) return kTooLarge;
+#define LB_TALK(COLS) LB_DISPATCH_DTYPE(dtype, { \
+        static size_t have = 0; \
+        ensure_dynamic_smem(talk_merge_kernel<T, COLS>, smem + 40 * 1024, have); \
+        talk_merge_kernel<T, COLS><<<dim3(tokens, Hkv, (vdim + COLS - 1) / COLS), 256, smem, (cudaStream_t)stream>>>( \
+            partial, token_list, talk, sinks, (T*)out, Hq, Hkv, vdim, splits); })
+    if (vdim <= 32) { LB_TALK(32); } else if (vdim <= 64) { LB_TALK(64); } else { LB_TALK(128); }
+#undef LB_TALK
+    return launch_status();
+}
+
+extern "C" int lb_talk_partial_offset() { return kTalkOff; }
+
+// Attention over a window and `keep` first tokens with mixed weights.  talk: float32 [Hq, Hq]; sinks: float32 [Hq] or null;
+// partial: float32 scratch of num_tokens * Hq * splits * (Hkv * vdim + kTalkOff); dim up to 1024
+extern "C" int lb_talk_attention_split(const void* q, const void* k_cache, const void* v_cache, const int* block_table, int table_width,
+                                       const int* token_req, const int* positions, const int* token_list, int num_tokens, float* partial,
+                                       void* out, const float* talk, const float* sinks, int Hq, int Hkv, int dim, int vdim, int page_size,
+                                       float scale, int window, int keep, int splits, int dtype, void* stream) {
+    if (num_tokens <= 0) return kOk;
+    if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || dim <= 0 || vdim <= 0 || page_size <= 0 || window <= 0 || keep < 0 || splits <= 0 || splits > 65535)
+        return kBadSize;
+    if (dim > 1024) return kTooLarge;
+    const int per = Hq / Hkv, width = Hkv * vdim;
+    const ScoreExtras extras{nullptr, nullptr, nullptr, 0, keep};
+    const ValueSpan span{width, width + kTalkOff, kTalkOff};
+    int code;
+#define LB_SPLIT(PER, REGS) LB_DISPATCH_DTYPE(dtype, code = (launch_split<T, PER, REGS>(q, k_cache, v_cache, k_cache, v_cache, block_table, table_width, \
+        block_table, table_width, token_req, positions, token_list, num_tokens, partial, Hq, Hkv, dim, min(width, 32 * REGS), page_size, scale, window, \
+        0, splits, extras, span, stream)))
+#define LB_SPLIT_PER(PER) { if (width <= 128) { LB_SPLIT(PER, 4); } else if (width <= 256) { LB_SPLIT(PER, 8); } else { LB_SPLIT(PER, 16); } }
+    if (per == 1) LB_SPLIT_PER(1) else if (per == 2) LB_SPLIT_PER(2) else LB_SPLIT_PER(4)
+#undef LB_SPLIT_PER
+#undef LB_SPLIT
+    if (code != 0) return code;
+    return launch_talk_merge(partial, token_list, num_tokens, talk, sinks, out, Hq, Hkv, vdim, splits, dtype, stream);
+}
+
+// The same for the long portions' runs on the tensor cores (see `lb_pooled_attention_tile`): the merge goes over ALL `tokens` rows,
+// those that no run covers get nothing of meaning.  bfloat16; dim a multiple of 16 up to 128, vdim a multiple of 8;
+// partial: float32 scratch of tokens * Hq * splits * (Hkv * vdim + kTalkOff)
+extern "C" int lb_talk_attention_tile(const void* q, const void* k_cache, const void* v_cache, const int* block_table, int table_width,
+                                      const int* cu, const int* start_pos, const int* tiles, int num_tiles, int tokens, float* partial,
+                                      void* out, const float* talk, const float* sinks, int Hq, int Hkv, int dim, int vdim, int page_size,
+                                      float scale, int window, int keep, int splits, void* stream) {
+    if (num_tiles <= 0 || tokens <= 0) return kOk;
+    if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || vdim <= 0) return kBadSize;
+    const int width = Hkv * vdim;
+    // value columns of a CTA: as few chunks as 128 columns allow, of about equal width
+    const int chunks = (width + 127) / 128, chunk = ((width + chunks - 1) / chunks + 7) / 8 * 8;
+    if ((long)Hq * chunks > 65535) return kTooLarge;
+    const int code = tile_dispatch(q, k_cache, v_cache, k_cache, v_cache, block_table, table_width, block_table, table_width, cu, start_pos, tiles,
+                                   num_tiles, nullptr, 0, 1, nullptr, Hq, Hkv, dim, chunk, page_size, scale, window, 0, partial, splits,
+                                   ScoreExtras{nullptr, nullptr, nullptr, 0, keep}, ValueSpan{width, width + kTalkOff, kTalkOff}, stream);
+    if (code != 0) return code;
+    return launch_talk_merge(partial, nullptr, tokens, talk, sinks, out, Hq, Hkv, vdim, splits, kBF16, stream);
 }
 
 // ------------------------------------------------------------------------------------------------------------------

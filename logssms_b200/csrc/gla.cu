@@ -12,6 +12,9 @@
 //  take bfloat16 operands, the scaled queries and keys and the state's copy then enter as TWO bfloat16 terms each (hi =
 //  bf16(x), lo = bf16(x - hi)), so that they are applied to 16 bits and more instead of 8 (values are bfloat16 as projected).
 //
+//  With a `Turn` q and k are first rotated by their position (in halves: of every head's first n columns, column i and column
+//  i + n/2) and k is multiplied by a number, all in 32-bit while they are loaded; the chunked form then takes two terms too.
+//
 //  gla_scan      : the recurrence over every request's tokens of a step, state read from and written back to the
 //                  request's slot (a request that starts at position 0 starts from zeros whatever the slot holds).
 //                  A CTA owns (request, head, a tile of value channels); a thread owns R state rows of one value
@@ -41,12 +44,32 @@ __device__ __forceinline__ float gate_log_decay(float z, float l, float key) {
     return l > 0.f ? logf(gate_decay(z, l)) : log_sigmoid(z);
 }
 
+// A rotation of q and k by the token's position, and a factor of k.
+struct Turn {
+    const float* table;       // [rows, n]: cos | sin of the n/2 pairs; not read with n = 0
+    int n, rows;
+    const int* positions;     // [tokens]
+    float k_scale;
+    __device__ __forceinline__ const float* row(size_t token) const {
+        return n > 0 ? table + (size_t)min(max(positions[token], 0), rows - 1) * n : nullptr;
+    }
+    // column d of a head's row x, turned
+    template <typename T>
+    __device__ __forceinline__ float at(const T* x, int d, const float* cs) const {
+        const float v = to_f32(x[d]);
+        if (d >= n) return v;
+        const int half = n >> 1;
+        if (d < half) return v * cs[d] - to_f32(x[d + half]) * cs[half + d];
+        return v * cs[d - half] + to_f32(x[d - half]) * cs[d];
+    }
+};
+
 template <typename T, int R, int DS>
 __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k, const T* __restrict__ v, long row_stride,
                                 const float* __restrict__ z, float* __restrict__ o, float* state,
                                 const int* __restrict__ cu, const int* __restrict__ start_pos, const int* __restrict__ slots,
                                 const int* __restrict__ request_list, int H, int dim, int vdim, float inv_tau, float q_scale,
-                                const float* __restrict__ head_decay, BoundedGate gate) {
+                                const float* __restrict__ head_decay, BoundedGate gate, Turn turn) {
     constexpr int DP = R * DS;                       // key channels, padded
     extern __shared__ float sm[];
     const int cols = blockDim.x / DS;
@@ -76,7 +99,8 @@ __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k
             float qv = 0.f, kv = 0.f, av = 0.f;
             if (d < dim) {
                 const size_t row = (size_t)(t0 + tt);
-                qv = to_f32(q[row * row_stride + h * dim + d]) * q_scale;
+                const float* cs = turn.row(row);
+                qv = turn.at(q + row * row_stride + h * dim, d, cs) * q_scale;
                 if (gate.lower != nullptr) {
                     const float l = gate.lower[h * dim + d];
                     const float zz = z[(row * H + h) * dim + d] + (gate.bias != nullptr ? gate.bias[h * dim + d] : 0.f);
@@ -84,7 +108,7 @@ __global__ void gla_scan_kernel(const T* __restrict__ q, const T* __restrict__ k
                     kv = gate_key(zz, l);
                     av = gate_decay(zz, l);
                 } else {
-                    kv = to_f32(k[row * row_stride + h * dim + d]);
+                    kv = turn.at(k + row * row_stride + h * dim, d, cs) * turn.k_scale;
                     av = head_decay != nullptr ? head_decay[h] : expf(log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau);
                 }
             }
@@ -122,7 +146,7 @@ template <typename T, int R, int DS>
 static int launch_gla_scan(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                            const int* cu, const int* start_pos, const int* slots, const int* request_list, int num_requests,
                            int H, int dim, int vdim, float inv_tau, float q_scale, const float* head_decay, BoundedGate gate,
-                           cudaStream_t stream) {
+                           Turn turn, cudaStream_t stream) {
     // few requests: narrow tiles, so that more CTAs share the work
     const int want = (num_requests * H * ((vdim * DS + 127) / 128) < 148) ? 32 : 128;
     const int threads = min(want, (vdim * DS + 31) / 32 * 32);
@@ -132,24 +156,28 @@ static int launch_gla_scan(const void* q, const void* k, const void* v, long row
     static size_t have = 0;
     ensure_dynamic_smem(gla_scan_kernel<T, R, DS>, smem, have);
     gla_scan_kernel<T, R, DS><<<grid, threads, smem, stream>>>((const T*)q, (const T*)k, (const T*)v, row_stride, z, o, state, cu,
-                                                               start_pos, slots, request_list, H, dim, vdim, inv_tau, q_scale, head_decay, gate);
+                                                               start_pos, slots, request_list, H, dim, vdim, inv_tau, q_scale, head_decay, gate,
+                                                               turn);
     return launch_status();
 }
 
 // q, k: [tokens, H*dim] and v: [tokens, H*vdim], column views of one projection buffer (common row stride, in
 // elements); z: float32 [tokens, H*dim]; o: float32 [tokens, H*vdim]; state: float32 [slots, H, dim, vdim].  With `lower`
-// (float32 [H*dim]; `z_bias` float32 [H*dim] or null) k is not read and q_scale must be 1.
+// (float32 [H*dim]; `z_bias` float32 [H*dim] or null) k is not read and q_scale must be 1.  rot_table: float32 [rot_rows, rot] (rot
+// 0: no rotation); k_scale: a factor of k.
 extern "C" int lb_gla_scan(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                            const int* cu, const int* start_pos, const int* slots, const int* request_list, int num_requests,
                            int H, int dim, int vdim, float tau, float q_scale, const float* head_decay, const float* lower,
-                           const float* z_bias, int dtype, void* stream) {
+                           const float* z_bias, const float* rot_table, int rot, int rot_rows, const int* positions, float k_scale,
+                           int dtype, void* stream) {
     if (num_requests <= 0) return kOk;
     if (H <= 0 || dim <= 0 || vdim <= 0 || !(tau > 0.f)) return kBadSize;
+    if (rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (rot_table == nullptr || positions == nullptr || rot_rows <= 0))) return kBadSize;
     if (lower != nullptr && (z == nullptr || head_decay != nullptr || q_scale != 1.f)) return kBadSize;
     if (dim > 512) return kTooLarge;
     cudaStream_t st = (cudaStream_t)stream;
 #define LB_GLA(R_, DS_) LB_DISPATCH_DTYPE(dtype, return (launch_gla_scan<T, R_, DS_>(q, k, v, row_stride, z, o, state, cu, start_pos, \
-        slots, request_list, num_requests, H, dim, vdim, 1.f / tau, q_scale, head_decay, BoundedGate{lower, z_bias}, st)))
+        slots, request_list, num_requests, H, dim, vdim, 1.f / tau, q_scale, head_decay, BoundedGate{lower, z_bias}, Turn{rot_table, rot, rot_rows, positions, k_scale}, st)))
     if (dim <= 16) { LB_GLA(16, 1); }
     else if (dim <= 32) { LB_GLA(32, 1); }
     else if (dim <= 64) { LB_GLA(64, 1); }
@@ -179,7 +207,7 @@ __global__ void gla_norm_gate_kernel(const float* __restrict__ o, const T* __res
             const float g = to_f32(gate[row * gate_stride + h * vdim + c]);
             f = sigmoid_gate ? 1.f / (1.f + expf(-g)) : silu_f(g);
         }
-        out[(row * H + h) * vdim + c] = from_f32<T>(orow[c] * inv * weight[c] * f);
+        out[(row * H + h) * vdim + c] = from_f32<T>(orow[c] * inv * (weight != nullptr ? weight[c] : 1.f) * f);
     }
 }
 
@@ -216,7 +244,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
         const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ k, long row_stride, const float* __restrict__ z,
         const int* __restrict__ cu, const int* __restrict__ chunks, __nv_bfloat16* __restrict__ q_in,
         __nv_bfloat16* __restrict__ k_end, float* __restrict__ A, float* __restrict__ D, int H, int dim, float inv_tau,
-        float q_scale, const float* __restrict__ head_decay, BoundedGate gate, size_t plane) {
+        float q_scale, const float* __restrict__ head_decay, BoundedGate gate, Turn turn, size_t plane) {
     extern __shared__ float sm[];
     float* b = sm;                         // [16][dim] log-decays, then their running sums
     float* qs = b + kChunk * dim;
@@ -231,7 +259,8 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
         float ld = 0.f, qv = 0.f, kv = 0.f;
         if (j < n) {
             const size_t row = (size_t)(t0 + j);
-            qv = to_f32(q[row * row_stride + h * dim + d]) * q_scale;
+            const float* cs = turn.row(row);
+            qv = turn.at(q + row * row_stride + h * dim, d, cs) * q_scale;
             if (gate.lower != nullptr) {
                 const float l = gate.lower[h * dim + d];
                 const float zz = z[(row * H + h) * dim + d] + (gate.bias != nullptr ? gate.bias[h * dim + d] : 0.f);
@@ -240,7 +269,7 @@ __global__ void __launch_bounds__(128) gla_chunk_prepare_kernel(
                 ld = gate_log_decay(zz, l, kv);
             } else {
                 ld = head_decay != nullptr ? logf(head_decay[h]) : log_sigmoid(z[(row * H + h) * dim + d]) * inv_tau;
-                kv = to_f32(k[row * row_stride + h * dim + d]);
+                kv = turn.at(k + row * row_stride + h * dim, d, cs) * turn.k_scale;
             }
         }
         b[i] = ld; qs[i] = qv; ks[i] = kv;
@@ -532,20 +561,23 @@ __global__ void gla_segment_pass_kernel(float* seg_state, const float* __restric
 // the scan; chunks: int32 [num_chunks, 2] (request, first token within its portion; request -1: nothing);
 // per_request: int32 [num_long, 3] (request, its first chunk, its number of chunks).  Scratch: q_in, k_end
 // [tokens, H, dim] bfloat16, A float32 [tokens, H, 16], D float32 [num_chunks, H, dim].  dim: a multiple of 16, <= 256.
-// With `lower` (see `lb_gla_scan`) q_in and k_end have two planes of `tokens` rows each.
+// With `lower` (see `lb_gla_scan`) or `two_terms` q_in and k_end have two planes of `tokens` rows each.
 extern "C" int lb_gla_chunked(const void* q, const void* k, const void* v, long row_stride, const float* z, float* o, float* state,
                               const int* cu, const int* start_pos, const int* slots, const int* chunks, int num_chunks,
                               const int* per_request, int num_long, void* q_in, void* k_end, float* A, float* D, int H, int dim,
                               int vdim, float tau, float q_scale, const int* segments, int num_segments, float* seg_state,
                               float* seg_decay, const float* head_decay, const float* lower, const float* z_bias, int tokens,
+                              const float* rot_table, int rot, int rot_rows, const int* positions, float k_scale, int two_terms,
                               void* stream) {
     if (num_chunks <= 0 || num_long <= 0) return kOk;
+    if (rot < 0 || rot > dim || (rot & 1) || (rot > 0 && (rot_table == nullptr || positions == nullptr || rot_rows <= 0))) return kBadSize;
+    if (two_terms && tokens <= 0) return kBadSize;
     if (lower != nullptr && (z == nullptr || head_decay != nullptr || q_scale != 1.f || tokens <= 0)) return kBadSize;
     if (H <= 0 || dim <= 0 || vdim <= 0 || !(tau > 0.f) || dim % 16) return kBadSize;
     if (dim > 256) return kTooLarge;
     cudaStream_t st = (cudaStream_t)stream;
     typedef __nv_bfloat16 bf;
-    const bool split = lower != nullptr;
+    const bool split = lower != nullptr || two_terms != 0;
     const size_t plane = split ? (size_t)tokens * H * dim : 0;
     {
         const size_t smem = (size_t)3 * kChunk * dim * sizeof(float);
@@ -553,7 +585,7 @@ extern "C" int lb_gla_chunked(const void* q, const void* k, const void* v, long 
         ensure_dynamic_smem(gla_chunk_prepare_kernel, smem, have);
         gla_chunk_prepare_kernel<<<dim3(num_chunks, H), 128, smem, st>>>((const bf*)q, (const bf*)k, row_stride, z, cu, chunks,
                                                                         (bf*)q_in, (bf*)k_end, A, D, H, dim, 1.f / tau, q_scale, head_decay,
-                                                                        BoundedGate{lower, z_bias}, plane);
+                                                                        BoundedGate{lower, z_bias}, Turn{rot_table, rot, rot_rows, positions, k_scale}, plane);
         const int rc = launch_status();
         if (rc != 0) return rc;
     }

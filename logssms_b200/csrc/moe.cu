@@ -23,6 +23,7 @@
 //                     more expert of that size (input gate | up, output), whose weight is dense column `tail_gate`, or 1.
 //  moe_add_identity : out += id_weight[t] * h
 //  gelu_tanh        : 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
+//  xielu            : a z^2 + z/2 for z > 0, b (e^z - 1 - z) + z/2 for z <= 0, with a and b read from memory
 #include "lb200/common.cuh"
 using namespace lb200;
 
@@ -327,6 +328,40 @@ __global__ void gelu_tanh_kernel(const T* __restrict__ in, T* __restrict__ out, 
 extern "C" int lb_gelu_tanh(const void* in, void* out, long n, int dtype, void* stream) {
     if (n <= 0) return kOk;
     LB_DISPATCH_DTYPE(dtype, gelu_tanh_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>((const T*)in, (T*)out, (size_t)n));
+    return launch_status();
+}
+
+__device__ __forceinline__ float xielu_f(float z, float a, float b) {
+    return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
+
+template <typename T>
+__global__ void xielu_kernel(const T* __restrict__ in, T* __restrict__ out, const float* __restrict__ ab, size_t n) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) out[i] = from_f32<T>(xielu_f(to_f32(in[i]), ab[0], ab[1]));
+}
+
+// bfloat16, eight values (one 16-byte word) per thread
+__global__ void xielu_vec_kernel(const uint4* __restrict__ in, uint4* __restrict__ out, const float* __restrict__ ab, size_t words) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= words) return;
+    const float a = ab[0], b = ab[1];
+    uint4 v = in[i];
+    __nv_bfloat162* p = reinterpret_cast<__nv_bfloat162*>(&v);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { const float2 f = __bfloat1622float2(p[e]); p[e] = __floats2bfloat162_rn(xielu_f(f.x, a, b), xielu_f(f.y, a, b)); }
+    out[i] = v;
+}
+
+// ab: float32 [2], the factors a and b
+extern "C" int lb_xielu(const void* in, void* out, const float* ab, long n, int dtype, void* stream) {
+    if (n <= 0) return kOk;
+    if (dtype == kBF16 && n % 8 == 0 && (((uintptr_t)in | (uintptr_t)out) & 15) == 0) {
+        const size_t words = (size_t)n / 8;
+        xielu_vec_kernel<<<(unsigned)((words + 255) / 256), 256, 0, (cudaStream_t)stream>>>((const uint4*)in, (uint4*)out, ab, words);
+        return launch_status();
+    }
+    LB_DISPATCH_DTYPE(dtype, xielu_kernel<T><<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>((const T*)in, (T*)out, ab, (size_t)n));
     return launch_status();
 }
 

@@ -316,3 +316,16 @@ extern "C" int lb_scale(const void* x, void* out, long n, float s, int to_f32_ou
     });
     return launch_status();
 }
+
+// x <- cap * tanh(x / cap) in place, in 32-bit: logits that saturate at +-cap
+__global__ void softcap_kernel(float* __restrict__ x, size_t n, float cap) {
+    const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < n) x[i] = cap * tanhf(x[i] / cap);
+}
+
+extern "C" int lb_softcap(float* x, long n, float cap, void* stream) {
+    if (n <= 0) return kOk;
+    if (!(cap > 0.f)) return kBadSize;
+    softcap_kernel<<<(unsigned)((n + 255) / 256), 256, 0, (cudaStream_t)stream>>>(x, (size_t)n, cap);
+    return launch_status();
+}

@@ -5,7 +5,8 @@
 //                     first divided by its root mean square, sqrt(mean(y^2) + unit_eps))
 //                     x_out = v (may be x itself), h = N(v) * w rounded to the activation dtype (what the next
 //                     sublayer's products read; N may be "none": h is v rounded)
-//   stream_add_many : v = x + sum_i s_i * y_i (up to four addends, a scalar each), x_out = v in place, h = N(v) * w
+//   stream_add_many : v = x + sum_i s_i * y_i (up to four addends, a scalar each) [+ b, one float32 vector for all rows],
+//                     x_out = v in place, h = N(v) * w
 //   stream_add_conv_step : stream_add_many for a decode batch (row t is the single new token of request t) whose normed row
 //                     also passes a short causal convolution per channel before it is stored: with u = N(v) * w rounded,
 //                       h = sum_j cw[c, j] * u_(t - taps + 1 + j)
@@ -117,11 +118,13 @@ extern "C" int lb_stream_add_norm(const float* x, const void* y, const float* ls
 }
 
 // v = x + sum_i s_i * y_i for up to four addends with a scalar each (the sublayers of a block whose mixers and feed-forward all
-// read one norm's output), x_out = v in place, h = N(v) * w as in `stream_add_norm`
+// read one norm's output) and, if there is one, a vector that every row gets, x_out = v in place, h = N(v) * w as in
+// `stream_add_norm`
 struct Addends {
     const void* y[4];
     float s[4];
     int n;
+    const float* row;         // [H] or null
 };
 
 template <typename T>
@@ -134,6 +137,7 @@ __global__ void stream_add_many_kernel(float* x, Addends a, const float* __restr
 #pragma unroll
         for (int i = 0; i < 4; ++i)
             if (i < a.n) v += a.s[i] * to_f32(((const T*)a.y[i])[base + c]);
+        if (a.row != nullptr) v += a.row[c];
         row[c] = v;
         x[base + c] = v;
     }
@@ -145,13 +149,13 @@ __global__ void stream_add_many_kernel(float* x, Addends a, const float* __restr
 }
 
 extern "C" int lb_stream_add_many(float* x, const void* y0, const void* y1, const void* y2, const void* y3, float s0, float s1, float s2,
-                                  float s3, int n, const float* w, float eps, void* h_out, int rows, int H, int kind, int dtype,
-                                  void* stream) {
+                                  float s3, int n, const float* row, const float* w, float eps, void* h_out, int rows, int H, int kind,
+                                  int dtype, void* stream) {
     if (rows <= 0) return kOk;
     if (H <= 0 || (size_t)H * sizeof(float) > 160 * 1024 || kind < kLayerNorm || kind > kNoNorm || n < 0 || n > 4) return kBadSize;
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     const size_t smem = (size_t)H * sizeof(float);
-    const Addends a = {{y0, y1, y2, y3}, {s0, s1, s2, s3}, n};
+    const Addends a = {{y0, y1, y2, y3}, {s0, s1, s2, s3}, n, row};
     LB_DISPATCH_DTYPE(dtype, {
         static size_t have = 0;
         ensure_dynamic_smem(stream_add_many_kernel<T>, smem, have);
@@ -175,8 +179,9 @@ __global__ void stream_add_conv_step_kernel(float* x, Addends a, const float* __
 #pragma unroll
         for (int i = 0; i < 4; ++i)
             if (i < a.n) v += a.s[i] * to_f32(((const T*)a.y[i])[base + c]);
+        if (a.row != nullptr) v += a.row[c];
         row[c] = v;
-        if (a.n > 0) x[base + c] = v;
+        if (a.n > 0 || a.row != nullptr) x[base + c] = v;
     }
     __syncthreads();
     float mean, inv;
@@ -198,14 +203,14 @@ __global__ void stream_add_conv_step_kernel(float* x, Addends a, const float* __
 }
 
 extern "C" int lb_stream_add_conv_step(float* x, const void* y0, const void* y1, const void* y2, const void* y3, float s0, float s1,
-                                       float s2, float s3, int n, const float* w, float eps, const float* cw, int taps, void* conv_state,
+                                       float s2, float s3, int n, const float* row, const float* w, float eps, const float* cw, int taps, void* conv_state,
                                        const int* slots, const int* start_pos, void* h_out, int rows, int H, int kind, int dtype,
                                        void* stream) {
     if (rows <= 0) return kOk;
     if (H <= 0 || (size_t)H * sizeof(float) > 160 * 1024 || kind < kLayerNorm || kind > kNoNorm || n < 0 || n > 4 || taps < 1) return kBadSize;
     const int threads = H >= 2048 ? 1024 : (H >= 512 ? 512 : 128);
     const size_t smem = (size_t)H * sizeof(float);
-    const Addends a = {{y0, y1, y2, y3}, {s0, s1, s2, s3}, n};
+    const Addends a = {{y0, y1, y2, y3}, {s0, s1, s2, s3}, n, row};
     LB_DISPATCH_DTYPE(dtype, {
         static size_t have = 0;
         ensure_dynamic_smem(stream_add_conv_step_kernel<T>, smem, have);

@@ -53,4 +53,8 @@ from ..config.dimudra import ARCHITECTURE as _DIMUDRA, DimudraConfig  # noqa: E4
 
 register_architecture(_DIMUDRA, DimudraConfig)
 
+from ..config.fosupel import ARCHITECTURE as _FOSUPEL, FosupelConfig  # noqa: E402
+
+register_architecture(_FOSUPEL, FosupelConfig)
+
 __all__ = ["Architecture", "DecoderModel", "build_model", "register_architecture"]

@@ -25,12 +25,13 @@ class DecoderModel(Part):
         self.layers = [BLOCKS.get(b.kind)(b, perturb_init=perturb_init, shared=shared) for b in spec.layers]
         self.final_norm = NORMS.get(spec.final_norm.kind)(spec.final_norm, perturb_init)
         self.lm_head = HEADS.get(spec.lm_head_kind)(spec.vocab_size, spec.hidden_size, spec.lm_head_multiplier,
-                                                    self.embedding if spec.tie_word_embeddings else None)
+                                                    self.embedding if spec.tie_word_embeddings else None,
+                                                    **dict(getattr(spec, "lm_head_options", ())))
         # parts that several layers share and whose tensors are stored at the model's root (a second embedding table that
         # every layer reads a slice of): a layer puts them into `shared["model_parts"]` under their checkpoint prefix
         self.model_parts = dict(shared.get("model_parts", {}))
         # what mixes the embedding's output into the stream again as a run of layers opens (`ScheduleEntry.opens`): a product
-        # over both, or their sum
+        # over both, their sum, or a vector of the pass's own
         from ..parts.block import STREAM_INPUTS
         self.stream_inputs = [STREAM_INPUTS[s.kind](s, perturb_init) for s in getattr(spec, "stream_inputs", ())]
         for s, part in zip(getattr(spec, "stream_inputs", ()), self.stream_inputs):
@@ -42,6 +43,8 @@ class DecoderModel(Part):
                 raise ValueError(f"schedule names layer {e.layer}, the model has {len(self.layers)}")
             if e.opens is not None and not 0 <= e.opens < len(self.stream_inputs):
                 raise ValueError(f"schedule names stream input {e.opens}, the model has {len(self.stream_inputs)}")
+            if e.opens is not None and not 0 <= e.turn < getattr(self.stream_inputs[e.opens].spec, "count", e.turn + 1):
+                raise ValueError(f"schedule names pass {e.turn} of a stream input that has fewer")
         self.num_cache_layers = max(e.cache for e in self.schedule) + 1
         # an embedding with per-request state (`needs_context`) gets a cache layer of its own behind the blocks'
         self.embedding_cache_layer = None
@@ -134,12 +137,12 @@ class DecoderModel(Part):
             # that closes this block, except where a tap wants the stream as it is before)
             if e.opens is not None and not joined:
                 with nvtx_range("stream input"):
-                    x = self.stream_inputs[e.opens].forward(x, x0, x0_scale)
+                    x = self.stream_inputs[e.opens].forward(x, x0, x0_scale, e.turn)
             opens = self.schedule[i + 1].opens if i + 1 < len(self.schedule) else None
             joined = (opens is not None and getattr(self.stream_inputs[opens], "is_addend", False) and tap is None
                       and getattr(self.layers[e.layer], "joins_opening", False))
             ctx.extras["next_opens"] = opens is not None and not joined
-            ctx.extras["next_addend"] = (x0, x0_scale) if joined else None
+            ctx.extras["next_addend"] = self.stream_inputs[opens].addend(x0, x0_scale, self.schedule[i + 1].turn) if joined else None
             if PROFILER.nvtx:                      # named ranges per layer (and per part inside it) for a timeline
                 with nvtx_range(f"layer {e.layer}"):
                     x, residual = self.layers[e.layer].forward(x, residual, ctx, e.cache, e.writes_cache)

@@ -188,6 +188,15 @@ def scale(x: torch.Tensor, s: float, to_f32: bool = False) -> torch.Tensor:
 
 
 # --------------------------------------------------------------------------- rotary + cache store
+def softcap(x: torch.Tensor, cap: float) -> torch.Tensor:
+    """x <- cap * tanh(x / cap), in place, float32."""
+    _cuda(x)
+    _need(x.dtype == torch.float32 and x.is_contiguous() and cap > 0, "softcap wants contiguous float32 and a positive cap")
+    f = _fn("norm", "lb_softcap", [c_void_p, c_long, c_float, c_void_p])
+    _check(f(_ptr(x), x.numel(), cap, _stream()), "softcap")
+    return x
+
+
 def rope_table(inv_freq: torch.Tensor, rows: int, magnitude: float = 1.0) -> torch.Tensor:
     """[rows, 2*half] float32: cos | sin of position * inv_freq, both times `magnitude`."""
     _cuda(inv_freq)
@@ -1103,17 +1112,31 @@ def _gla_gate_checks(lower, z_bias, z, head_decay, q_scale: float, H: int, dk: i
         _need(t is None or (t.is_cuda and t.dtype == torch.float32 and t.shape == (H * dk,) and t.is_contiguous()), f"{name} must be float32 [H*key_dim]")
 
 
+def _gla_turn(turn, positions, T: int, dk: int) -> tuple:
+    """(table, its width, its rows, positions) of a rotation of q and k; `turn` None: no rotation."""
+    if turn is None or turn.shape[1] == 0:
+        return None, 0, 0, None
+    _need(turn.is_cuda and turn.dtype == torch.float32 and turn.dim() == 2 and turn.is_contiguous() and turn.shape[1] <= dk,
+          "the rotation table must be contiguous float32 [positions, n <= key_dim]")
+    _i32(positions, "positions")
+    _need(positions.numel() >= T, "one position per token")
+    return _ptr(turn), turn.shape[1], turn.shape[0], _ptr(positions)
+
+
 def gla_scan(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor,
              slots: torch.Tensor, num_requests: int, num_heads: int, key_dim: int, value_dim: int, tau: float,
              q_scale: float, request_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
              head_decay: torch.Tensor | None = None, lower: torch.Tensor | None = None,
-             z_bias: torch.Tensor | None = None) -> torch.Tensor:
+             z_bias: torch.Tensor | None = None, turn: torch.Tensor | None = None, positions: torch.Tensor | None = None,
+             k_scale: float = 1.0) -> torch.Tensor:
     """Token-by-token recurrence S <- diag(sigmoid(z)^(1/tau)) S + k v^T, o = S^T (q * q_scale) per head over every
     request's tokens.  qkv: [tokens, >= 2*H*key_dim + H*value_dim] with columns q | k | v first (unit column stride);
     z: float32 [tokens, H*key_dim]; state: float32 [slots, H, key_dim, value_dim], updated in place.  Returns float32
     [tokens, H*value_dim].  With `head_decay` (float32 [H]) every key channel of head h decays by head_decay[h] at every
     token, and z (then None) is not read.  With `lower` (float32 [H*key_dim]; `z_bias` float32 [H*key_dim] is added to z) the
-    decay is a = lower + (1 - lower) sigmoid(z), the key is 1 - a, q passes silu first, and qkv holds the columns q | v."""
+    decay is a = lower + (1 - lower) sigmoid(z), the key is 1 - a, q passes silu first, and qkv holds the columns q | v.
+    `turn` (float32 [positions, n], cos | sin of n/2 pairs, column i with column i + n/2): q and k of the token at `positions`
+    are rotated as they are loaded, and k is multiplied by `k_scale`, both in 32-bit."""
     _cuda(qkv, z, state, cu_seqlens, start_pos, slots, request_list, head_decay, lower, z_bias)
     H, dk, dv = num_heads, key_dim, value_dim
     T = qkv.shape[0]
@@ -1133,11 +1156,11 @@ def gla_scan(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seqlens
     item, base = qkv.element_size(), qkv.data_ptr()
     stride = qkv.stride(0) if T > 1 else qkv.shape[1]
     f = _fn("gla", "lb_gla_scan", [c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
-                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p, c_int,
-                                   c_void_p])
+                                   c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_float, c_float, c_void_p, c_void_p, c_void_p,
+                                   c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_void_p])
     _check(f(base, base + H * dk * item, base + (H * dk + keys) * item, stride, _ptr(z), _ptr(o), _ptr(state), _ptr(cu_seqlens),
              _ptr(start_pos), _ptr(slots), _ptr(request_list), n, H, dk, dv, tau, q_scale, _ptr(head_decay), _ptr(lower), _ptr(z_bias),
-             _code(qkv), _stream()),
+             *_gla_turn(turn, positions, T, dk), k_scale, _code(qkv), _stream()),
            "gla_scan", f"(key_dim {dk}, value_dim {dv})")
     return o
 
@@ -1157,13 +1180,15 @@ def gla_chunked(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seql
                 num_heads: int, key_dim: int, value_dim: int, tau: float, q_scale: float, out: torch.Tensor,
                 segments: torch.Tensor | None = None, segment_requests: torch.Tensor | None = None,
                 head_decay: torch.Tensor | None = None, lower: torch.Tensor | None = None,
-                z_bias: torch.Tensor | None = None) -> torch.Tensor:
+                z_bias: torch.Tensor | None = None, turn: torch.Tensor | None = None, positions: torch.Tensor | None = None,
+                k_scale: float = 1.0, two_terms: bool = False) -> torch.Tensor:
     """The recurrence of `gla_scan` over the long portions of a step in chunks of `GLA_CHUNK` tokens on the tensor cores
     (see `csrc/gla.cu`); the rows of the other requests in `out` (float32 [tokens, H*value_dim]) are left alone.
     `chunks`, `per_request`: the work lists of `StepContext.long_portion_chunks(GLA_CHUNK)`.  With `segments` and
     `segment_requests` (`StepContext.long_portion_segments`) every request's segments run side by side, twice, with a
     pass over their states between: for steps whose few long portions would leave most of the GPU idle.  `lower`, `z_bias`:
-    as for `gla_scan`; the products' operands are then handed to the tensor cores as two bfloat16 terms each."""
+    as for `gla_scan`; the products' operands are then handed to the tensor cores as two bfloat16 terms each, and so they are
+    with `two_terms`.  `turn`, `positions`, `k_scale`: as for `gla_scan`."""
     _cuda(qkv, z, state, cu_seqlens, start_pos, slots, chunks, per_request, out, head_decay, lower, z_bias)
     H, dk, dv = num_heads, key_dim, value_dim
     T = qkv.shape[0]
@@ -1177,7 +1202,7 @@ def gla_chunked(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seql
     _need(out.dtype == torch.float32 and out.shape == (T, H * dv) and out.is_contiguous(), "out must be contiguous float32 [tokens, H*value_dim]")
     for t, name in ((cu_seqlens, "cu_seqlens"), (start_pos, "start_pos"), (slots, "slots"), (chunks, "chunks"), (per_request, "per_request")):
         _i32(t, name)
-    planes = 1 if lower is None else 2
+    planes = 2 if lower is not None or two_terms else 1
     q_in = torch.empty((planes, T, H, dk), dtype=torch.bfloat16, device=qkv.device)
     k_end = torch.empty((planes, T, H, dk), dtype=torch.bfloat16, device=qkv.device)
     A = torch.empty((T, H, GLA_CHUNK), dtype=torch.float32, device=qkv.device)
@@ -1195,11 +1220,13 @@ def gla_chunked(qkv: torch.Tensor, z: torch.Tensor, state: torch.Tensor, cu_seql
     item, base = qkv.element_size(), qkv.data_ptr()
     f = _fn("gla", "lb_gla_chunked", [c_void_p, c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p,
                                       c_void_p, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_int, c_int,
-                                      c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_void_p])
+                                      c_float, c_float, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
+                                      c_void_p, c_int, c_int, c_void_p, c_float, c_int, c_void_p])
     _check(f(base, base + H * dk * item, base + (H * dk + keys) * item, qkv.stride(0) if T > 1 else qkv.shape[1], _ptr(z), _ptr(out),
              _ptr(state), _ptr(cu_seqlens), _ptr(start_pos), _ptr(slots), _ptr(chunks), num_chunks, _ptr(per_request), num_long,
              _ptr(q_in), _ptr(k_end), _ptr(A), _ptr(D), H, dk, dv, tau, q_scale, _ptr(segments), n_seg, _ptr(seg_state),
-             _ptr(seg_decay), _ptr(head_decay), _ptr(lower), _ptr(z_bias), T, _stream()), "gla_chunked", f"(key_dim {dk}, value_dim {dv})", launches=2 if segments is None else 4)
+             _ptr(seg_decay), _ptr(head_decay), _ptr(lower), _ptr(z_bias), T, *_gla_turn(turn, positions, T, dk), k_scale, int(two_terms),
+             _stream()), "gla_chunked", f"(key_dim {dk}, value_dim {dv})", launches=2 if segments is None else 4)
     return out
 
 
@@ -1212,18 +1239,19 @@ def gla_segmented_pays(num_tokens: int, num_long: int, num_heads: int, value_dim
     return num_tokens >= 2 * GLA_SEGMENT * GLA_CHUNK and num_long * num_heads * -(-value_dim // 32) < _SM_COUNT
 
 
-def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tensor, eps: float, num_heads: int,
+def gla_norm_gate(o: torch.Tensor, gate: torch.Tensor | None, weight: torch.Tensor | None, eps: float, num_heads: int,
                   sigmoid_gate: bool = False, out_dtype: torch.dtype | None = None) -> torch.Tensor:
     """RMSNorm of every head's float32 output with one weight [value_dim] for all heads, times silu(gate) (or, with
     `sigmoid_gate`, sigmoid(gate)); the result has the gate's dtype.  `gate` may be a column view of a wider matrix.  With
-    `num_heads` 1 it is the gated norm over the whole row.  `gate` None: the norm alone, in `out_dtype`."""
+    `num_heads` 1 it is the gated norm over the whole row.  `gate` None: the norm alone, in `out_dtype`; `weight` None: a norm
+    without a weight."""
     _cuda(o, gate, weight)
     rows, width = o.shape
     dv = width // num_heads
     _need(o.dtype == torch.float32 and o.is_contiguous() and width == num_heads * dv, "o must be contiguous float32 [rows, H*value_dim]")
     _need(gate is not None or out_dtype is not None, "without a gate the result's dtype must be given")
     _need(gate is None or (gate.shape == o.shape and gate.stride(1) == 1), "gate must match o, unit column stride")
-    _need(weight.dtype == torch.float32 and weight.shape == (dv,) and weight.is_contiguous(), "weight must be float32 [value_dim]")
+    _need(weight is None or (weight.dtype == torch.float32 and weight.shape == (dv,) and weight.is_contiguous()), "weight must be float32 [value_dim]")
     out = torch.empty((rows, width), dtype=out_dtype if gate is None else gate.dtype, device=o.device)
     f = _fn("gla", "lb_gla_norm_gate", [c_void_p, c_void_p, c_long, c_void_p, c_void_p, c_int, c_int, c_int, c_float, c_int, c_int, c_void_p])
     stride = 0 if gate is None else (gate.stride(0) if rows > 1 else gate.shape[1])
@@ -1260,24 +1288,35 @@ def latent_prepare(proj: torch.Tensor, num_heads: int, nope_dim: int, rot_dim: i
              _ptr(kr_cache), int(write_cache), int(neighbours), T, _code(proj), _stream()), "latent_prepare")
 
 
-def heads_matmul(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None) -> torch.Tensor:
+def heads_matmul(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """out[t, h, :] = a[t, h, :] @ w[h]  with a [tokens, H, K] (any token and head strides, unit stride in K), w
-    contiguous [H, K, N]; 32-bit accumulation, result in a's dtype."""
-    _cuda(a, w, out)
+    contiguous [H, K, N]; 32-bit accumulation, result in a's dtype.  `gate` (logits [tokens, H*N] in a's dtype, a column view is
+    fine): every output column is multiplied by sigmoid of its logit."""
+    _cuda(a, w, out, gate)
     T, H, Kd = a.shape
     _need(a.stride(2) == 1 and w.is_contiguous() and w.shape[:2] == (H, Kd) and w.dtype == a.dtype, "heads_matmul wants a [T, H, K] and w [H, K, N]")
     N = w.shape[2]
-    if out is None and a.dtype == torch.bfloat16 and T > SKINNY_MAX_ROWS:
+    _need(gate is None or (gate.shape == (T, H * N) and gate.dtype == a.dtype and gate.stride(1) == 1), "gate must be [T, H*N] of a's dtype")
+    g_row = 0 if gate is None else (gate.stride(0) if T > 1 else max(gate.stride(0), gate.shape[1]))
+    pairs = gate is None or (N % 2 == 0 and g_row % 2 == 0 and gate.data_ptr() % 4 == 0)      # what the gate's own kernel takes
+    if out is None and a.dtype == torch.bfloat16 and T > SKINNY_MAX_ROWS and pairs:
         # many rows: the library's batched product over the heads (as `linear` leaves its products of many rows to it);
         # the result is a [T, H, N] view of its [H, T, N] output
         product = lambda: torch.bmm(a.transpose(0, 1), w).transpose(0, 1)
-        return PROFILER.timed("library", "bmm", product) if PROFILER.enabled else product()
+        made = PROFILER.timed("library", "bmm", product) if PROFILER.enabled else product()
+        if gate is None:
+            return made
+        out = torch.empty((T, H, N), dtype=a.dtype, device=a.device)
+        f = _fn("attention_latent", "lb_column_gate", [c_void_p, c_long, c_long, c_void_p, c_long, c_void_p, c_int, c_int, c_int, c_void_p])
+        _check(f(_ptr(made), made.stride(0), made.stride(1), _ptr(gate), g_row, _ptr(out), T, H, N, _stream()), "column_gate", f"(columns {N})")
+        return out
     if out is None:
         out = torch.empty((T, H, N), dtype=a.dtype, device=a.device)
     _need(out.shape == (T, H, N) and out.stride(2) == 1 and out.dtype == a.dtype, "out must be [T, H, N]")
     f = _fn("attention_latent", "lb_heads_matmul", [c_void_p, c_long, c_long, c_void_p, c_void_p, c_long, c_long, c_int, c_int,
-                                                    c_int, c_int, c_int, c_void_p])
-    _check(f(_ptr(a), a.stride(0), a.stride(1), _ptr(w), _ptr(out), out.stride(0), out.stride(1), T, H, Kd, N, _code(a), _stream()),
+                                                    c_int, c_int, c_void_p, c_long, c_int, c_void_p])
+    _check(f(_ptr(a), a.stride(0), a.stride(1), _ptr(w), _ptr(out), out.stride(0), out.stride(1), T, H, Kd, N, _ptr(gate), g_row, _code(a),
+             _stream()),
            "heads_matmul", f"(K {Kd}, N {N})")
     return out
 
@@ -1498,6 +1537,17 @@ def gelu_tanh(x: torch.Tensor) -> torch.Tensor:
     out = torch.empty_like(x)
     f = _fn("moe", "lb_gelu_tanh", [c_void_p, c_void_p, c_long, c_int, c_void_p])
     _check(f(_ptr(x), _ptr(out), x.numel(), _code(x), _stream()), "gelu_tanh")
+    return out
+
+
+def xielu(x: torch.Tensor, factors: torch.Tensor) -> torch.Tensor:
+    """a z^2 + z/2 for z > 0, b (e^z - 1 - z) + z/2 for z <= 0, with `factors` = [a, b] (float32, on the device)."""
+    _cuda(x, factors)
+    _need(x.is_contiguous() and factors.dtype == torch.float32 and factors.shape == (2,) and factors.is_contiguous(),
+          "xielu wants a contiguous tensor and float32 factors [2]")
+    out = torch.empty_like(x)
+    f = _fn("moe", "lb_xielu", [c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
+    _check(f(_ptr(x), _ptr(out), _ptr(factors), x.numel(), _code(x), _stream()), "xielu")
     return out
 
 
@@ -1788,10 +1838,12 @@ def _rows(t: torch.Tensor | None) -> int:
     return 1 if t is None else max(t.shape[0], 1)
 
 
-def _score_extras(num_heads: int, pool: int, pooled_table, slopes, sinks, gate=None, like=None) -> None:
+def _score_extras(num_heads: int, pool: int, pooled_table, slopes, sinks, gate=None, like=None, keep: int = 0) -> None:
     """Checks of the options that the pooled-attention kernels share.  `slopes[h] * (i - j)` is taken off the scaled score of
     query i (head h) and token j; `exp(sinks[h])` joins the softmax's denominator with no key and no value; `gate` (logits of
-    `like`'s shape and dtype, a column view is fine): every output column is multiplied by sigmoid of its logit."""
+    `like`'s shape and dtype, a column view is fine): every output column is multiplied by sigmoid of its logit; `keep`: the
+    sequence's first so many tokens stay visible behind the window (without pooled blocks)."""
+    _need(keep >= 0 and (keep == 0 or pool == 0), "kept first tokens go without pooled blocks")
     _need(pool >= 0 and (pool == 0 or pooled_table is not None), "pooled blocks need their caches and table (pool 0: none)")
     for t, name in ((slopes, "slopes"), (sinks, "sinks")):
         _need(t is None or (t.is_cuda and t.dtype == torch.float32 and t.shape == (num_heads,) and t.is_contiguous()),
@@ -1808,11 +1860,11 @@ def pooled_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
                      block_table: torch.Tensor, pooled_table: torch.Tensor, token_req: torch.Tensor, positions: torch.Tensor,
                      v_table: torch.Tensor, scale: float, window: int, pool: int, token_list: torch.Tensor | None = None,
                      out: torch.Tensor | None = None, slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                     gate: torch.Tensor | None = None) -> torch.Tensor:
+                     gate: torch.Tensor | None = None, keep: int = 0) -> torch.Tensor:
     """[tokens, heads * value_dim]: attention of every (listed) token over its window's tokens and the pooled blocks
     behind it, a warp per (token, head), everything in float32; the summed values are turned back by the query's position.
     `pool` 0: no blocks (the pooled caches and their table may be None); `v_table` None: values are not rotated; `slopes`,
-    `sinks` (float32 per query head, may be None), `gate`: see `_score_extras`."""
+    `sinks` (float32 per query head, may be None), `gate`, `keep`: see `_score_extras`."""
     _cuda(q, k_cache, v_cache, kp_cache, vp_cache, block_table, pooled_table, token_req, positions, v_table, token_list)
     for t, name in ((block_table, "block_table"), (pooled_table, "pooled_table"), (token_req, "token_req"), (positions, "positions")):
         if t is not None:
@@ -1826,11 +1878,11 @@ def pooled_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tens
     n = T if token_list is None else token_list.numel()
     f = _fn("attention_pooled", "lb_pooled_attention", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                         c_void_p, c_int, c_int, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
+            + [c_float, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(token_req), _ptr(positions), _ptr(token_list), n, _ptr(v_table),
              _width(v_table), _rows(v_table), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool, _ptr(slopes),
-             _ptr(sinks), _ptr(gate), _gate_stride(gate), _code(q), _stream()), "pooled_attention", f"(dim {dim}, value dim {vdim})")
+             _ptr(sinks), _ptr(gate), _gate_stride(gate), keep, _code(q), _stream()), "pooled_attention", f"(dim {dim}, value dim {vdim})")
     return out
 
 
@@ -1863,7 +1915,7 @@ def pooled_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
                           block_table: torch.Tensor, pooled_table: torch.Tensor, cu_seqlens: torch.Tensor, start_pos: torch.Tensor,
                           positions: torch.Tensor, tiles: torch.Tensor, v_table: torch.Tensor, scale: float, window: int, pool: int,
                           out: torch.Tensor, splits: int = 1, slopes: torch.Tensor | None = None,
-                          sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+                          sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None, keep: int = 0) -> torch.Tensor:
     """The same attention for the long portions' runs of `pooled_attention_tile_q()` tokens (work list of
     `StepContext.long_portion_tiles`) on the tensor cores; writes those tokens' rows of `out` [tokens, heads * value_dim].
     With `splits` > 1 that many CTAs share a run's keys and a merge follows, which also writes the rows that no run covers
@@ -1881,11 +1933,11 @@ def pooled_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     partial = torch.empty((T, H, splits, vdim + 2), dtype=torch.float32, device=q.device) if splits > 1 else None
     f = _fn("attention_pooled", "lb_pooled_attention_tile", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                              c_void_p, c_int, c_void_p, c_int, c_int, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_void_p])
+            + [c_float, c_int, c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(cu_seqlens), _ptr(start_pos), _ptr(tiles), tiles.shape[0], _ptr(positions), T,
              _ptr(v_table), _width(v_table), _rows(v_table), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool,
-             _ptr(partial), splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), _stream()),
+             _ptr(partial), splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), keep, _stream()),
            "pooled_attention_tile", f"(dim {dim}, value dim {vdim})", launches=2 if splits > 1 else 1)
     return out
 
@@ -1905,7 +1957,7 @@ def pooled_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
                            v_table: torch.Tensor, scale: float, window: int, pool: int, splits: int,
                            token_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
                            slopes: torch.Tensor | None = None, sinks: torch.Tensor | None = None,
-                           gate: torch.Tensor | None = None) -> torch.Tensor:
+                           gate: torch.Tensor | None = None, keep: int = 0) -> torch.Tensor:
     """The attention of `pooled_attention` with every token's keys cut into `splits` ranges that run side by side and all
     query heads of a key/value head in one CTA; a merge kernel joins the ranges (two launches)."""
     _cuda(q, k_cache, v_cache, kp_cache, vp_cache, block_table, pooled_table, token_req, positions, v_table, token_list)
@@ -1922,11 +1974,77 @@ def pooled_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torc
     partial = torch.empty((n, H, splits, vdim + 2), dtype=torch.float32, device=q.device)
     f = _fn("attention_pooled", "lb_pooled_attention_split", [c_void_p] * 6 + [c_int, c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                                               c_void_p, c_int, c_int, c_void_p, c_void_p] + [c_int] * 5
-            + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_void_p])
+            + [c_float, c_int, c_int, c_int, c_void_p, c_void_p, c_void_p, c_long, c_int, c_int, c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(kp_cache), _ptr(vp_cache), _ptr(block_table), block_table.shape[1],
              _ptr(pooled_table), _width(pooled_table), _ptr(token_req), _ptr(positions), _ptr(token_list), n, _ptr(v_table),
              _width(v_table), _rows(v_table), _ptr(partial), _ptr(out), H, G, dim, vdim, k_cache.shape[1], scale, window, pool,
-             splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), _code(q), _stream()), "pooled_attention_split", f"(dim {dim}, value dim {vdim}, {splits} ranges)", launches=2)
+             splits, _ptr(slopes), _ptr(sinks), _ptr(gate), _gate_stride(gate), keep, _code(q), _stream()), "pooled_attention_split", f"(dim {dim}, value dim {vdim}, {splits} ranges)", launches=2)
+    return out
+
+
+# --------------------------------------------------------------------------- attention whose heads mix their weights
+TALK_OFFSET = 8          # floats in front of the columns of a partial result (kTalkOff of csrc/attention_pooled.cu)
+
+
+def _talk_checks(q, k_cache, v_cache, block_table, token_index, positions, talk, sinks, out) -> tuple:
+    _cuda(q, k_cache, v_cache, block_table, token_index, positions, talk, sinks, out)
+    T, H, dim = q.shape
+    G, vdim = v_cache.shape[2], v_cache.shape[3]
+    for t, name in ((block_table, "block_table"), (token_index, "token_req or cu_seqlens"), (positions, "positions or start_pos")):
+        _i32(t, name)
+    _need(q.is_contiguous() and q.dtype == k_cache.dtype == v_cache.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
+          and k_cache.shape[2:] == (G, dim), "queries must be contiguous [tokens, heads, dim] in the caches' dtype")
+    _need(talk.dtype == torch.float32 and talk.shape == (H, H) and talk.is_contiguous(), "talk must be float32 [heads, heads]")
+    _need(sinks is None or (sinks.dtype == torch.float32 and sinks.shape == (H,) and sinks.is_contiguous()), "sinks must be float32 [heads]")
+    _need(out is None or (out.shape == (T, H * vdim) and out.dtype == q.dtype and out.is_contiguous()), "out must be [tokens, heads * value_dim]")
+    return T, H, dim, G, vdim
+
+
+def talk_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, token_req: torch.Tensor,
+                         positions: torch.Tensor, talk: torch.Tensor, scale: float, window: int, keep: int, splits: int,
+                         token_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
+                         sinks: torch.Tensor | None = None) -> torch.Tensor:
+    """[tokens, heads * value_dim]: softmax attention over a window and the sequence's `keep` first tokens whose heads mix their
+    weights before they are applied: head h applies sum_g talk[h, g] w_g(i, j) to the values of its own key/value head.  exp(sinks[g])
+    joins head g's denominator and is not mixed.  Every (listed) token's keys are cut into `splits` ranges that run side by side;
+    the kernel that joins them mixes (two launches, everything in float32)."""
+    T, H, dim, G, vdim = _talk_checks(q, k_cache, v_cache, block_table, token_req, positions, talk, sinks, out)
+    if out is None:
+        out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
+    n = T if token_list is None else token_list.numel()
+    partial = torch.empty((n, H, splits, G * vdim + TALK_OFFSET), dtype=torch.float32, device=q.device)
+    f = _fn("attention_pooled", "lb_talk_attention_split", [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int] + [c_void_p] * 4 + [c_int] * 5
+            + [c_float] + [c_int] * 4 + [c_void_p])
+    _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(token_req), _ptr(positions), _ptr(token_list), n,
+             _ptr(partial), _ptr(out), _ptr(talk), _ptr(sinks), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits, _code(q), _stream()),
+           "talk_attention_split", f"(dim {dim}, value dim {vdim}, {G} key/value heads, {splits} ranges)", launches=2)
+    return out
+
+
+def talk_attention_tile_ok(q: torch.Tensor, v_cache: torch.Tensor) -> bool:
+    """Does the tensor-core form take these sizes?  bfloat16, heads of a multiple of 16 up to 128 columns, value heads of a
+    multiple of 8."""
+    return POOLED_TILE and q.dtype == torch.bfloat16 and q.shape[2] % 16 == 0 and q.shape[2] <= 128 and v_cache.shape[3] % 8 == 0
+
+
+def talk_tile_splits(num_tiles: int, num_heads: int, width: int) -> int:
+    """CTAs that share a run's keys, as `pooled_tile_splits`, where the value columns of all heads already take several."""
+    return pooled_tile_splits(num_tiles, num_heads * -(-width // 128))
+
+
+def talk_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
+                        start_pos: torch.Tensor, tiles: torch.Tensor, talk: torch.Tensor, scale: float, window: int, keep: int,
+                        out: torch.Tensor, splits: int = 1, sinks: torch.Tensor | None = None) -> torch.Tensor:
+    """`talk_attention_split` for the long portions' runs of `pooled_attention_tile_q()` tokens on the tensor cores; the rows that no
+    run covers get nothing of meaning (the caller fills them afterwards)."""
+    T, H, dim, G, vdim = _talk_checks(q, k_cache, v_cache, block_table, cu_seqlens, start_pos, talk, sinks, out)
+    _i32(tiles, "tiles")
+    partial = torch.empty((T, H, splits, G * vdim + TALK_OFFSET), dtype=torch.float32, device=q.device)
+    f = _fn("attention_pooled", "lb_talk_attention_tile", [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int] * 2 + [c_void_p] * 4 + [c_int] * 5
+            + [c_float] + [c_int] * 3 + [c_void_p])
+    _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(cu_seqlens), _ptr(start_pos), _ptr(tiles), tiles.shape[0],
+             T, _ptr(partial), _ptr(out), _ptr(talk), _ptr(sinks), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits, _stream()),
+           "talk_attention_tile", f"(dim {dim}, value dim {vdim}, {G} key/value heads)", launches=2)
     return out
 
 
@@ -2163,10 +2281,15 @@ def delta_scan_chunks(qkv: torch.Tensor, z: torch.Tensor, dt_bias: torch.Tensor,
 
 
 # --------------------------------------------------------------------------- a 32-bit stream whose sublayers all read one norm
+def _row_vector(row, H: int):
+    _need(row is None or (row.is_cuda and row.dtype == torch.float32 and row.shape == (H,) and row.is_contiguous()), "row must be float32 [width]")
+    return _ptr(row)
+
+
 def stream_add_many(x: torch.Tensor, addends, weight: torch.Tensor | None, eps: float, kind: str,
-                    act_dtype: torch.dtype) -> tuple[torch.Tensor, torch.Tensor | None]:
-    """x += sum of scale * y over `addends` (up to four pairs (y, scale), y activations of the stream's shape) in place on the
-    float32 stream, then norm(x) * weight rounded to `act_dtype` (None without a weight; kind "none": x rounded).
+                    act_dtype: torch.dtype, row: torch.Tensor | None = None) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """x += sum of scale * y over `addends` (up to four pairs (y, scale), y activations of the stream's shape), plus `row` (float32
+    [width], may be None) on every row, in place on the float32 stream, then norm(x) * weight rounded to `act_dtype` (None without a weight; kind "none": x rounded).
     Returns (x, normed)."""
     rows, H = x.shape
     ys = [y for y, _ in addends]
@@ -2177,19 +2300,20 @@ def stream_add_many(x: torch.Tensor, addends, weight: torch.Tensor | None, eps: 
         _need(y.shape == x.shape and y.dtype == act_dtype and y.is_contiguous(), "an addend must match the stream's shape")
     _need(weight is None or (weight.dtype == torch.float32 and weight.shape == (H,) and weight.is_contiguous()), "weight must be float32 [width]")
     h = None if (weight is None and kind != "none") else torch.empty((rows, H), dtype=act_dtype, device=x.device)
-    if not addends and h is None:
+    if not addends and h is None and row is None:
         return x, None
     ptrs = [_ptr(y) for y in ys] + [None] * (4 - len(ys))
     scales = [float(s) for _, s in addends] + [0.0] * (4 - len(ys))
-    f = _fn("stream_layer", "lb_stream_add_many", [c_void_p] * 5 + [c_float] * 4 + [c_int, c_void_p, c_float, c_void_p, c_int, c_int, c_int,
-                                                   c_int, c_void_p])
-    _check(f(_ptr(x), *ptrs, *scales, len(ys), _ptr(weight), eps, _ptr(h), rows, H, NORM_KINDS[kind], _DTYPE_CODE[act_dtype], _stream()),
+    f = _fn("stream_layer", "lb_stream_add_many", [c_void_p] * 5 + [c_float] * 4 + [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int,
+                                                   c_int, c_int, c_void_p])
+    _check(f(_ptr(x), *ptrs, *scales, len(ys), _row_vector(row, H), _ptr(weight), eps, _ptr(h), rows, H, NORM_KINDS[kind], _DTYPE_CODE[act_dtype], _stream()),
            "stream_add_many", f"(width {H})")
     return x, h
 
 
 def stream_add_conv_step(x: torch.Tensor, addends, weight: torch.Tensor | None, eps: float, kind: str, conv_weight: torch.Tensor,
-                         conv_state: torch.Tensor | None, slots: torch.Tensor, start_pos: torch.Tensor, act_dtype: torch.dtype) -> torch.Tensor:
+                         conv_state: torch.Tensor | None, slots: torch.Tensor, start_pos: torch.Tensor, act_dtype: torch.dtype,
+                         row: torch.Tensor | None = None) -> torch.Tensor:
     """`stream_add_many` for a decode batch (every row the single new token of its own request) whose normed rows also pass a
     short causal convolution per channel: `conv_weight` float32 [width, taps] over the request's last taps - 1 normed rows
     (`conv_state` [slots, width, taps - 1] in `act_dtype`, shifted in place; None with one tap) and this one.  Returns the
@@ -2211,9 +2335,9 @@ def stream_add_conv_step(x: torch.Tensor, addends, weight: torch.Tensor | None, 
     h = torch.empty((rows, H), dtype=act_dtype, device=x.device)
     ptrs = [_ptr(y) for y in ys] + [None] * (4 - len(ys))
     scales = [float(s) for _, s in addends] + [0.0] * (4 - len(ys))
-    f = _fn("stream_layer", "lb_stream_add_conv_step", [c_void_p] * 5 + [c_float] * 4 + [c_int, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
+    f = _fn("stream_layer", "lb_stream_add_conv_step", [c_void_p] * 5 + [c_float] * 4 + [c_int, c_void_p, c_void_p, c_float, c_void_p, c_int, c_void_p, c_void_p,
                                                         c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p])
-    _check(f(_ptr(x), *ptrs, *scales, len(ys), _ptr(weight), eps, _ptr(conv_weight), taps, _ptr(conv_state), _ptr(slots), _ptr(start_pos),
+    _check(f(_ptr(x), *ptrs, *scales, len(ys), _row_vector(row, H), _ptr(weight), eps, _ptr(conv_weight), taps, _ptr(conv_state), _ptr(slots), _ptr(start_pos),
              _ptr(h), rows, H, NORM_KINDS[kind], _DTYPE_CODE[act_dtype], _stream()), "stream_add_conv_step", f"(width {H}, {taps} taps)")
     return h
 

@@ -1,7 +1,7 @@
 from .base import MATRIX, TABLE, VECTOR, ParamSpec, Part
 from .context import Runtime, StepContext
 from .norm import LayerNorm, RMSNorm
-from .rope import RampRotaryEmbedding, RotaryEmbedding, inverse_frequencies, ramp_frequencies
+from .rope import LinearRotaryEmbedding, RampRotaryEmbedding, RotaryEmbedding, inverse_frequencies, ramp_frequencies
 from .attention import Attention
 from .mamba2 import Mamba2
 from .mlp import GatedMLP
@@ -18,8 +18,10 @@ from .moe import GLU
 from .mamba import Mamba
 from .hgrn2 import HGRN2
 from .gated_attention import GatedAttention
-from .embedding import BareLMHead, Embedding, LMHead, NormedEmbedding, PairEmbedding, StreamEmbedding
-from .block import ParallelStreamBlock, PostNormBlock, PreNormParallelBlock, PreNormStreamBlock, StreamInput, TokenSideInput, OutNormStreamBlock, InputConv, StreamAdd
+from .talking_attention import TalkingAttention
+from .retention import Retention
+from .embedding import BareLMHead, Embedding, LMHead, NormedEmbedding, PairEmbedding, SoftcapLMHead, StreamEmbedding
+from .block import ParallelStreamBlock, PostNormBlock, PreNormParallelBlock, PreNormStreamBlock, StreamInput, TokenSideInput, OutNormStreamBlock, InputConv, StreamAdd, StreamVector
 
 __all__ = ["MATRIX", "TABLE", "VECTOR", "ParamSpec", "Part", "Runtime", "StepContext", "RMSNorm",
            "RotaryEmbedding", "inverse_frequencies", "Attention", "Mamba2", "GatedMLP", "Embedding", "LMHead",
@@ -27,4 +29,5 @@ __all__ = ["MATRIX", "TABLE", "VECTOR", "ParamSpec", "Part", "Runtime", "StepCon
            "PairEmbedding", "BareLMHead", "LayerNorm", "MinGRU", "PooledWindowAttention", "ClampedGLU", "NormedEmbedding",
            "PreNormStreamBlock", "TokenSideInput", "ChannelDelta", "LightningAttention", "MixerPair", "SinkAttention", "GLU",
            "StreamEmbedding", "ParallelStreamBlock", "StreamInput", "GatedDelta", "ConvAttention", "OutNormStreamBlock",
-           "RampRotaryEmbedding", "ramp_frequencies", "Mamba", "HGRN2", "GatedAttention", "InputConv", "StreamAdd"]
+           "RampRotaryEmbedding", "ramp_frequencies", "Mamba", "HGRN2", "GatedAttention", "InputConv", "StreamAdd",
+           "TalkingAttention", "Retention", "LinearRotaryEmbedding", "SoftcapLMHead", "StreamVector"]

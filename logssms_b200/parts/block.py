@@ -392,6 +392,9 @@ class PreNormStreamBlock(Part):
                 raise ValueError("prenorm_stream blocks need norms with a form on a 32-bit stream (`norm_kind`)")
         self.side = None if spec.side is None else TokenSideInput(spec.side, perturb_init, shared)
         self.input_conv = InputConv(spec.mixer_norm.size, spec.input_conv) if getattr(spec, "input_conv", 0) else None
+        self.residual_scale = float(getattr(spec, "residual_scale", 1.0))
+        if self.residual_scale != 1.0 and (spec.layer_scale or spec.side is not None):
+            raise ValueError("a residual scale goes without layer scales and side input")
         self._plain = not spec.layer_scale and spec.side is None        # nothing but sums between the sublayers
         self.joins_opening = self._plain      # forward() adds `ctx.extras["next_addend"]` to the stream as it closes the block
         self._jitter = 0.3 if perturb_init else 0.0
@@ -455,8 +458,8 @@ class PreNormStreamBlock(Part):
         scale = self.scale_mixer
         if self.feed_forward is not None:
             n = self.ff_norm
-            if isinstance(y, list):
-                _, h = K.stream_add_many(stream, y, n.weight, n.eps, n.norm_kind, act)
+            if isinstance(y, list) or self.residual_scale != 1.0:
+                _, h = K.stream_add_many(stream, _addends(y, self.residual_scale), n.weight, n.eps, n.norm_kind, act)
             else:
                 _, h = K.stream_add_norm(stream, y, scale, n.weight, n.eps, n.norm_kind, act)
             with nvtx_range(self.spec.feed_forward.kind):
@@ -481,21 +484,25 @@ class PreNormStreamBlock(Part):
     def _close(self, stream, y, nxt, ctx, act):
         """x += what is left (each with a scalar), then what the next block reads: its norm, and in a decode step its input
         convolution."""
-        joins = _addends(y)
+        joins, row = _addends(y, self.residual_scale), None
         if ctx.extras.get("next_addend") is not None:
-            joins.append(ctx.extras["next_addend"])
+            rows, scale = ctx.extras["next_addend"]
+            if rows.dim() == 1:                 # one vector for every row
+                row = rows
+            else:
+                joins.append((rows, scale))
         while len(joins) > 4:
             K.stream_add_many(stream, joins[:4], None, 0.0, "rmsnorm", act)
             joins = joins[4:]
         if nxt is None:
-            K.stream_add_many(stream, joins, None, 0.0, "rmsnorm", act)
+            K.stream_add_many(stream, joins, None, 0.0, "rmsnorm", act, row=row)
             return K.StreamRows(stream, stream.new_empty((0, stream.shape[1]), dtype=act))
         conv, layer = ctx.extras.get("next_input_conv") or (None, None)
         if conv is not None and ctx.max_len == 1:
             h = K.stream_add_conv_step(stream, joins, nxt.weight, nxt.eps, nxt.norm_kind, conv.weight, conv.state(ctx, layer), ctx.slots,
-                                       ctx.start_pos, act)
+                                       ctx.start_pos, act, row=row)
             return K.StreamRows(stream, h, normed_by=nxt, convolved=True)
-        _, h = K.stream_add_many(stream, joins, nxt.weight, nxt.eps, nxt.norm_kind, act)
+        _, h = K.stream_add_many(stream, joins, nxt.weight, nxt.eps, nxt.norm_kind, act, row=row)
         return K.StreamRows(stream, h, normed_by=nxt)
 
 
@@ -517,7 +524,7 @@ class StreamInput(Part):
     def bind(self, t):
         self.weight = t[""]
 
-    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0):
+    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0, turn: int = 0):
         if not isinstance(x, K.StreamRows):
             raise ValueError("a stream input mixes a 32-bit stream (`StreamRows`) with the rows it began as")
         if x0_scale != 1.0:
@@ -535,14 +542,45 @@ class StreamAdd(Part):
     def __init__(self, spec, perturb_init: bool = False):
         self.spec = spec
 
-    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0):
+    def addend(self, x0: torch.Tensor, x0_scale: float, turn: int):
+        """What a block that closes with `joins_opening` adds: (rows, scale), or (one float32 vector for every row, 1)."""
+        return x0, x0_scale
+
+    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0, turn: int = 0):
         if not isinstance(x, K.StreamRows):
             raise ValueError("the embedding's output is added to a 32-bit stream (`StreamRows`)")
         K.stream_add_many(x.f32, [(x0, x0_scale)], None, 0.0, "rmsnorm", x0.dtype)
         return K.StreamRows(x.f32, x0[:0])
 
 
-STREAM_INPUTS = {"product": StreamInput, "add": StreamAdd}
+class StreamVector(Part):
+    """x <- x + b_turn on a 32-bit stream, the same vector for every row: row `turn` of a table [count, width] stored at the
+    model's root.  A block that closes with `joins_opening` does it in its closing kernel instead."""
+    kernels = ("stream_layer",)
+    is_addend = True
+
+    def __init__(self, spec, perturb_init: bool = False):
+        self.spec = spec
+        self.table = None
+
+    def param_specs(self):
+        from .base import VECTOR, ParamSpec, normal_init
+        return {"": ParamSpec((self.spec.count, self.spec.hidden_size), VECTOR, normal_init(0.5))}
+
+    def bind(self, t):
+        self.table = t[""].contiguous()
+
+    def addend(self, x0: torch.Tensor, x0_scale: float, turn: int):
+        return self.table[turn], 1.0
+
+    def forward(self, x, x0: torch.Tensor, x0_scale: float = 1.0, turn: int = 0):
+        if not isinstance(x, K.StreamRows):
+            raise ValueError("a vector per pass is added to a 32-bit stream (`StreamRows`)")
+        K.stream_add_many(x.f32, [], None, 0.0, "rmsnorm", x0.dtype, row=self.table[turn])
+        return K.StreamRows(x.f32, x0[:0])
+
+
+STREAM_INPUTS = {"product": StreamInput, "add": StreamAdd, "vector": StreamVector}
 
 
 def _addends(y, scale: float = 1.0) -> list:

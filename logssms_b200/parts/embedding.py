@@ -149,3 +149,15 @@ class LMHead(Part):
 class BareLMHead(LMHead):
     """The same head whose matrix is stored under the head's prefix itself (`head`, not `head.weight`)."""
     param_name = ""
+
+
+@HEADS.register("lm_head_softcap")
+class SoftcapLMHead(LMHead):
+    """logits <- cap * tanh(logits / cap) on the head's float32 logits."""
+
+    def __init__(self, vocab_size: int, hidden_size: int, multiplier: float, tied_to, *, cap: float):
+        super().__init__(vocab_size, hidden_size, multiplier, tied_to)
+        self.cap = float(cap)
+
+    def forward(self, h: torch.Tensor) -> torch.Tensor:
+        return K.softcap(super().forward(h), self.cap)

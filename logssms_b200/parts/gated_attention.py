@@ -17,7 +17,8 @@ class GatedAttention(Part):
     j reads key/value head j // (heads / kv_heads).  `qk_norm` "row": q and k are each RMS-normed over their whole row (all heads
     at once, a weight per column); "head_unit": each head's columns are divided by their root mean square, without a weight, after
     the rotation (which does not change it).  `position`: rotation in halves over every head's first `rotary_dim` columns.
-    Scores times `softmax_scale`; position i sees j with 0 <= i - j < window (None: every j <= i); with `sink_zero` the softmax's
+    Scores times `softmax_scale`; position i sees j with 0 <= i - j < window (None: every j <= i), and with `keep_first` the
+    sequence's first so many tokens; with `sink_zero` the softmax's
     denominator holds one more term exp(0) without key or value.  The heads' outputs are multiplied element by element with
     sigmoid(W_g h), then the output projection.
 
@@ -66,7 +67,7 @@ class GatedAttention(Part):
 
     def cache_needs(self) -> CacheNeeds:
         s = self.spec
-        return CacheNeeds(kv=KVNeed(s.num_kv_heads, s.head_dim, s.window, s.value_dim))
+        return CacheNeeds(kv=KVNeed(s.num_kv_heads, s.head_dim, s.window, s.value_dim, s.keep_first))
 
     def forward(self, x: torch.Tensor, ctx, cache_layer: int, writes_cache: bool = True) -> torch.Tensor:
         s = self.spec
@@ -79,8 +80,8 @@ class GatedAttention(Part):
         q = K.qk_prepare(proj[:, :rows], H, G, s.head_dim, s.value_dim, ctx.positions, ctx.slot_mappings[gi], self.position.table, norm,
                          self.q_norm, self.k_norm, s.norm_eps, k_cache, v_cache, writes_cache)
         table = ctx.block_tables[gi]
-        extras = {"slopes": None, "sinks": self.sinks, "gate": proj[:, rows:]}
-        most_keys = min(window, ctx.max_context)
+        extras = {"slopes": None, "sinks": self.sinks, "gate": proj[:, rows:], "keep": s.keep_first}
+        most_keys = min(window + s.keep_first, ctx.max_context)
 
         def few_rows(token_list=None, out=None, n=x.shape[0]):
             # decoded tokens and short portions: key ranges side by side where the sizes allow, else a warp per (token, head)

@@ -9,6 +9,30 @@ from ..registry import MIXERS
 from .base import MATRIX, VECTOR, ParamSpec, Part, normal_init, ones_init
 
 
+def step_recurrence(ctx, qkv: torch.Tensor, z: torch.Tensor | None, state: torch.Tensor, sizes: tuple, *, two_terms: bool = False,
+                    **options) -> torch.Tensor:
+    """The gated-linear-attention recurrence over one step's batch: float32 [tokens, heads * value_dim], states updated in place.
+    `sizes`: (heads, key_dim, value_dim, tau, query scale); `options` and `two_terms`: see `K.gla_scan`, `K.gla_chunked`.  Long
+    portions of a bfloat16 engine run in chunks on the tensor cores (a lone prompt's segments side by side instead of one CTA
+    walking each), decoded tokens and short portions, which are other requests and other rows, token by token."""
+    H, dk, dv = sizes[:3]
+    if not (ctx.has_long_portions and K.gla_chunked_ok(qkv, dk)):
+        return K.gla_scan(qkv, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes, **options)
+    chunks, n_chunks, per_request, n_long = ctx.long_portion_chunks(K.GLA_CHUNK)
+    _, _, short_list, n_short = ctx.requests_by_portion()
+    o = torch.empty((qkv.shape[0], H * dv), dtype=torch.float32, device=qkv.device)
+    seg = {}
+    if K.gla_segmented_pays(ctx.num_tokens, n_long, H, dv):
+        segments, _, seg_requests, _ = ctx.long_portion_segments(K.GLA_CHUNK, K.GLA_SEGMENT)
+        seg = {"segments": segments, "segment_requests": seg_requests}
+    K.gla_chunked(qkv, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, chunks, n_chunks, per_request, n_long, *sizes, out=o,
+                  two_terms=two_terms, **options, **seg)
+    if n_short > 0:
+        K.gla_scan(qkv, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes, request_list=short_list, out=o,
+                   **options)
+    return o
+
+
 @MIXERS.register("gla")
 class GatedLinearAttention(Part):
     """q, k [heads, key_dim], v, g [heads, value_dim] from the input h; z = a2 (a1 h) + a2.b gives the decay
@@ -66,23 +90,6 @@ class GatedLinearAttention(Part):
         z = K.linear(low, self.a2_w, self.a2_b, out_f32=True)
         state = ctx.cache.states[cache_layer]["gla"]
         sizes = (s.num_heads, s.key_dim, s.value_dim, s.tau, s.key_dim ** -0.5)
-        if ctx.has_long_portions and K.gla_chunked_ok(proj, s.key_dim):
-            # long portions in chunks on the tensor cores; decoded tokens and short portions (other requests, other rows
-            # of o) token by token
-            chunks, n_chunks, per_request, n_long = ctx.long_portion_chunks(K.GLA_CHUNK)
-            _, _, short_list, n_short = ctx.requests_by_portion()
-            o = torch.empty((x.shape[0], vg), dtype=torch.float32, device=x.device)
-            seg = {}
-            if K.gla_segmented_pays(ctx.num_tokens, n_long, s.num_heads, s.value_dim):
-                # few long portions (a lone prompt): their segments side by side instead of one CTA walking each
-                segments, _, seg_requests, _ = ctx.long_portion_segments(K.GLA_CHUNK, K.GLA_SEGMENT)
-                seg = {"segments": segments, "segment_requests": seg_requests}
-            K.gla_chunked(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, chunks, n_chunks, per_request, n_long,
-                          *sizes, out=o, **seg)
-            if n_short > 0:
-                K.gla_scan(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes,
-                           request_list=short_list, out=o)
-        else:
-            o = K.gla_scan(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes)
+        o = step_recurrence(ctx, proj, z, state, sizes)
         y = K.gla_norm_gate(o, proj[:, 2 * qk + vg: 2 * qk + 2 * vg], self.norm_w, s.norm_eps, s.num_heads)
         return K.linear(y, self.o_w)

@@ -7,6 +7,7 @@ from ..cache import CacheNeeds, StateNeed
 from ..ops import kernels as K
 from ..registry import MIXERS
 from .base import MATRIX, VECTOR, ParamSpec, Part, normal_init, ones_init
+from .gla import step_recurrence
 
 
 @MIXERS.register("hgrn2")
@@ -58,23 +59,5 @@ class HGRN2(Part):
         proj = K.linear(x, self.in_w)                                     # q | v
         z = K.linear_f32(x, self.f_w)
         state = ctx.cache.states[cache_layer]["hgrn2"]
-        sizes = (H, dk, dv, 1.0, 1.0)
-        gate = {"lower": self.lower, "z_bias": self.f_b}
-        if ctx.has_long_portions and K.gla_chunked_ok(proj, dk):
-            # long portions in chunks on the tensor cores; decoded tokens and short portions (other requests, other rows
-            # of o) token by token
-            chunks, n_chunks, per_request, n_long = ctx.long_portion_chunks(K.GLA_CHUNK)
-            _, _, short_list, n_short = ctx.requests_by_portion()
-            o = torch.empty((x.shape[0], H * dv), dtype=torch.float32, device=x.device)
-            seg = {}
-            if K.gla_segmented_pays(ctx.num_tokens, n_long, H, dv):
-                segments, _, seg_requests, _ = ctx.long_portion_segments(K.GLA_CHUNK, K.GLA_SEGMENT)
-                seg = {"segments": segments, "segment_requests": seg_requests}
-            K.gla_chunked(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, chunks, n_chunks, per_request, n_long,
-                          *sizes, out=o, **gate, **seg)
-            if n_short > 0:
-                K.gla_scan(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes,
-                           request_list=short_list, out=o, **gate)
-        else:
-            o = K.gla_scan(proj, z, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes, **gate)
+        o = step_recurrence(ctx, proj, z, state, (H, dk, dv, 1.0, 1.0), lower=self.lower, z_bias=self.f_b)
         return K.linear(K.gla_norm_gate(o, None, self.norm_w, s.norm_eps, H, out_dtype=x.dtype), self.o_w)

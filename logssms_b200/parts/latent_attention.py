@@ -23,7 +23,8 @@ class LatentAttention(Part):
 
     Options of the spec: `pairing` "neighbours" rotates columns (2i, 2i + 1) instead of (i, i + n/2); `sink`: exp(sink_h), a
     stored number per head, joins the softmax's denominator with no key and no value (tensor sink); `head_gate`: a head's
-    output is multiplied by sigmoid((W_g h)_h) (tensor g, its rows ride in the input product); `own_latents` False: the layer
+    output is multiplied by sigmoid((W_g h)_h) (tensor g, its rows ride in the input product); `column_gate`: the same with one
+    gate per column of every head's output, applied in the fold through W_uv; `own_latents` False: the layer
     has no dkv and no dkv.norm, and reads the latents and rotated key parts that another layer stored in the cache layer the
     schedule gives it (with `writes_cache=False`)."""
     kernels = ("attention_latent", "attention_pooled", "rope", "linear_skinny", "gemm_tcgen05")
@@ -43,6 +44,8 @@ class LatentAttention(Part):
                     shared[key] = self.position
         if spec.pairing not in ("halves", "neighbours"):
             raise ValueError("the rotation pairs halves or neighbours")
+        if spec.head_gate and spec.column_gate:
+            raise ValueError("a latent attention has a gate per head or per column, not both")
         self.in_w = self.norm_w = self.uk = self.uv_t = self.o_w = self.sinks = None
 
     def param_specs(self):
@@ -60,14 +63,14 @@ class LatentAttention(Part):
             specs["dkv.norm"] = ParamSpec((s.kv_rank,), VECTOR, ones_init(self._jitter))
         if s.sink:
             specs["sink"] = ParamSpec((s.num_heads,), VECTOR, normal_init(1.0))
-        if s.head_gate:
-            specs["g"] = ParamSpec((s.num_heads, s.hidden_size), MATRIX, fan)
+        if s.head_gate or s.column_gate:
+            specs["g"] = ParamSpec((s.num_heads * (s.value_dim if s.column_gate else 1), s.hidden_size), MATRIX, fan)
         return specs
 
     def bind(self, t):
         s = self.spec
         # rows of the one input product: queries | down-projection (a layer with latents of its own) | gate logits
-        self.in_w = torch.cat([t["q"]] + ([t["dkv"]] if s.own_latents else []) + ([t["g"]] if s.head_gate else []), 0).contiguous()
+        self.in_w = torch.cat([t["q"]] + ([t["dkv"]] if s.own_latents else []) + ([t["g"]] if "g" in t else []), 0).contiguous()
         self.norm_w, self.o_w, self.sinks = t.get("dkv.norm"), t["o"], t.get("sink")
         self.uk = t["uk"].view(s.num_heads, s.nope_dim, s.kv_rank).contiguous()                       # [H, K = nope, N = rank]
         self.uv_t = t["uv"].view(s.num_heads, s.value_dim, s.kv_rank).transpose(1, 2).contiguous()     # [H, K = rank, N = value]
@@ -115,7 +118,7 @@ class LatentAttention(Part):
             qa = qa if qa.is_contiguous() else qa.contiguous()
             lat = K.latent_attention(qa, q[:, :, s.nope_dim:], c_cache, kr_cache, ctx.block_tables[gi], ctx.token_req,
                                      ctx.positions, s.softmax_scale, s.window or 0, sinks=self.sinks)
-        o = K.heads_matmul(lat, self.uv_t)                                 # [T, H, value]
+        o = K.heads_matmul(lat, self.uv_t, gate=proj[:, own:] if s.column_gate else None)      # [T, H, value]
         o = o.reshape(T, H * s.value_dim)
         if s.head_gate:
             K.head_gate(o, proj[:, own:], H)

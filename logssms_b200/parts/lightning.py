@@ -7,6 +7,7 @@ from ..cache import CacheNeeds, StateNeed
 from ..ops import kernels as K
 from ..registry import MIXERS
 from .base import MATRIX, VECTOR, ParamSpec, Part, normal_init, ones_init
+from .gla import step_recurrence
 
 
 @MIXERS.register("lightning_attention")
@@ -57,23 +58,6 @@ class LightningAttention(Part):
         qk, vv = H * dk, H * dv
         proj = K.silu_columns(K.linear(x, self.in_w), 2 * qk + vv)        # silu(q | k | v) | gate
         state = ctx.cache.states[cache_layer]["lightning"]
-        sizes = (H, dk, dv, 1.0, 1.0)
-        if ctx.has_long_portions and K.gla_chunked_ok(proj, dk):
-            # long portions in chunks on the tensor cores; decoded tokens and short portions token by token
-            chunks, n_chunks, per_request, n_long = ctx.long_portion_chunks(K.GLA_CHUNK)
-            _, _, short_list, n_short = ctx.requests_by_portion()
-            o = torch.empty((x.shape[0], vv), dtype=torch.float32, device=x.device)
-            seg = {}
-            if K.gla_segmented_pays(ctx.num_tokens, n_long, H, dv):
-                segments, _, seg_requests, _ = ctx.long_portion_segments(K.GLA_CHUNK, K.GLA_SEGMENT)
-                seg = {"segments": segments, "segment_requests": seg_requests}
-            K.gla_chunked(proj, None, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, chunks, n_chunks, per_request, n_long,
-                          *sizes, out=o, head_decay=self.decay, **seg)
-            if n_short > 0:
-                K.gla_scan(proj, None, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes,
-                           request_list=short_list, out=o, head_decay=self.decay)
-        else:
-            o = K.gla_scan(proj, None, state, ctx.cu_seqlens, ctx.start_pos, ctx.slots, ctx.num_requests, *sizes,
-                           head_decay=self.decay)
+        o = step_recurrence(ctx, proj, None, state, (H, dk, dv, 1.0, 1.0), head_decay=self.decay)
         y = K.gla_norm_gate(o, proj[:, 2 * qk + vv:], self.norm_w, s.norm_eps, 1, sigmoid_gate=True)
         return K.linear(y, self.o_w)

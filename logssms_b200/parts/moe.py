@@ -10,28 +10,35 @@ from .base import MATRIX, VECTOR, ParamSpec, Part, normal_init
 
 @FEED_FORWARDS.register("dense_mlp")
 class DenseMLP(Part):
-    """down(act(up(x))) with the tanh form of GELU.  Tensors: up, down."""
+    """down(act(up(x))), act the tanh form of GELU, or "xielu": softplus(p) z^2 + z/2 for z > 0, (1/2 + softplus(q)) (e^z - 1 - z) +
+    z/2 for z <= 0 with two stored numbers (p, q), whose factors are made once, when they arrive.  Tensors: up, down; act."""
     kernels = ("moe", "linear_skinny", "gemm_tcgen05")
 
     def __init__(self, spec, perturb_init: bool = False, shared: dict | None = None):
-        if spec.activation != "gelu_tanh":
-            raise ValueError(f"dense_mlp knows the activation gelu_tanh, not {spec.activation!r}")
+        if spec.activation not in ("gelu_tanh", "xielu"):
+            raise ValueError(f"dense_mlp knows the activations gelu_tanh and xielu, not {spec.activation!r}")
         self.spec = spec
-        self.up = self.down = None
+        self.up = self.down = self.factors = None
 
     def param_specs(self):
         s = self.spec
-        return {"up": ParamSpec((s.intermediate_size, s.hidden_size), MATRIX, normal_init(s.hidden_size ** -0.5)),
-                "down": ParamSpec((s.hidden_size, s.intermediate_size), MATRIX, normal_init(2.0 * s.intermediate_size ** -0.5))}
+        specs = {"up": ParamSpec((s.intermediate_size, s.hidden_size), MATRIX, normal_init(s.hidden_size ** -0.5)),
+                 "down": ParamSpec((s.hidden_size, s.intermediate_size), MATRIX, normal_init(2.0 * s.intermediate_size ** -0.5))}
+        if s.activation == "xielu":
+            specs["act"] = ParamSpec((2,), VECTOR, normal_init(0.7))
+        return specs
 
     def bind(self, t):
         self.up, self.down = t["up"], t["down"]
+        if self.spec.activation == "xielu":
+            self.factors = (torch.nn.functional.softplus(t["act"].double()) + torch.tensor([0.0, 0.5], device=t["act"].device)).float().contiguous()
 
     def setup(self, rt) -> None:
         pass
 
     def forward(self, x: torch.Tensor):
-        return K.linear(K.gelu_tanh(K.linear(x, self.up)), self.down)
+        z = K.linear(x, self.up)
+        return K.linear(K.gelu_tanh(z) if self.factors is None else K.xielu(z, self.factors), self.down)
 
 
 @FEED_FORWARDS.register("clamped_glu")

@@ -93,6 +93,18 @@ class RampRotaryEmbedding(RotaryEmbedding):
         return ramp_frequencies(self.spec.rotary_dim, self.spec.theta, self.spec.scaling)
 
 
+@POSITION_ENCODINGS.register("rope_linear")
+class LinearRotaryEmbedding(RotaryEmbedding):
+    """The same table with every frequency theta^(-2i/n) divided by the number `factor` of `spec.scaling` (None: plain
+    frequencies); worked out in float64, handed on as float32."""
+
+    def frequencies(self) -> tuple[torch.Tensor, float]:
+        n, scaling = self.spec.rotary_dim, dict(self.spec.scaling or ())
+        factor = float(scaling.get("factor", 1.0))
+        f = torch.tensor([self.spec.theta ** (-2.0 * i / n) / factor for i in range(n // 2)], dtype=torch.float64)
+        return f.to(torch.float32), 1.0
+
+
 class NoPositionEncoding(Part):
     """Stand-in for attention without rotation: an empty table (rotary_dim 0)."""
 
