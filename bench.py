@@ -866,8 +866,38 @@ DIMUDRA_SIZES = {
     "w1024": (_dimudra_config(1024, 8, 2, 64, 128, 1024, 16, 8, 2, 1024, 1024, 32768), PUPOPEL_SIZES["w1024"][0]),
     "w2048": (_dimudra_config(2048, 16, 4, 128, 128, 2048, 16, 16, 4, 1408, 1408, 65536), PUPOPEL_SIZES["w2048"][0]),
 }
+
+
+def _fosupel_config(width: int, heads: int, kv_heads: int, key_dim: int, value_dim: int, window: int, keep: int, kv_rank: int, rot: int,
+                    experts: int, top: int, expert_ff: int, shared_ff: int, dense_ff: int, vocab: int) -> dict:
+    """Layer sizes that resemble a real model's: three pairs of attention over a window (and kept first tokens) with mixed weights
+    and retention to one attention over cached latents, routed feed-forwards with a gated shared expert and one dense one in
+    front; a loop of one pass (the closest model's layers run once too)."""
+    rotation = {"base": 10000.0, "dims": key_dim // 2}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": key_dim, "vdim": key_dim, "scale": key_dim ** -0.5,
+            "mask": {"size": window, "keep_first": keep}, "rot": {**rotation, "scaling": {"factor": 4.0}}}
+    right = {"heads": heads, "dim": key_dim, "vdim": value_dim, "rot": rotation,
+             "decay": [1.0 - 2.0 ** (-5 - 5 * h / max(heads - 1, 1)) for h in range(heads)]}
+    pair = {"type": "parallel", "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}}
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": heads, "dim": key_dim, "rot_dim": rot, "vdim": key_dim, "kv_rank": kv_rank,
+                        "rot": {"base": 10000.0, "dims": rot}, "scale": (key_dim + rot) ** -0.5}}
+    moe = {"kind": "moe", "expert": {"ff": expert_ff}, "router": {"experts": experts, "top": top}, "shared": {"ff": shared_ff}}
+    layers = [{**pair, "mlp": {"kind": "dense", "ff": dense_ff}}, {**pair, "mlp": moe}, {**latent, "mlp": moe}, {**pair, "mlp": moe}]
+    return {"architecture": "Fosupel", "layers": layers, "loop": {"start": 1, "stop": 3, "times": 1}, "norm": {"eps": 1e-5},
+            "residual_mult": 0.5, "logit_softcap": 30.0, "vocab": vocab, "width": width}
+
+
+# Fosupel beside Pupopel (the closest existing model: a 32-bit stream, a pair of softmax attention with a sink and linear attention
+# with a fixed decay on the same kernels, routed feed-forwards with a shared expert and one dense one in front) at the same width,
+# depth, vocabulary, head, expert and dense sizes; its latent attention is Dudurax's and Zarisun's kernel
+FOSUPEL_SIZES = {
+    "w1024": (_fosupel_config(1024, 8, 2, 64, 128, 1024, 64, 256, 32, 8, 2, 1024, 1024, 2048, 32768), PUPOPEL_SIZES["w1024"][0]),
+    "w2048": (_fosupel_config(2048, 16, 4, 128, 128, 2048, 64, 512, 64, 16, 4, 1408, 1408, 8192, 65536), PUPOPEL_SIZES["w2048"][0]),
+}
 DESIGNS = {"dudurax": (DESIGN_SIZES, "falcon_h1"), "kuvazen": (KUVAZEN_SIZES, "dudurax"), "pupopel": (PUPOPEL_SIZES, "dudurax"),
-           "zarisun": (ZARISUN_SIZES, "pupopel"), "dimudra": (DIMUDRA_SIZES, "pupopel")}
+           "zarisun": (ZARISUN_SIZES, "pupopel"), "dimudra": (DIMUDRA_SIZES, "pupopel"),
+           "fosupel": (FOSUPEL_SIZES, "pupopel")}
 
 
 def _design_point(cfg: dict, vocab: int, K: int, W: int, batch: int, context: int) -> dict:
@@ -940,7 +970,7 @@ def _design_point(cfg: dict, vocab: int, K: int, W: int, batch: int, context: in
 
 def run_design(args) -> dict:
     """`--design NAME`: that design at a few layer sizes beside the closest existing model at the same width and depth
-    (Dudurax beside Falcon-H1, Kuvazen and Pupopel beside Dudurax, Zarisun and Dimudra beside Pupopel)."""
+    (Dudurax beside Falcon-H1, Kuvazen and Pupopel beside Dudurax, Zarisun, Dimudra and Fosupel beside Pupopel)."""
     table, beside = DESIGNS[args.design]
     sizes = {}
     for name, (new, closest) in table.items():
@@ -1001,7 +1031,7 @@ def main() -> int:
     ap.add_argument("--reference-timeout", type=int, default=900, help="seconds the reference arm may take")
     ap.add_argument("--probe", choices=["decode", "prefill", "mixed"], default=None,
                     help="a short run of one kind of step for a profiler (see profiles/); prints no benchmark line")
-    ap.add_argument("--design", choices=["dudurax", "kuvazen", "pupopel", "zarisun", "dimudra"], default=None,
+    ap.add_argument("--design", choices=["dudurax", "kuvazen", "pupopel", "zarisun", "dimudra", "fosupel"], default=None,
                     help="prefill and decode of another design at a few layer sizes beside the closest existing model "
                          "(one JSON line of its own; the default workload is untouched)")
     args = ap.parse_args()

@@ -31,8 +31,8 @@
 //   pooled_attention_tile : bfloat16 prompt portions on the tensor cores: a CTA per (run of up to 64 neighbouring tokens
 //                           of a request, query head); the keys the run sees go through shared memory once for all
 //                           its queries (described at the kernel)
-//   talk_merge            : attention whose heads mix their softmax weights before they are applied to the values: the two
-//                           kernels above sum every head's weights over ALL key/value heads' values, and this one mixes
+//   talk_merge            : attention whose heads mix their softmax weights before they are applied to the values: an attention
+//                           kernel sums every head's weights over ALL key/value heads' values, and this one mixes
 //                           (described at the kernel)
 #include "lb200/common.cuh"
 using namespace lb200;
@@ -635,15 +635,12 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         int table_width, const int* __restrict__ pooled_table, int pooled_width, const int* __restrict__ cu,
         const int* __restrict__ start_pos, const int* __restrict__ tiles, const float* __restrict__ v_table, int v_rot,
         int table_rows, __nv_bfloat16* __restrict__ out, int Hq, int Hkv, int dim, int vdim, int page_size, float scale,
-        int window, int pool, float* __restrict__ partial, int splits, ScoreExtras extras, ValueSpan span) {
+        int window, int pool, float* __restrict__ partial, int splits, ScoreExtras extras) {
     extern __shared__ __align__(16) unsigned char tile_smem[];
     const int b = tiles[2 * blockIdx.x];
     if (b < 0) return;
     const int t0 = tiles[2 * blockIdx.x + 1];
-    const int head = blockIdx.y % Hq, g = head / (Hq / Hkv);
-    const int v_row = span.width > 0 ? span.width : Hkv * vdim;     // value elements of a token
-    const int v_col = span.width > 0 ? (blockIdx.y / Hq) * vdim : g * vdim;
-    const int cols = span.width > 0 ? min(vdim, span.width - v_col) : vdim;
+    const int head = blockIdx.y, g = head / (Hq / Hkv);
     const int keep = extras.keep;
     const int n_q = min(kTileQ, cu[b + 1] - cu[b] - t0);
     const int row0 = cu[b] + t0, pos0 = start_pos[b] + t0;
@@ -658,7 +655,7 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
     __nv_bfloat16* Ks0 = reinterpret_cast<__nv_bfloat16*>(tile_smem);
     __nv_bfloat16* Vs0 = Ks0 + 2 * kTileK * k_stride;
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, gq = lane >> 2, tq = lane & 3;
-    const int dsteps = dim / 16, vtiles = cols / 8;
+    const int dsteps = dim / 16, vtiles = vdim / 8;
     const int* pages = block_table + (size_t)b * table_width;
     const int* pooled_pages = pooled_table + (size_t)b * pooled_width;
 
@@ -702,9 +699,9 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         long row = -1;
         bool pooled = false;
         if (kk < keys) row = key_row(kk, blocks, first, pages, pooled_pages, page_size, pooled);
-        const int n = is_v ? cols : dim;
+        const int n = is_v ? vdim : dim;
         const __nv_bfloat16* src = is_v ? (pooled ? vp_cache : v_cache) : (pooled ? kp_cache : k_cache);
-        if (row >= 0) src += is_v ? (size_t)row * v_row + v_col : ((size_t)row * Hkv + g) * dim;
+        if (row >= 0) src += ((size_t)row * Hkv + g) * n;
         __nv_bfloat16* dst = is_v ? Vs0 + ((size_t)buf * kTileK + r) * v_stride : Ks0 + ((size_t)buf * kTileK + r) * k_stride;
         const uint32_t dst_addr = (uint32_t)__cvta_generic_to_shared(dst);
         const int bytes = row >= 0 ? 16 : 0;
@@ -810,19 +807,17 @@ __global__ void __launch_bounds__(kTileThreads) pooled_attention_tile_kernel(
         }
     }
     if (partial != nullptr) {
-        float* p_lo = partial + (((size_t)(row0 + r_lo) * Hq + head) * splits + blockIdx.z) * span.stride;
-        float* p_hi = partial + (((size_t)(row0 + r_hi) * Hq + head) * splits + blockIdx.z) * span.stride;
-        const bool with_sums = tq == 0 && (span.width == 0 || v_col == 0);
-        if (with_sums && r_lo < n_q) { p_lo[0] = m_lo; p_lo[1] = l_lo; }
-        if (with_sums && r_hi < n_q) { p_hi[0] = m_hi; p_hi[1] = l_hi; }
-        p_lo += span.off + (span.width > 0 ? v_col : 0);
-        p_hi += span.off + (span.width > 0 ? v_col : 0);
+        const int stride = vdim + 2;
+        float* p_lo = partial + (((size_t)(row0 + r_lo) * Hq + head) * splits + blockIdx.z) * stride;
+        float* p_hi = partial + (((size_t)(row0 + r_hi) * Hq + head) * splits + blockIdx.z) * stride;
+        if (tq == 0 && r_lo < n_q) { p_lo[0] = m_lo; p_lo[1] = l_lo; }
+        if (tq == 0 && r_hi < n_q) { p_hi[0] = m_hi; p_hi[1] = l_hi; }
 #pragma unroll
-        for (int n = 0; n < kValueTiles; ++n) {      // (even offsets and strides: 8-byte stores)
+        for (int n = 0; n < kValueTiles; ++n) {
             if (n >= vtiles) continue;
             const int c = n * 8 + 2 * tq;
-            if (r_lo < n_q) *reinterpret_cast<float2*>(p_lo + c) = make_float2(o[n][0], o[n][1]);
-            if (r_hi < n_q) *reinterpret_cast<float2*>(p_hi + c) = make_float2(o[n][2], o[n][3]);
+            if (r_lo < n_q) { p_lo[2 + c] = o[n][0]; p_lo[3 + c] = o[n][1]; }
+            if (r_hi < n_q) { p_hi[2 + c] = o[n][2]; p_hi[3 + c] = o[n][3]; }
         }
         return;
     }
@@ -862,16 +857,16 @@ static int launch_tile(const void* q, const void* k_cache, const void* v_cache, 
                        const int* block_table, int table_width, const int* pooled_table, int pooled_width, const int* cu,
                        const int* start_pos, const int* tiles, int num_tiles, const float* v_table, int v_rot, int table_rows,
                        void* out, int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int pool,
-                       float* partial, int splits, ScoreExtras extras, ValueSpan span, void* stream) {
+                       float* partial, int splits, ScoreExtras extras, void* stream) {
     const size_t smem = (size_t)2 * kTileK * ((dim + 8) + (vdim + 8)) * sizeof(__nv_bfloat16);
     static size_t have = 0;
     ensure_dynamic_smem(pooled_attention_tile_kernel<kDimSteps, kValueTiles>, smem, have);
-    dim3 grid(num_tiles, Hq * (span.width > 0 ? (span.width + vdim - 1) / vdim : 1), splits);
+    dim3 grid(num_tiles, Hq, splits);
     pooled_attention_tile_kernel<kDimSteps, kValueTiles><<<grid, kTileThreads, smem, (cudaStream_t)stream>>>(
         (const __nv_bfloat16*)q, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, (const __nv_bfloat16*)kp_cache,
         (const __nv_bfloat16*)vp_cache, block_table, table_width, pooled_table, pooled_width, cu, start_pos, tiles, v_table, v_rot,
-        table_rows, (__nv_bfloat16*)out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits > 1 || span.width > 0 ? partial : nullptr,
-        splits, extras, span);
+        table_rows, (__nv_bfloat16*)out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, splits > 1 ? partial : nullptr, splits,
+        extras);
     return launch_status();
 }
 
@@ -885,17 +880,16 @@ static int tile_dispatch(const void* q, const void* k_cache, const void* v_cache
                                         int pooled_width, const int* cu, const int* start_pos, const int* tiles, int num_tiles,
                                         const float* v_table, int v_rot, int table_rows, void* out, int Hq, int Hkv, int dim,
                                         int vdim, int page_size, float scale, int window, int pool, float* partial, int splits,
-                                        ScoreExtras extras, ValueSpan span, void* stream) {
+                                        ScoreExtras extras, void* stream) {
     if (num_tiles <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hq > 65535 || dim <= 0 || dim % 16 || vdim <= 0 || vdim % 8 || page_size <= 0 || window <= 0
-        || pool < 0 || (v_rot & 1) || v_rot > vdim || table_rows <= 0 || extras.keep < 0 || (extras.keep > 0 && pool > 0)
-        || span.width % 8 || span.stride % 2 || span.off % 2)
+        || pool < 0 || (v_rot & 1) || v_rot > vdim || table_rows <= 0 || extras.keep < 0 || (extras.keep > 0 && pool > 0))
         return kBadSize;
-    if (dim > 128 || vdim > 128 || splits < 1 || splits > 64 || ((splits > 1 || span.width > 0) && partial == nullptr)) return kTooLarge;
+    if (dim > 128 || vdim > 128 || splits < 1 || splits > 64 || (splits > 1 && partial == nullptr)) return kTooLarge;
     if (extras.keep > 0) { kp_cache = k_cache; vp_cache = v_cache; pooled_table = block_table; pooled_width = table_width; }
 #define LB_TILE(DS, VT) return launch_tile<DS, VT>(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, pooled_table, \
         pooled_width, cu, start_pos, tiles, num_tiles, v_table, v_rot, table_rows, out, Hq, Hkv, dim, vdim, page_size, scale, window, pool, \
-        partial, splits, extras, span, stream)
+        partial, splits, extras, stream)
     const int ds = dim / 16, vt = vdim / 8;
     if (ds <= 2) { if (vt <= 4) LB_TILE(2, 4); if (vt <= 8) LB_TILE(2, 8); if (vt <= 12) LB_TILE(2, 12); LB_TILE(2, 16); }
     if (ds <= 4) { if (vt <= 4) LB_TILE(4, 4); if (vt <= 8) LB_TILE(4, 8); if (vt <= 12) LB_TILE(4, 12); LB_TILE(4, 16); }
@@ -916,8 +910,7 @@ extern "C" int lb_pooled_attention_tile(const void* q, const void* k_cache, cons
     // (with several CTAs per run the sink joins in the merge, once)
     const int code = tile_dispatch(q, k_cache, v_cache, kp_cache, vp_cache, block_table, table_width, pooled_table, pooled_width, cu,
                                    start_pos, tiles, num_tiles, v_table, v_rot, table_rows, out, Hq, Hkv, dim, vdim, page_size, scale,
-                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks, gate, gate_stride, keep},
-                                   ValueSpan{0, vdim + 2, 2}, stream);
+                                   window, pool, partial, splits, ScoreExtras{slopes, splits > 1 ? nullptr : sinks, gate, gate_stride, keep}, stream);
     if (code != 0 || splits <= 1 || num_tiles <= 0 || tokens <= 0) return code;
     dim3 grid(tokens, Hq);
     pooled_merge_kernel<__nv_bfloat16><<<grid, 32, 0, (cudaStream_t)stream>>>(partial, positions, nullptr, v_table, v_rot, table_rows,
@@ -930,9 +923,9 @@ extern "C" int lb_pooled_attention_tile(const void* q, const void* k_cache, cons
 // With w_g(i, j) the softmax weights of head g (its denominator holds the sink, which has no weight of its own), head h of
 // key/value head c applies sum_g M[h, g] w_g(i, j) to the values of c.  The mix moves behind the sum over the keys:
 //     o_h(i) = sum_g M[h, g] U_gc(i),     U_gc(i) = sum_j w_g(i, j) v_c(j)
-// so the attention kernels above sum the weights of every head over the values of ALL key/value heads (`ValueSpan`) in one
-// ordinary online softmax, and leave (maximum, sum, weighted values) per key range; this kernel joins the ranges and the
-// sink, divides, and mixes, all in float32.
+// so an attention kernel (the one with key ranges above, with a `ValueSpan`, or those of attention_talk.cu) sums the weights of
+// every head over the values of ALL key/value heads in one ordinary online softmax, and leaves (maximum, sum, weighted values)
+// per key range; this kernel joins the ranges and the sink, divides, and mixes, all in float32.
 // grid (tokens, Hkv, column blocks of kTalkCols), 256 threads: 256 / kTalkCols slices of the heads g share a column, their
 // sums meet in shared memory.  Dynamic shared memory: Hq * splits floats (what a range's sums are multiplied by).
 constexpr int kTalkOff = 8;               // floats in front of the value columns of a partial result
@@ -974,10 +967,8 @@ __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict
         for (int r = 0; r < kTalkHeads; ++r) acc[r] = 0.f;
         for (int g = slice; g < Hq; g += kSlices) {
             float u = 0.f;
-            for (int s = 0; s < splits; ++s) {
-                const float f = factor[g * splits + s];
-                if (f != 0.f) u += f * column[((size_t)g * splits + s) * stride];     // (a range without keys holds no sums)
-            }
+#pragma unroll 4
+            for (int s = 0; s < splits; ++s) u += factor[g * splits + s] * column[((size_t)g * splits + s) * stride];
 #pragma unroll
             for (int r = 0; r < kTalkHeads; ++r)
                 if (r < nr) acc[r] += mix[(size_t)r * Hq + g] * u;
@@ -997,8 +988,12 @@ __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict
     }
 }
 
-static int launch_talk_merge(const float* partial, const int* token_list, int tokens, const float* talk, const float* sinks, void* out,
+// partial: float32 [rows, Hq, splits, Hkv * vdim + kTalkOff], row by row of the batch or of `token_list`; talk: float32 [Hq, Hq];
+// sinks: float32 [Hq] or null; out: [tokens, Hq * vdim]
+extern "C" int lb_talk_merge(const float* partial, const int* token_list, int tokens, const float* talk, const float* sinks, void* out,
                              int Hq, int Hkv, int vdim, int splits, int dtype, void* stream) {
+    if (tokens <= 0) return kOk;
+    if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || vdim <= 0 || splits <= 0) return kBadSize;
     const size_t smem = (size_t)Hq * splits * sizeof(float);
     if (smem > 96 * 1024) return kTooLarge;
 #define LB_TALK(COLS) LB_DISPATCH_DTYPE(dtype, { \
@@ -1006,19 +1001,18 @@ static int launch_talk_merge(const float* partial, const int* token_list, int to
         ensure_dynamic_smem(talk_merge_kernel<T, COLS>, smem + 40 * 1024, have); \
         talk_merge_kernel<T, COLS><<<dim3(tokens, Hkv, (vdim + COLS - 1) / COLS), 256, smem, (cudaStream_t)stream>>>( \
             partial, token_list, talk, sinks, (T*)out, Hq, Hkv, vdim, splits); })
-    if (vdim <= 32) { LB_TALK(32); } else if (vdim <= 64) { LB_TALK(64); } else { LB_TALK(128); }
+    // few tokens: narrow column blocks, so that more CTAs and more slices of the heads share the ranges
+    if (vdim <= 32 || tokens <= 32) { LB_TALK(32); } else if (vdim <= 64) { LB_TALK(64); } else { LB_TALK(128); }
 #undef LB_TALK
     return launch_status();
 }
 
-extern "C" int lb_talk_partial_offset() { return kTalkOff; }
-
-// Attention over a window and `keep` first tokens with mixed weights.  talk: float32 [Hq, Hq]; sinks: float32 [Hq] or null;
-// partial: float32 scratch of num_tokens * Hq * splits * (Hkv * vdim + kTalkOff); dim up to 1024
+// The sums of every head's weights over a window and `keep` first tokens, for any sizes in either dtype (`lb_talk_merge` joins and
+// mixes them).  partial: float32 [num_tokens, Hq, splits, Hkv * vdim + kTalkOff]; dim up to 1024
 extern "C" int lb_talk_attention_split(const void* q, const void* k_cache, const void* v_cache, const int* block_table, int table_width,
                                        const int* token_req, const int* positions, const int* token_list, int num_tokens, float* partial,
-                                       void* out, const float* talk, const float* sinks, int Hq, int Hkv, int dim, int vdim, int page_size,
-                                       float scale, int window, int keep, int splits, int dtype, void* stream) {
+                                       int Hq, int Hkv, int dim, int vdim, int page_size, float scale, int window, int keep, int splits,
+                                       int dtype, void* stream) {
     if (num_tokens <= 0) return kOk;
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || dim <= 0 || vdim <= 0 || page_size <= 0 || window <= 0 || keep < 0 || splits <= 0 || splits > 65535)
         return kBadSize;
@@ -1034,28 +1028,7 @@ extern "C" int lb_talk_attention_split(const void* q, const void* k_cache, const
     if (per == 1) LB_SPLIT_PER(1) else if (per == 2) LB_SPLIT_PER(2) else LB_SPLIT_PER(4)
 #undef LB_SPLIT_PER
 #undef LB_SPLIT
-    if (code != 0) return code;
-    return launch_talk_merge(partial, token_list, num_tokens, talk, sinks, out, Hq, Hkv, vdim, splits, dtype, stream);
-}
-
-// The same for the long portions' runs on the tensor cores (see `lb_pooled_attention_tile`): the merge goes over ALL `tokens` rows,
-// those that no run covers get nothing of meaning.  bfloat16; dim a multiple of 16 up to 128, vdim a multiple of 8;
-// partial: float32 scratch of tokens * Hq * splits * (Hkv * vdim + kTalkOff)
-extern "C" int lb_talk_attention_tile(const void* q, const void* k_cache, const void* v_cache, const int* block_table, int table_width,
-                                      const int* cu, const int* start_pos, const int* tiles, int num_tiles, int tokens, float* partial,
-                                      void* out, const float* talk, const float* sinks, int Hq, int Hkv, int dim, int vdim, int page_size,
-                                      float scale, int window, int keep, int splits, void* stream) {
-    if (num_tiles <= 0 || tokens <= 0) return kOk;
-    if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || vdim <= 0) return kBadSize;
-    const int width = Hkv * vdim;
-    // value columns of a CTA: as few chunks as 128 columns allow, of about equal width
-    const int chunks = (width + 127) / 128, chunk = ((width + chunks - 1) / chunks + 7) / 8 * 8;
-    if ((long)Hq * chunks > 65535) return kTooLarge;
-    const int code = tile_dispatch(q, k_cache, v_cache, k_cache, v_cache, block_table, table_width, block_table, table_width, cu, start_pos, tiles,
-                                   num_tiles, nullptr, 0, 1, nullptr, Hq, Hkv, dim, chunk, page_size, scale, window, 0, partial, splits,
-                                   ScoreExtras{nullptr, nullptr, nullptr, 0, keep}, ValueSpan{width, width + kTalkOff, kTalkOff}, stream);
-    if (code != 0) return code;
-    return launch_talk_merge(partial, nullptr, tokens, talk, sinks, out, Hq, Hkv, vdim, splits, kBF16, stream);
+    return code;
 }
 
 // ------------------------------------------------------------------------------------------------------------------

@@ -2000,52 +2000,93 @@ def _talk_checks(q, k_cache, v_cache, block_table, token_index, positions, talk,
     return T, H, dim, G, vdim
 
 
-def talk_attention_split(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, token_req: torch.Tensor,
-                         positions: torch.Tensor, talk: torch.Tensor, scale: float, window: int, keep: int, splits: int,
-                         token_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
-                         sinks: torch.Tensor | None = None) -> torch.Tensor:
+def _talk_merge(partial, token_list, n: int, talk, sinks, out, H: int, G: int, vdim: int, splits: int) -> torch.Tensor:
+    f = _fn("attention_pooled", "lb_talk_merge", [c_void_p, c_void_p, c_int] + [c_void_p] * 3 + [c_int] * 5 + [c_void_p])
+    _check(f(_ptr(partial), _ptr(token_list), n, _ptr(talk), _ptr(sinks), _ptr(out), H, G, vdim, splits, _code(out), _stream()), "talk_merge",
+           f"({H} heads, {splits} ranges)")
+    return out
+
+
+def talk_step_ok(q: torch.Tensor, v_cache: torch.Tensor) -> bool:
+    """Does the tensor-core form for single tokens take these sizes (else: the float32 form, for any sizes)?"""
+    if not POOLED_TILE or q.dtype != torch.bfloat16:
+        return False
+    f = _fn("attention_talk", "lb_talk_step_ok", [c_int] * 4)
+    return bool(f(q.shape[1], v_cache.shape[2], q.shape[2], v_cache.shape[3]))
+
+
+def talk_splits(num_tokens: int, num_heads: int, num_kv_heads: int, value_dim: int, keys: int, tensor_cores: bool) -> int:
+    """Key ranges per token: enough CTAs to fill the GPU (twice where a CTA's buffers leave room for two), at least 64 keys each."""
+    if not tensor_cores:
+        return pooled_splits(num_tokens, num_kv_heads, keys)
+    width = num_kv_heads * value_dim
+    ctas = num_tokens * -(-num_heads // 16) * -(-width // 512)
+    return max(1, min(-(-keys // 64), (1 if width > 256 else 2) * _SM_COUNT // max(ctas, 1), 32))
+
+
+def talk_attention(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, token_req: torch.Tensor,
+                   positions: torch.Tensor, talk: torch.Tensor, scale: float, window: int, keep: int, keys: int,
+                   token_list: torch.Tensor | None = None, out: torch.Tensor | None = None,
+                   sinks: torch.Tensor | None = None, splits: int | None = None) -> torch.Tensor:
     """[tokens, heads * value_dim]: softmax attention over a window and the sequence's `keep` first tokens whose heads mix their
     weights before they are applied: head h applies sum_g talk[h, g] w_g(i, j) to the values of its own key/value head.  exp(sinks[g])
-    joins head g's denominator and is not mixed.  Every (listed) token's keys are cut into `splits` ranges that run side by side;
-    the kernel that joins them mixes (two launches, everything in float32)."""
+    joins head g's denominator and is not mixed.  Every (listed) token is taken by itself, its keys (at most `keys` of them) cut
+    into ranges that run side by side; the kernel that joins them mixes (two launches).  Sizes that the tensor cores do not take
+    and float32 run on float32 arithmetic throughout."""
     T, H, dim, G, vdim = _talk_checks(q, k_cache, v_cache, block_table, token_req, positions, talk, sinks, out)
     if out is None:
         out = torch.empty((T, H * vdim), dtype=q.dtype, device=q.device)
     n = T if token_list is None else token_list.numel()
+    mma = talk_step_ok(q, v_cache)
+    splits = splits or talk_splits(n, H, G, vdim, keys, mma)
     partial = torch.empty((n, H, splits, G * vdim + TALK_OFFSET), dtype=torch.float32, device=q.device)
-    f = _fn("attention_pooled", "lb_talk_attention_split", [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int] + [c_void_p] * 4 + [c_int] * 5
-            + [c_float] + [c_int] * 4 + [c_void_p])
-    _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(token_req), _ptr(positions), _ptr(token_list), n,
-             _ptr(partial), _ptr(out), _ptr(talk), _ptr(sinks), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits, _code(q), _stream()),
-           "talk_attention_split", f"(dim {dim}, value dim {vdim}, {G} key/value heads, {splits} ranges)", launches=2)
-    return out
+    args = [_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(token_req), _ptr(positions), _ptr(token_list), n,
+            _ptr(partial), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits]
+    types = [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int, c_void_p] + [c_int] * 5 + [c_float] + [c_int] * 3
+    detail = f"(dim {dim}, value dim {vdim}, {G} key/value heads, {splits} ranges)"
+    if mma:
+        _check(_fn("attention_talk", "lb_talk_step", types + [c_void_p])(*args, _stream()), "talk_step", detail)
+    else:
+        _check(_fn("attention_pooled", "lb_talk_attention_split", types + [c_int, c_void_p])(*args, _code(q), _stream()), "talk_attention_split", detail)
+    return _talk_merge(partial, token_list, n, talk, sinks, out, H, G, vdim, splits)
+
+
+_talk_tile_q = None
+
+
+def talk_tile_q() -> int:
+    """Query tokens per CTA of `talk_attention_tile` (the kernel's constant)."""
+    global _talk_tile_q
+    if _talk_tile_q is None:
+        _talk_tile_q = int(_fn("attention_talk", "lb_talk_tile_q", [])())
+    return _talk_tile_q
 
 
 def talk_attention_tile_ok(q: torch.Tensor, v_cache: torch.Tensor) -> bool:
-    """Does the tensor-core form take these sizes?  bfloat16, heads of a multiple of 16 up to 128 columns, value heads of a
-    multiple of 8."""
+    """Does the tensor-core form for prompt portions take these sizes?  bfloat16, heads of a multiple of 16 up to 128 columns,
+    value heads of a multiple of 8."""
     return POOLED_TILE and q.dtype == torch.bfloat16 and q.shape[2] % 16 == 0 and q.shape[2] <= 128 and v_cache.shape[3] % 8 == 0
 
 
 def talk_tile_splits(num_tiles: int, num_heads: int, width: int) -> int:
-    """CTAs that share a run's keys, as `pooled_tile_splits`, where the value columns of all heads already take several."""
-    return pooled_tile_splits(num_tiles, num_heads * -(-width // 128))
+    """CTAs that share a run's keys: 1 where the runs fill the GPU by themselves, up to 4 for a short lone prompt."""
+    return max(1, min(4, _SM_COUNT // max(num_tiles * num_heads * -(-width // 512), 1)))
 
 
 def talk_attention_tile(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, block_table: torch.Tensor, cu_seqlens: torch.Tensor,
                         start_pos: torch.Tensor, tiles: torch.Tensor, talk: torch.Tensor, scale: float, window: int, keep: int,
                         out: torch.Tensor, splits: int = 1, sinks: torch.Tensor | None = None) -> torch.Tensor:
-    """`talk_attention_split` for the long portions' runs of `pooled_attention_tile_q()` tokens on the tensor cores; the rows that no
-    run covers get nothing of meaning (the caller fills them afterwards)."""
+    """`talk_attention` for the long portions' runs of `talk_tile_q()` tokens (work list of `StepContext.long_portion_tiles`) on the
+    tensor cores; the rows that no run covers get nothing of meaning (the caller fills them afterwards)."""
     T, H, dim, G, vdim = _talk_checks(q, k_cache, v_cache, block_table, cu_seqlens, start_pos, talk, sinks, out)
     _i32(tiles, "tiles")
     partial = torch.empty((T, H, splits, G * vdim + TALK_OFFSET), dtype=torch.float32, device=q.device)
-    f = _fn("attention_pooled", "lb_talk_attention_tile", [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int] * 2 + [c_void_p] * 4 + [c_int] * 5
-            + [c_float] + [c_int] * 3 + [c_void_p])
+    f = _fn("attention_talk", "lb_talk_tile", [c_void_p] * 4 + [c_int] + [c_void_p] * 3 + [c_int, c_void_p] + [c_int] * 5 + [c_float] + [c_int] * 3
+            + [c_void_p])
     _check(f(_ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(block_table), block_table.shape[1], _ptr(cu_seqlens), _ptr(start_pos), _ptr(tiles), tiles.shape[0],
-             T, _ptr(partial), _ptr(out), _ptr(talk), _ptr(sinks), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits, _stream()),
-           "talk_attention_tile", f"(dim {dim}, value dim {vdim}, {G} key/value heads)", launches=2)
-    return out
+             _ptr(partial), H, G, dim, vdim, k_cache.shape[1], scale, window, keep, splits, _stream()), "talk_tile",
+           f"(dim {dim}, value dim {vdim}, {G} key/value heads)")
+    return _talk_merge(partial, None, T, talk, sinks, out, H, G, vdim, splits)
 
 
 # --------------------------------------------------------------------------- selective scan (a decay per channel and state)

@@ -22,10 +22,10 @@ class TalkingAttention(Part):
     Keys (rotated, at their true positions) and values are cached in pages; a page goes back once the window has passed it, except
     for those of the first tokens.  Rotation and cache store are one kernel (`K.qk_prepare`).  The mix moves behind the sum over
     the keys: every head's weights are summed over the values of ALL key/value heads in one online softmax, and the kernel that
-    joins the key ranges mixes the sums (`K.talk_attention_tile` for prompt portions of a bfloat16 engine, on the tensor cores;
-    `K.talk_attention_split` for decoded tokens, short portions, other sizes and float32 engines).  Angles, scores, weights,
+    joins the key ranges mixes the sums (`K.talk_attention_tile` for prompt portions of a bfloat16 engine; `K.talk_attention` for
+    decoded tokens, short portions, other sizes and float32 engines).  Angles, scores, weights,
     sums and the mix are 32-bit.  Tensors: q, k, v, talk, sink, o."""
-    kernels = ("attention_pooled", "rope", "linear_skinny", "gemm_tcgen05")
+    kernels = ("attention_talk", "attention_pooled", "rope", "linear_skinny", "gemm_tcgen05")
 
     def __init__(self, spec, perturb_init: bool = False, shared: dict | None = None):
         if spec.num_heads % spec.num_kv_heads:
@@ -70,19 +70,19 @@ class TalkingAttention(Part):
         table = ctx.block_tables[gi]
         most_keys = min(window + s.keep_first, ctx.max_context)
 
-        def few_rows(token_list=None, out=None, n=x.shape[0]):
-            return K.talk_attention_split(q, k_cache, v_cache, table, ctx.token_req, ctx.positions, self.talk, s.softmax_scale, window, s.keep_first,
-                                          K.pooled_splits(n, G, most_keys), token_list=token_list, out=out, sinks=self.sinks)
+        def few_rows(token_list=None, out=None):
+            return K.talk_attention(q, k_cache, v_cache, table, ctx.token_req, ctx.positions, self.talk, s.softmax_scale, window, s.keep_first,
+                                    most_keys, token_list=token_list, out=out, sinks=self.sinks)
 
         if ctx.has_long_portions and K.talk_attention_tile_ok(q, v_cache):
             # long portions on the tensor cores: runs of neighbouring tokens share their keys through shared memory
-            tiles, n_tiles = ctx.long_portion_tiles(K.pooled_attention_tile_q())
+            tiles, n_tiles = ctx.long_portion_tiles(K.talk_tile_q())
             short, n_short = ctx.short_portion_tokens()
             o = torch.empty((x.shape[0], H * s.value_dim), dtype=q.dtype, device=q.device)
             K.talk_attention_tile(q, k_cache, v_cache, table, ctx.cu_seqlens, ctx.start_pos, tiles, self.talk, s.softmax_scale, window,
                                   s.keep_first, o, splits=K.talk_tile_splits(n_tiles, H, G * s.value_dim), sinks=self.sinks)
             if n_short > 0:
-                few_rows(short, o, n_short)
+                few_rows(short, o)
         else:
             o = few_rows()
         return K.linear(o, self.o_w)
