@@ -926,18 +926,19 @@ extern "C" int lb_pooled_attention_tile(const void* q, const void* k_cache, cons
 // so an attention kernel (the one with key ranges above, with a `ValueSpan`, or those of attention_talk.cu) sums the weights of
 // every head over the values of ALL key/value heads in one ordinary online softmax, and leaves (maximum, sum, weighted values)
 // per key range; this kernel joins the ranges and the sink, divides, and mixes, all in float32.
-// grid (tokens, Hkv, column blocks of kTalkCols), 256 threads: 256 / kTalkCols slices of the heads g share a column, their
-// sums meet in shared memory.  Dynamic shared memory: Hq * splits floats (what a range's sums are multiplied by).
+// grid (tokens, Hkv, column blocks of kCols), 256 threads: a thread owns V neighbouring columns (16-byte loads with V = 4), the
+// 256 * V / kCols slices of the (head g, range) pairs share a column, their sums meet in shared memory.  Dynamic shared memory: Hq * splits
+// floats (what a range's sums are multiplied by).
 constexpr int kTalkOff = 8;               // floats in front of the value columns of a partial result
 constexpr int kTalkHeads = 8;             // output heads at a time
-template <typename T, int kTalkCols>
+template <typename T, int kCols, int V>
 __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict__ partial, const int* __restrict__ token_list,
                                                          const float* __restrict__ talk, const float* __restrict__ sinks,
                                                          T* __restrict__ out, int Hq, int Hkv, int vdim, int splits) {
-    constexpr int kSlices = 256 / kTalkCols;
+    constexpr int kSlices = 256 * V / kCols;
     extern __shared__ float factor[];                          // [Hq][splits]
-    __shared__ float red[kSlices][kTalkHeads][kTalkCols];
-    const int slot = blockIdx.x, c = blockIdx.y, col0 = blockIdx.z * kTalkCols;
+    __shared__ __align__(16) float red[kSlices][kTalkHeads][kCols];
+    const int slot = blockIdx.x, c = blockIdx.y, col0 = blockIdx.z * kCols;
     const int t = token_list != nullptr ? token_list[slot] : slot;
     if (t < 0) return;
     const int per = Hq / Hkv, stride = Hkv * vdim + kTalkOff;
@@ -945,8 +946,10 @@ __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict
     for (int g = threadIdx.x; g < Hq; g += blockDim.x) {
         const float* s0 = src + (size_t)g * splits * stride;
         float mm = sinks != nullptr ? sinks[g] : -INFINITY;
+#pragma unroll 4
         for (int s = 0; s < splits; ++s) mm = fmaxf(mm, s0[(size_t)s * stride]);
         float ll = sinks != nullptr ? expf(sinks[g] - mm) : 0.f;
+#pragma unroll 4
         for (int s = 0; s < splits; ++s) {
             const float m = s0[(size_t)s * stride], f = m == -INFINITY ? 0.f : expf(m - mm);
             factor[g * splits + s] = f;
@@ -956,29 +959,43 @@ __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict
         for (int s = 0; s < splits; ++s) factor[g * splits + s] *= inv;
     }
     __syncthreads();
-    const int slice = threadIdx.x / kTalkCols, col = threadIdx.x % kTalkCols;
-    const bool live = col0 + col < vdim;
-    const float* column = src + kTalkOff + c * vdim + col0 + (live ? col : 0);
+    const int slice = threadIdx.x / (kCols / V), col = threadIdx.x % (kCols / V) * V;
+    const float* column = src + kTalkOff + c * vdim + (col0 + col < vdim ? col0 + col : 0);
     for (int r0 = 0; r0 < per; r0 += kTalkHeads) {
         const int nr = min(kTalkHeads, per - r0);
         const float* mix = talk + (size_t)(c * per + r0) * Hq;
-        float acc[kTalkHeads];
+        float acc[kTalkHeads][V];
 #pragma unroll
-        for (int r = 0; r < kTalkHeads; ++r) acc[r] = 0.f;
-        for (int g = slice; g < Hq; g += kSlices) {
-            float u = 0.f;
-#pragma unroll 4
-            for (int s = 0; s < splits; ++s) u += factor[g * splits + s] * column[((size_t)g * splits + s) * stride];
+        for (int r = 0; r < kTalkHeads; ++r)
+#pragma unroll
+            for (int e = 0; e < V; ++e) acc[r][e] = 0.f;
+#pragma unroll 2
+        for (int p = slice; p < Hq * splits; p += kSlices) {          // (head, range) pairs
+            const float f = factor[p];
+            const float* at = column + (size_t)p * stride;
+            float u[V];
+            if (V == 4) {
+                const float4 x = *reinterpret_cast<const float4*>(at);
+                u[0] = f * x.x; u[1 % V] = f * x.y; u[2 % V] = f * x.z; u[3 % V] = f * x.w;
+            } else u[0] = f * at[0];
+            const int g = p / splits;
 #pragma unroll
             for (int r = 0; r < kTalkHeads; ++r)
-                if (r < nr) acc[r] += mix[(size_t)r * Hq + g] * u;
+                if (r < nr) {
+                    const float w = mix[(size_t)r * Hq + g];
+#pragma unroll
+                    for (int e = 0; e < V; ++e) acc[r][e] += w * u[e];
+                }
         }
         __syncthreads();
 #pragma unroll
-        for (int r = 0; r < kTalkHeads; ++r) red[slice][r][col] = acc[r];
+        for (int r = 0; r < kTalkHeads; ++r)
+            if (r < nr)
+#pragma unroll
+                for (int e = 0; e < V; ++e) red[slice][r][col + e] = acc[r][e];
         __syncthreads();
-        for (int i = threadIdx.x; i < nr * kTalkCols; i += blockDim.x) {
-            const int r = i / kTalkCols, cc = i % kTalkCols;
+        for (int i = threadIdx.x; i < nr * kCols; i += blockDim.x) {
+            const int r = i / kCols, cc = i % kCols;
             if (col0 + cc >= vdim) continue;
             float sum = 0.f;
 #pragma unroll
@@ -996,13 +1013,15 @@ extern "C" int lb_talk_merge(const float* partial, const int* token_list, int to
     if (Hq <= 0 || Hkv <= 0 || Hq % Hkv || Hkv > 65535 || vdim <= 0 || splits <= 0) return kBadSize;
     const size_t smem = (size_t)Hq * splits * sizeof(float);
     if (smem > 96 * 1024) return kTooLarge;
-#define LB_TALK(COLS) LB_DISPATCH_DTYPE(dtype, { \
+#define LB_TALK(COLS, V) LB_DISPATCH_DTYPE(dtype, { \
         static size_t have = 0; \
-        ensure_dynamic_smem(talk_merge_kernel<T, COLS>, smem + 40 * 1024, have); \
-        talk_merge_kernel<T, COLS><<<dim3(tokens, Hkv, (vdim + COLS - 1) / COLS), 256, smem, (cudaStream_t)stream>>>( \
+        ensure_dynamic_smem(talk_merge_kernel<T, COLS, V>, smem + 40 * 1024, have); \
+        talk_merge_kernel<T, COLS, V><<<dim3(tokens, Hkv, (vdim + COLS - 1) / COLS), 256, smem, (cudaStream_t)stream>>>( \
             partial, token_list, talk, sinks, (T*)out, Hq, Hkv, vdim, splits); })
-    // few tokens: narrow column blocks, so that more CTAs and more slices of the heads share the ranges
-    if (vdim <= 32 || tokens <= 32) { LB_TALK(32); } else if (vdim <= 64) { LB_TALK(64); } else { LB_TALK(128); }
+    // few tokens: narrow column blocks, so that more CTAs and more slices share the ranges
+    if (vdim % 4 == 0 && ((uintptr_t)partial & 15) == 0) {
+        if (tokens <= 32) { LB_TALK(32, 4); } else if (vdim <= 64) { LB_TALK(64, 4); } else { LB_TALK(128, 4); }
+    } else if (vdim <= 32 || tokens <= 32) { LB_TALK(32, 1); } else { LB_TALK(64, 1); }
 #undef LB_TALK
     return launch_status();
 }

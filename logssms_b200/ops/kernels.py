@@ -2007,12 +2007,17 @@ def _talk_merge(partial, token_list, n: int, talk, sinks, out, H: int, G: int, v
     return out
 
 
+_talk_step_sizes: dict = {}
+
+
 def talk_step_ok(q: torch.Tensor, v_cache: torch.Tensor) -> bool:
     """Does the tensor-core form for single tokens take these sizes (else: the float32 form, for any sizes)?"""
     if not POOLED_TILE or q.dtype != torch.bfloat16:
         return False
-    f = _fn("attention_talk", "lb_talk_step_ok", [c_int] * 4)
-    return bool(f(q.shape[1], v_cache.shape[2], q.shape[2], v_cache.shape[3]))
+    sizes = (q.shape[1], v_cache.shape[2], q.shape[2], v_cache.shape[3])
+    if sizes not in _talk_step_sizes:
+        _talk_step_sizes[sizes] = bool(_fn("attention_talk", "lb_talk_step_ok", [c_int] * 4)(*sizes))
+    return _talk_step_sizes[sizes]
 
 
 def talk_splits(num_tokens: int, num_heads: int, num_kv_heads: int, value_dim: int, keys: int, tensor_cores: bool) -> int:
