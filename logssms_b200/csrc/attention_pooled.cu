@@ -1005,6 +1005,72 @@ __global__ void __launch_bounds__(256) talk_merge_kernel(const float* __restrict
     }
 }
 
+// The same for many tokens: a warp takes a token's 128 neighbouring columns (of the Hkv * vdim), a lane four of them, and walks
+// the (head, range) pairs with several 16-byte loads in flight; nothing is shared between warps but the mix.
+// grid (ceil(tokens * column blocks / kMergeWarps)); dynamic shared memory: Hq * Hq floats, then Hq * splits floats per warp
+constexpr int kMergeWarps = 8;
+template <typename T>
+__global__ void __launch_bounds__(kMergeWarps * 32) talk_merge_rows_kernel(const float* __restrict__ partial, const int* __restrict__ token_list,
+                                                                           const float* __restrict__ talk, const float* __restrict__ sinks,
+                                                                           T* __restrict__ out, int tokens, int Hq, int Hkv, int vdim, int splits) {
+    extern __shared__ float merge_smem[];
+    float* mix = merge_smem;                                   // [Hq][Hq]
+    for (int i = threadIdx.x; i < Hq * Hq; i += blockDim.x) mix[i] = talk[i];
+    __syncthreads();
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+    float* factor = merge_smem + Hq * Hq + warp * Hq * splits;
+    const int per = Hq / Hkv, width = Hkv * vdim, stride = width + kTalkOff, blocks = (width + 127) / 128;
+    const long unit = (long)blockIdx.x * kMergeWarps + warp;
+    const long slot = unit / blocks;
+    if (slot >= tokens) return;
+    const int t = token_list != nullptr ? token_list[slot] : (int)slot;
+    if (t < 0) return;
+    const float* src = partial + (size_t)slot * Hq * splits * stride;
+    for (int g = lane; g < Hq; g += 32) {
+        const float* s0 = src + (size_t)g * splits * stride;
+        float mm = sinks != nullptr ? sinks[g] : -INFINITY;
+        for (int s = 0; s < splits; ++s) mm = fmaxf(mm, s0[(size_t)s * stride]);
+        float ll = sinks != nullptr ? expf(sinks[g] - mm) : 0.f;
+        for (int s = 0; s < splits; ++s) {
+            const float m = s0[(size_t)s * stride], f = m == -INFINITY ? 0.f : expf(m - mm);
+            factor[g * splits + s] = f;
+            ll += f * s0[(size_t)s * stride + 1];
+        }
+        const float inv = ll > 0.f ? 1.f / ll : 0.f;
+        for (int s = 0; s < splits; ++s) factor[g * splits + s] *= inv;
+    }
+    __syncwarp();
+    const int col = (int)(unit % blocks) * 128 + lane * 4;
+    if (col >= width) return;
+    const int c = col / vdim, d = col - c * vdim;
+    for (int r0 = 0; r0 < per; r0 += kTalkHeads) {
+        const int nr = min(kTalkHeads, per - r0);
+        const float* rows = mix + (size_t)(c * per + r0) * Hq;
+        float acc[kTalkHeads][4];
+#pragma unroll
+        for (int r = 0; r < kTalkHeads; ++r) acc[r][0] = acc[r][1] = acc[r][2] = acc[r][3] = 0.f;
+#pragma unroll 8
+        for (int p = 0; p < Hq * splits; ++p) {                 // (head, range) pairs
+            const float f = factor[p];
+            const float4 x = *reinterpret_cast<const float4*>(src + (size_t)p * stride + kTalkOff + col);
+            const int g = splits == 1 ? p : p / splits;
+#pragma unroll
+            for (int r = 0; r < kTalkHeads; ++r)
+                if (r < nr) {
+                    const float w = rows[(size_t)r * Hq + g] * f;
+                    acc[r][0] += w * x.x; acc[r][1] += w * x.y; acc[r][2] += w * x.z; acc[r][3] += w * x.w;
+                }
+        }
+#pragma unroll
+        for (int r = 0; r < kTalkHeads; ++r) {
+            if (r >= nr) continue;
+            T* dst = out + ((size_t)t * Hq + c * per + r0 + r) * vdim + d;
+#pragma unroll
+            for (int e = 0; e < 4; ++e) dst[e] = from_f32<T>(acc[r][e]);
+        }
+    }
+}
+
 // partial: float32 [rows, Hq, splits, Hkv * vdim + kTalkOff], row by row of the batch or of `token_list`; talk: float32 [Hq, Hq];
 // sinks: float32 [Hq] or null; out: [tokens, Hq * vdim]
 extern "C" int lb_talk_merge(const float* partial, const int* token_list, int tokens, const float* talk, const float* sinks, void* out,
@@ -1019,8 +1085,19 @@ extern "C" int lb_talk_merge(const float* partial, const int* token_list, int to
         talk_merge_kernel<T, COLS, V><<<dim3(tokens, Hkv, (vdim + COLS - 1) / COLS), 256, smem, (cudaStream_t)stream>>>( \
             partial, token_list, talk, sinks, (T*)out, Hq, Hkv, vdim, splits); })
     // few tokens: narrow column blocks, so that more CTAs and more slices share the ranges
-    if (vdim % 4 == 0 && ((uintptr_t)partial & 15) == 0) {
-        if (tokens <= 32) { LB_TALK(32, 4); } else if (vdim <= 64) { LB_TALK(64, 4); } else { LB_TALK(128, 4); }
+    const bool pieces = vdim % 4 == 0 && ((uintptr_t)partial & 15) == 0;
+    const size_t rows_smem = ((size_t)Hq * Hq + (size_t)kMergeWarps * Hq * splits) * sizeof(float);
+    if (pieces && tokens > 32 && rows_smem <= 96 * 1024) {
+        const long units = (long)tokens * ((Hkv * vdim + 127) / 128);
+        LB_DISPATCH_DTYPE(dtype, {
+            static size_t have = 0;
+            ensure_dynamic_smem(talk_merge_rows_kernel<T>, rows_smem, have);
+            talk_merge_rows_kernel<T><<<(unsigned)((units + kMergeWarps - 1) / kMergeWarps), kMergeWarps * 32, rows_smem, (cudaStream_t)stream>>>(
+                partial, token_list, talk, sinks, (T*)out, tokens, Hq, Hkv, vdim, splits); });
+        return launch_status();
+    }
+    if (pieces) {
+        if (tokens <= 32 || vdim <= 32) { LB_TALK(32, 4); } else { LB_TALK(64, 4); }
     } else if (vdim <= 32 || tokens <= 32) { LB_TALK(32, 1); } else { LB_TALK(64, 1); }
 #undef LB_TALK
     return launch_status();
